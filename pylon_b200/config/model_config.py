@@ -955,3 +955,143 @@ class RirusunConfig:
                     layer = replace(layer, left=replace(layer.left, bias_rows=int(table[0])))
             layers.append(layer)
         return replace(self, layers=tuple(layers))
+
+
+# ---------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class ZabusunAttention:
+    """The attending half of a Zabusun mixer: grouped-query attention whose weights are sigmoids of the scores (times ``scale``, plus a
+    learnt number per head) instead of a softmax; q and k RMS-normed per head and partly rotated; the heads gated."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Optional[RotarySpec] = None
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "ZabusunAttention":
+        heads, kv_heads, dim = _positive_int(data, "heads"), _positive_int(data, "kv_heads"), _positive_int(data, "dim")
+        if heads % kv_heads:
+            raise ConfigError(f"{where}: {heads} heads cannot be grouped over {kv_heads} kv_heads")
+        rot = None
+        if data.get("rot") is not None:
+            rot = RotarySpec.from_dict(_mapping(data, "rot"), where, ("factor", "original", "fast", "slow"))
+            if rot.dims > dim:
+                raise ConfigError(f"{where}: rot.dims {rot.dims} exceeds the head's dim {dim}")
+        return cls(heads, kv_heads, dim, _positive_int(data, "vdim"), _number(data, "scale"), rot)
+
+    def to_dict(self) -> dict[str, Any]:
+        data: dict[str, Any] = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale}
+        if self.rot is not None:
+            data["rot"] = self.rot.to_dict()
+        return data
+
+
+@dataclass(frozen=True)
+class ZabusunFeedForward:
+    """``dense``: one clamped gated unit of inner width ``ff``.  ``moe``: ``experts`` such units of which a token uses ``top``."""
+
+    kind: str
+    ff: int
+    limit: float
+    experts: Optional[int] = None
+    top: Optional[int] = None
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "ZabusunFeedForward":
+        kind = _require(data, "kind", str)
+        if kind not in ("dense", "moe"):
+            raise ConfigError(f"{where}: unknown feed-forward kind {kind!r} (dense, moe)")
+        unit = data if kind == "dense" else _mapping(data, "expert")
+        ff, limit = _positive_int(unit, "ff"), _number(unit, "limit")
+        if not limit > 0:
+            raise ConfigError(f"{where}: the feed-forward's limit must be positive")
+        if kind == "dense":
+            return cls(kind, ff, limit)
+        router = _mapping(data, "router")
+        experts, top = _positive_int(router, "experts"), _positive_int(router, "top")
+        if top > experts:
+            raise ConfigError(f"{where}: a token cannot use {top} of {experts} experts")
+        return cls(kind, ff, limit, experts, top)
+
+    def to_dict(self) -> dict[str, Any]:
+        unit = {"ff": self.ff, "limit": self.limit}
+        if self.kind == "dense":
+            return {"kind": "dense", **unit}
+        return {"kind": "moe", "expert": unit, "router": {"experts": self.experts, "top": self.top}}
+
+
+@dataclass(frozen=True)
+class ZabusunLayer:
+    """One layer: the ``parallel`` mixer (``left`` attends, ``right`` is a gated recurrence of ``right_width`` channels, their outputs
+    added with a factor each) and its feed-forward, or none."""
+
+    left: ZabusunAttention
+    right_width: int
+    left_scale: float
+    right_scale: float
+    mlp: Optional[ZabusunFeedForward] = None
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], index: int) -> "ZabusunLayer":
+        kind, where = _require(data, "type", str), f"layer {index}"
+        if kind != "parallel":
+            raise ConfigError(f"{where}: unknown type {kind!r} (parallel)")
+        mixer, mlp = _mapping(data, "mixer"), data.get("mlp")
+        if mlp is not None and not isinstance(mlp, dict):
+            raise ConfigError(f"{where}: 'mlp' must be an object or null")
+        return cls(ZabusunAttention.from_dict(_mapping(mixer, "left"), where), _positive_int(_mapping(mixer, "right"), "width"),
+                   _number(mixer, "left_scale"), _number(mixer, "right_scale"), None if mlp is None else ZabusunFeedForward.from_dict(mlp, where))
+
+    def to_dict(self) -> dict[str, Any]:
+        mixer = {"left": self.left.to_dict(), "left_scale": self.left_scale, "right": {"width": self.right_width}, "right_scale": self.right_scale}
+        return {"type": "parallel", "mixer": mixer, "mlp": None if self.mlp is None else self.mlp.to_dict()}
+
+
+@dataclass(frozen=True)
+class ZabusunConfig:
+    """Zabusun: a decoder whose sublayers read the residual stream as it is and whose norms stand on the sublayers' outputs.  Every
+    layer mixes tokens by sigmoid attention beside a minimal gated recurrence, then goes through a clamped gated unit, a mixture of
+    such units that a token enters times its router score, or nothing.  The embedding is normed, the head is the embedding table,
+    the logits are times a factor.
+
+    ``config.json`` names the model by ``"architecture": "Zabusun"``.  Field names follow its keys.
+    """
+
+    architecture: ClassVar[str] = "Zabusun"
+
+    vocab: int
+    width: int
+    layers: tuple[ZabusunLayer, ...]
+    norm_eps: float
+    logit_scale: float = 1.0
+    eos_token_ids: tuple[int, ...] = field(default_factory=tuple)
+
+    def __post_init__(self) -> None:
+        if not self.layers:
+            raise ConfigError("a model needs at least one layer")
+        if not self.norm_eps > 0:
+            raise ConfigError(f"norm.eps must be positive, got {self.norm_eps}")
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any]) -> "ZabusunConfig":
+        layers, eos = _require(data, "layers", list), data.get("eos_token_id")
+        return cls(
+            vocab=_positive_int(data, "vocab"),
+            width=_positive_int(data, "width"),
+            layers=tuple(ZabusunLayer.from_dict(layer, index) for index, layer in enumerate(layers)),
+            norm_eps=_number(_mapping(data, "norm"), "eps"),
+            logit_scale=1.0 if data.get("logit_scale") is None else _number(data, "logit_scale"),
+            eos_token_ids=() if eos is None else ((eos,) if isinstance(eos, int) else tuple(int(x) for x in eos)),
+        )
+
+    def to_dict(self) -> dict[str, Any]:
+        data: dict[str, Any] = {
+            "architecture": self.architecture, "vocab": self.vocab, "width": self.width, "layers": [layer.to_dict() for layer in self.layers],
+            "norm": {"eps": self.norm_eps}, "logit_scale": self.logit_scale,
+        }
+        if self.eos_token_ids:
+            data["eos_token_id"] = list(self.eos_token_ids)
+        return data

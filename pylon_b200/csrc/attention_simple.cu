@@ -18,6 +18,10 @@
 // With `bias` (float32 [bias_rows, nq]) the scaled (and capped) score of the key d = p - j positions back gets
 // bias[min(d, bias_rows - 1), h] added: a learnt function of the distance that is constant from bias_rows - 1 on.
 //
+// With `sigmoid` weights nothing is normalised: a visible key's weight is sigmoid(score + score_bias[h]) (score_bias float32 [nq] or
+// null).  `gate` ([tokens, >= nq] in the compute dtype, or null): head h's output is multiplied by sigmoid(gate[t, h]); `factor`
+// multiplies every output; the output's rows may lie out_stride elements apart.
+//
 // The keys of a token are walked in chunks of 128 positions aligned at position 0, so a
 // token's result depends on its position only, not on how the step was cut or batched.
 #include "common.cuh"
@@ -34,7 +38,8 @@ __global__ void __launch_bounds__(SIMPLE_THREADS) paged_attention_simple_kernel(
     const int* __restrict__ token_row, const int* __restrict__ block_table, int table_width, int page_size,
     int num_pages, int nq, int nkv, int d, int dv, int window, int chunk, float softcap, float scale,
     const float* __restrict__ sinks, long long k_row_stride, long long v_row_stride, int keep_first, const float* __restrict__ bias,
-    int bias_rows) {
+    int bias_rows, int sigmoid, const float* __restrict__ score_bias, const T* __restrict__ gate, long long gate_stride, float factor,
+    long long out_stride) {
   extern __shared__ long long shared[];
   long long* offsets = shared;                                      // [128] cache rows of the keys (page, head, slot), -1: none
   float* probs = reinterpret_cast<float*>(offsets + SIMPLE_THREADS);  // [128]
@@ -77,15 +82,21 @@ __global__ void __launch_bounds__(SIMPLE_THREADS) paged_attention_simple_kernel(
       }
     }
     offsets[tid] = offset;
-    const float chunk_max = block_max(score, scratch);
-    const float new_max = fmaxf(running_max, chunk_max);
-    // new_max is finite: the chunk holds at least key `pos` (or an earlier chunk did).
-    const float p = offset >= 0 ? expf(score - new_max) : 0.f;
-    probs[tid] = p;
-    const float chunk_sum = block_sum(p, scratch);  // also orders probs/offsets writes
-    const float rescale = running_max == -INFINITY ? 0.f : expf(running_max - new_max);
-    running_sum = running_sum * rescale + chunk_sum;
-    running_max = new_max;
+    float rescale = 1.f;
+    if (sigmoid) {
+      probs[tid] = offset >= 0 ? 1.f / (1.f + expf(-(score + (score_bias ? score_bias[h] : 0.f)))) : 0.f;
+      __syncthreads();
+    } else {
+      const float chunk_max = block_max(score, scratch);
+      const float new_max = fmaxf(running_max, chunk_max);
+      // new_max is finite: the chunk holds at least key `pos` (or an earlier chunk did).
+      const float p = offset >= 0 ? expf(score - new_max) : 0.f;
+      probs[tid] = p;
+      const float chunk_sum = block_sum(p, scratch);  // also orders probs/offsets writes
+      rescale = running_max == -INFINITY ? 0.f : expf(running_max - new_max);
+      running_sum = running_sum * rescale + chunk_sum;
+      running_max = new_max;
+    }
     const int valid = pos - c0 + 1 < SIMPLE_THREADS ? pos - c0 + 1 : SIMPLE_THREADS;
 #pragma unroll
     for (int k = 0; k < SIMPLE_MAX_DIMS_PER_THREAD; ++k) {
@@ -101,8 +112,10 @@ __global__ void __launch_bounds__(SIMPLE_THREADS) paged_attention_simple_kernel(
     }
     __syncthreads();
   }
-  T* orow = out + ((size_t)t * nq + h) * dv;
-  const float inv = running_sum > 0.f ? 1.f / running_sum : 0.f;
+  T* orow = out + (size_t)t * out_stride + (size_t)h * dv;
+  float inv = sigmoid ? 1.f : (running_sum > 0.f ? 1.f / running_sum : 0.f);
+  inv *= factor;
+  if (gate) inv *= 1.f / (1.f + expf(-to_float<T>(gate[(size_t)t * gate_stride + h])));
 #pragma unroll
   for (int k = 0; k < SIMPLE_MAX_DIMS_PER_THREAD; ++k) {
     const int e = tid + k * SIMPLE_THREADS;
@@ -120,7 +133,8 @@ extern "C" int pylon_paged_attention_simple(const void* q, long long q_token_str
                                             int page_size, int num_pages, int nq, int nkv, int d, int dv, int window,
                                             int chunk, float softcap, float scale, const float* sinks,
                                             long long k_row_stride, long long v_row_stride, int num_tokens, int dtype,
-                                            int keep_first, const float* bias, int bias_rows, cudaStream_t stream) {
+                                            int keep_first, const float* bias, int bias_rows, int sigmoid, const float* score_bias,
+                                            const void* gate, long long gate_stride, float factor, long long out_stride, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (d < 1 || d > 2048) PYLON_REFUSE("paged_attention_simple: head size %d is outside 1..2048", d);
   if (k_row_stride == 0) k_row_stride = d;
@@ -131,6 +145,8 @@ extern "C" int pylon_paged_attention_simple(const void* q, long long q_token_str
   if (chunk < 0 || softcap < 0.f) PYLON_REFUSE("paged_attention_simple: chunk %d, soft cap %f", chunk, softcap);
   if (keep_first < 0 || (keep_first > 0 && chunk > 0)) PYLON_REFUSE("paged_attention_simple: %d kept first keys (not with chunks)", keep_first);
   if (bias && bias_rows < 1) PYLON_REFUSE("paged_attention_simple: a bias table of %d rows", bias_rows);
+  if (out_stride == 0) out_stride = (long long)nq * dv;
+  if (out_stride < (long long)nq * dv || (score_bias && !sigmoid) || (sigmoid && sinks)) PYLON_REFUSE("paged_attention_simple: output rows %lld apart, a number per head on the scores without sigmoid weights, or a sink with them", out_stride);
   if (nkv < 1 || nq < 1 || nq % nkv) PYLON_REFUSE("paged_attention_simple: %d query heads over %d KV heads", nq, nkv);
   if (nq > 65535) PYLON_REFUSE("paged_attention_simple: %d query heads", nq);
   if (page_size < 1 || table_width < 1 || window < 0)
@@ -141,12 +157,13 @@ extern "C" int pylon_paged_attention_simple(const void* q, long long q_token_str
     paged_attention_simple_kernel<float><<<grid, SIMPLE_THREADS, smem, stream>>>(
         (const float*)q, q_token_stride, (const float*)k_pages, (const float*)v_pages, (float*)out, positions,
         token_row, block_table, table_width, page_size, num_pages, nq, nkv, d, dv, window, chunk, softcap, scale, sinks, k_row_stride, v_row_stride,
-        keep_first, bias, bias_rows);
+        keep_first, bias, bias_rows, sigmoid, score_bias, (const float*)gate, gate_stride, factor, out_stride);
   else if (dtype == PYLON_DTYPE_BF16)
     paged_attention_simple_kernel<__nv_bfloat16><<<grid, SIMPLE_THREADS, smem, stream>>>(
         (const __nv_bfloat16*)q, q_token_stride, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages,
         (__nv_bfloat16*)out, positions, token_row, block_table, table_width, page_size, num_pages, nq, nkv, d, dv,
-        window, chunk, softcap, scale, sinks, k_row_stride, v_row_stride, keep_first, bias, bias_rows);
+        window, chunk, softcap, scale, sinks, k_row_stride, v_row_stride, keep_first, bias, bias_rows, sigmoid, score_bias,
+        (const __nv_bfloat16*)gate, gate_stride, factor, out_stride);
   else
     PYLON_REFUSE("paged_attention_simple: unknown dtype %d", dtype);
   PYLON_CHECK_LAUNCH("paged_attention_simple");

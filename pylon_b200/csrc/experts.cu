@@ -10,6 +10,11 @@
 // router matrix may have `extra` rows behind the experts': their logits leave as sigmoid(z) in extra_out [T, extra] (the gate of an
 // expert that every token goes through, say).  An ungated expert is W_down act(W_up h): the first product applies act itself.
 //
+// The shares may also stay the plain scores (normalize 0), and a share may weigh what an expert reads instead of what it gives:
+// out = sum of expert_e(share_e * h).  An expert's first product is linear, so its sums are multiplied by the slot's share before the
+// unit (slot_share, written by the plan), and the rows are then added up as they are.  Activation 4 is the clamped gated unit:
+// g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + 1).
+//
 // Nothing here needs the host to know how many tokens an expert got, so the step stays one sequence of launches (and
 // can be captured): the (token, choice) pairs are sorted by expert into row tiles of ROWS slots, every expert's span
 // padded to whole tiles, and the grouped products run over the most tiles there can be; a tile beyond the last one, and
@@ -37,6 +42,15 @@ __device__ __forceinline__ float expert_activation(float x, int kind) {
   if (kind == 1) return fmaxf(x, 0.f);
   if (kind == 3) return 0.5f * x * (1.f + erff(x * 0.7071067811865476f));   // gelu, exact form
   return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
+
+// A gated unit: act(gate) * up, or (kind 4) the clamped one.
+__device__ __forceinline__ float expert_unit(float g, float u, int kind, float limit, float alpha) {
+  if (kind == 4) {
+    g = fminf(g, limit);
+    return g / (1.f + expf(-alpha * g)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  }
+  return expert_activation(g, kind) * u;
 }
 
 // The row of w that holds column n of the gate (half 0) or of the up projection (half 1): the two halves one after the other, or
@@ -83,6 +97,7 @@ struct RouteScored {
   const float* correction;   // [experts] or null
   int groups, keep;
   float share_eps;
+  int normalize;             // 0: the shares are the scores as they are
   int extra;                 // rows of the router behind the experts'
   float* extra_out;          // [T, extra]
 };
@@ -151,6 +166,7 @@ __device__ __forceinline__ void route_choose_scored(float* logits, float* choice
     }
     __syncwarp();
   }
+  if (!mode.normalize) return;
   const float inv = 1.f / (total + mode.share_eps);
   if (lane < top) share[t * top + lane] *= inv;
   for (int k = 32 + lane; k < top; k += 32) share[t * top + k] *= inv;
@@ -262,16 +278,20 @@ __global__ void __launch_bounds__(128) experts_route_block_kernel(const T* __res
 }
 
 // One block.  chosen [pairs]; slot_of [pairs] out; source [max_slots] out: the pair in a slot, or -1; tile_expert [max_tiles] out:
-// the expert of a row tile of tile_rows slots, or -1.  Shared memory: 2 * experts + 1 ints.
+// the expert of a row tile of tile_rows slots, or -1; slot_share [max_slots] out, or null: the share of the pair in a slot.  Shared memory: 2 * experts + 1 ints.
 __global__ void experts_plan_kernel(const int* __restrict__ chosen, int* __restrict__ slot_of, int* __restrict__ source,
-                                    int* __restrict__ tile_expert, int pairs, int experts, int max_slots, int max_tiles, int tile_rows) {
+                                    int* __restrict__ tile_expert, int pairs, int experts, int max_slots, int max_tiles, int tile_rows,
+                                    const float* __restrict__ share, float* __restrict__ slot_share) {
   extern __shared__ int plan[];
   grid_dependency_wait();
   allow_dependents();
   int* count = plan;                 // tokens per expert, then the next free slot of each
   int* first = plan + experts;       // first slot of each expert, [experts + 1]
   for (int e = threadIdx.x; e < experts; e += blockDim.x) count[e] = 0;
-  for (int s = threadIdx.x; s < max_slots; s += blockDim.x) source[s] = -1;
+  for (int s = threadIdx.x; s < max_slots; s += blockDim.x) {
+    source[s] = -1;
+    if (slot_share) slot_share[s] = 0.f;
+  }
   for (int tile = threadIdx.x; tile < max_tiles; tile += blockDim.x) tile_expert[tile] = -1;
   __syncthreads();
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&count[chosen[i]], 1);
@@ -294,6 +314,7 @@ __global__ void experts_plan_kernel(const int* __restrict__ chosen, int* __restr
     const int slot = atomicAdd(&count[chosen[i]], 1);   // the order inside an expert's span does not matter: rows do not see each other
     slot_of[i] = slot;
     source[slot] = i;
+    if (slot_share) slot_share[slot] = share[i];
   }
 }
 
@@ -304,7 +325,8 @@ template <typename T, bool GLU>
 __global__ void __launch_bounds__(256) experts_product_kernel(const T* __restrict__ a, long long lda, const T* __restrict__ w,
                                                               const int* __restrict__ source, const int* __restrict__ tile_expert,
                                                               int gathered, int divide, void* __restrict__ out_v, int n_out, int k_size,
-                                                              int kind, int interleaved, int act_out) {
+                                                              int kind, int interleaved, int act_out,
+                                                              const float* __restrict__ slot_share, float limit, float alpha) {
   constexpr int TN = 64, TK = 16;
   __shared__ float a_tile[EXPERT_ROWS][TK + 1];
   __shared__ float b_tile[GLU ? 2 : 1][TN][TK + 1];
@@ -366,11 +388,12 @@ __global__ void __launch_bounds__(256) experts_product_kernel(const T* __restric
     const int r = ty * 2 + i;
     if (rows[r] < 0) continue;
     const long long slot = (long long)tile * EXPERT_ROWS + r;
+    const float reads = GLU && slot_share ? slot_share[slot] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= n_out) continue;
-      if (GLU) ((T*)out_v)[slot * n_out + n] = from_float<T>(expert_activation(acc[0][i][j], kind) * acc[GLU ? 1 : 0][i][j]);
+      if (GLU) ((T*)out_v)[slot * n_out + n] = from_float<T>(expert_unit(reads * acc[0][i][j], reads * acc[GLU ? 1 : 0][i][j], kind, limit, alpha));
       else if (act_out) ((T*)out_v)[slot * n_out + n] = from_float<T>(expert_activation(acc[0][i][j], kind));   // an ungated expert's first product
       else ((float*)out_v)[slot * n_out + n] = acc[0][i][j];
     }
@@ -397,7 +420,8 @@ template <bool GLU>
 __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfloat16* __restrict__ a, long long lda,
                                                                   const __nv_bfloat16* __restrict__ w, const int* __restrict__ source,
                                                                   const int* __restrict__ tile_expert, int gathered, int divide,
-                                                                  void* __restrict__ out_v, int n_out, int k_size, int kind, int interleaved, int act_out) {
+                                                                  void* __restrict__ out_v, int n_out, int k_size, int kind, int interleaved, int act_out,
+                                                                  const float* __restrict__ slot_share, float limit, float alpha) {
   constexpr int TN = MMA_TN, TK = MMA_TK, LD = MMA_TK + MMA_PAD, G = GLU ? 2 : 1, MMA_STAGES = mma_stages(GLU);
   constexpr int A_ELEMENTS = EXPERT_ROWS * LD, STAGE_ELEMENTS = mma_stage_elements(GLU);
   extern __shared__ __align__(16) unsigned char mma_shared[];
@@ -489,6 +513,7 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
       const int r = 16 * i + group + 8 * half;
       if (rows[r] < 0) continue;
       const long long slot = (long long)tile * EXPERT_ROWS + r;
+      const float reads = GLU && slot_share ? slot_share[slot] : 1.f;
 #pragma unroll
       for (int j = 0; j < 2; ++j)
 #pragma unroll
@@ -496,13 +521,14 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
           const int n = n0 + 16 * warp + 8 * j + 2 * quad + e;
           if (n >= n_out) continue;
           const float value = acc[0][i][j][2 * half + e];
-          if (GLU) ((__nv_bfloat16*)out_v)[slot * n_out + n] = __float2bfloat16_rn(expert_activation(value, kind) * acc[G - 1][i][j][2 * half + e]);
+          if (GLU) ((__nv_bfloat16*)out_v)[slot * n_out + n] = __float2bfloat16_rn(expert_unit(reads * value, reads * acc[G - 1][i][j][2 * half + e], kind, limit, alpha));
           else if (act_out) ((__nv_bfloat16*)out_v)[slot * n_out + n] = __float2bfloat16_rn(expert_activation(value, kind));
           else ((float*)out_v)[slot * n_out + n] = value;
         }
     }
 }
 
+// share null: the rows are added up as they are.
 // out[t, c] = sum_k share[t, k] * y[slot_of[t * top + k], c], the choices in their order; y in float32 or in the compute dtype.
 // With `common` ([T, width] in C, an expert that every token goes through) and `gate` (float32 [T]): + gate[t] * common[t, c].
 template <typename Y, typename C>
@@ -516,7 +542,7 @@ __global__ void experts_gather_kernel(const Y* __restrict__ y, const int* __rest
   const long long t = item / width;
   const int c = (int)(item % width);
   float acc = 0.f;
-  for (int k = 0; k < top; ++k) acc = fmaf(share[t * top + k], to_float<Y>(y[(long long)slot_of[t * top + k] * width + c]), acc);
+  for (int k = 0; k < top; ++k) acc = fmaf(share ? share[t * top + k] : 1.f, to_float<Y>(y[(long long)slot_of[t * top + k] * width + c]), acc);
   if (common != nullptr) acc = fmaf(gate[t], to_float<C>(common[item]), acc);
   out[item] = acc;
 }
@@ -544,14 +570,14 @@ extern "C" int pylon_experts_row_tile() { return EXPERT_ROWS; }
 // scored != 0: the sigmoid form (see RouteScored); router is then float32 [experts + extra, width].
 extern "C" int pylon_experts_route(const void* h, long long ld, const float* router, const float* bias, int* chosen, float* share, int width,
                                    int experts, int top, int num_tokens, int dtype, int scored, const float* correction, int groups, int keep,
-                                   float share_eps, int extra, float* extra_out, cudaStream_t stream) {
+                                   float share_eps, int normalize, int extra, float* extra_out, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (experts < 1 || top < 1 || top > experts || experts > 2048) PYLON_REFUSE("experts_route: %d of %d experts (at most 2048)", top, experts);
   if (!scored && (correction || groups || extra)) PYLON_REFUSE("experts_route: a correction, groups and extra rows go with the sigmoid form");
   if (scored && (groups < 0 || (groups > 0 && (experts % groups || keep < 1 || keep > groups || top > keep * (experts / groups))) || extra < 0 || extra > 64 ||
                  (extra > 0 && !extra_out)))
     PYLON_REFUSE("experts_route: %d groups of which %d are kept for %d of %d experts, %d extra rows", groups, keep, top, experts, extra);
-  const RouteScored mode{scored ? 1 : 0, correction, groups, keep, share_eps, extra, extra_out};
+  const RouteScored mode{scored ? 1 : 0, correction, groups, keep, share_eps, normalize, extra, extra_out};
   const int per_token = experts + extra + (scored ? experts + groups : 0);
   if (num_tokens < 512) {   // a step of few tokens wants many threads a token
     const size_t smem = (size_t)(4 * 8 + per_token) * sizeof(float);
@@ -575,12 +601,13 @@ extern "C" int pylon_experts_route(const void* h, long long ld, const float* rou
 
 // tile_rows: the slots of a row tile (pylon_experts_row_tile() for the products of this file, 128 for the grouped tcgen05 product).
 extern "C" int pylon_experts_plan(const int* chosen, int* slot_of, int* source, int* tile_expert, int pairs, int experts, int max_slots,
-                                  int max_tiles, int tile_rows, cudaStream_t stream) {
+                                  int max_tiles, int tile_rows, const float* share, float* slot_share, cudaStream_t stream) {
   if (pairs <= 0) return 0;
+  if (slot_share && !share) PYLON_REFUSE("experts_plan: shares per slot need the shares per choice");
   if (tile_rows < 1 || max_slots < pairs || (long long)max_tiles * tile_rows < max_slots)
     PYLON_REFUSE("experts_plan: %d slots in %d tiles of %d for %d pairs", max_slots, max_tiles, tile_rows, pairs);
   launch_dependent(experts_plan_kernel, dim3(1), dim3(1024), (size_t)(2 * experts + 1) * sizeof(int), stream, chosen, slot_of, source, tile_expert,
-                   pairs, experts, max_slots, max_tiles, tile_rows);
+                   pairs, experts, max_slots, max_tiles, tile_rows, share, slot_share);
   PYLON_CHECK_LAUNCH("experts_plan");
 }
 
@@ -598,17 +625,17 @@ static void allow_mma_shared_memory() {
 // glu == 2: no gate, but the activation on the product itself, out in dtype (the first product of an ungated expert).
 extern "C" int pylon_experts_product(const void* a, long long lda, const void* w, const int* source, const int* tile_expert, int gathered,
                                      int divide, void* out, int n_out, int k_size, int max_tiles, int glu, int kind, int interleaved, int dtype,
-                                     cudaStream_t stream) {
+                                     const float* slot_share, float limit, float alpha, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
   const int act_out = glu == 2 ? 1 : 0;
   if (act_out) glu = 0;
-  if (n_out <= 0 || k_size <= 0 || divide < 1 || kind < 0 || kind > 3) PYLON_REFUSE("experts_product: n %d, k %d, divide %d, activation %d", n_out, k_size, divide, kind);
+  if (n_out <= 0 || k_size <= 0 || divide < 1 || kind < 0 || kind > 4 || (kind == 4 && glu && !(limit > 0.f)) || (kind == 4 && act_out)) PYLON_REFUSE("experts_product: n %d, k %d, divide %d, activation %d", n_out, k_size, divide, kind);
   if (max_tiles > 65535) PYLON_REFUSE("experts_product: %d row tiles", max_tiles);
   if (interleaved && (!glu || n_out % 8)) PYLON_REFUSE("experts_product: interleaved rows need a gated product of a multiple of 8 columns, got %d", n_out);
   const dim3 grid((unsigned)((n_out + 63) / 64), (unsigned)max_tiles);
   if (dtype == PYLON_DTYPE_F32) {
-    if (glu) launch_dependent(experts_product_kernel<float, true>, grid, dim3(256), 0, stream, (const float*)a, lda, (const float*)w, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out);
-    else launch_dependent(experts_product_kernel<float, false>, grid, dim3(256), 0, stream, (const float*)a, lda, (const float*)w, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out);
+    if (glu) launch_dependent(experts_product_kernel<float, true>, grid, dim3(256), 0, stream, (const float*)a, lda, (const float*)w, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
+    else launch_dependent(experts_product_kernel<float, false>, grid, dim3(256), 0, stream, (const float*)a, lda, (const float*)w, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
   } else if (dtype == PYLON_DTYPE_BF16) {
     const __nv_bfloat16* ab = (const __nv_bfloat16*)a;
     const __nv_bfloat16* wb = (const __nv_bfloat16*)w;
@@ -616,14 +643,14 @@ extern "C" int pylon_experts_product(const void* a, long long lda, const void* w
     if (vectors) {
       if (glu) {
         allow_mma_shared_memory<true>();
-        launch_dependent(experts_product_mma_kernel<true>, grid, dim3(128), mma_shared_bytes(true), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out);
+        launch_dependent(experts_product_mma_kernel<true>, grid, dim3(128), mma_shared_bytes(true), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
       } else {
         allow_mma_shared_memory<false>();
-        launch_dependent(experts_product_mma_kernel<false>, grid, dim3(128), mma_shared_bytes(false), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out);
+        launch_dependent(experts_product_mma_kernel<false>, grid, dim3(128), mma_shared_bytes(false), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
       }
     } else {
-      if (glu) launch_dependent(experts_product_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out);
-      else launch_dependent(experts_product_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out);
+      if (glu) launch_dependent(experts_product_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
+      else launch_dependent(experts_product_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
     }
   } else PYLON_REFUSE("experts_product: unknown dtype %d", dtype);
   PYLON_CHECK_LAUNCH("experts_product");

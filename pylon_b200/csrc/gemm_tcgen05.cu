@@ -176,6 +176,7 @@ struct RotateArgs {
   // the gated unit of a SWIGLU epilogue: limit 0 is silu(gate) * up; limit > 0 the clamped unit,
   // min(gate, limit) * sigmoid(alpha * min(gate, limit)) * (clamp(up, -limit, limit) + 1)
   float unit_limit = 0.f, unit_alpha = 1.f;
+  const float* unit_row_scale = nullptr;   // not null: a row's sums of gate and up are multiplied by its number before the unit (a row of the operand times it)
 };
 enum TcMode { TC_PLAIN = 0, TC_SWIGLU = 1, TC_ROTATE = 2 };
 
@@ -410,6 +411,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(const __gri
       tc_fence_after();
       const int row0 = m0 + quarter * 32;
       const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + buffer * BN;
+      const float row_scale = SWIGLU && rot.unit_row_scale && row0 + lane < M ? rot.unit_row_scale[row0 + lane] : 1.f;
       if constexpr (MODE == TC_ROTATE) {
         rotate_epilogue<BN, D>(rot, taddr, my_staging, row0, n0, M, lane);
       } else
@@ -428,8 +430,8 @@ __global__ void __launch_bounds__(TC_THREADS, 1) gemm_tcgen05_kernel(const __gri
             for (int group = 0; group < 2; ++group)
 #pragma unroll
               for (int j = 0; j < 8; j += 2) {
-                const float g0 = __uint_as_float(raw[group * 16 + j]), g1 = __uint_as_float(raw[group * 16 + j + 1]);
-                const float u0 = __uint_as_float(raw[group * 16 + 8 + j]), u1 = __uint_as_float(raw[group * 16 + 8 + j + 1]);
+                const float g0 = row_scale * __uint_as_float(raw[group * 16 + j]), g1 = row_scale * __uint_as_float(raw[group * 16 + j + 1]);
+                const float u0 = row_scale * __uint_as_float(raw[group * 16 + 8 + j]), u1 = row_scale * __uint_as_float(raw[group * 16 + 8 + j + 1]);
                 packed[group * 4 + j / 2] = pack2(gated_unit_fast(g0, u0, rot.unit_limit, rot.unit_alpha), gated_unit_fast(g1, u1, rot.unit_limit, rot.unit_alpha));
               }
           } else {
@@ -507,7 +509,7 @@ static bool make_map(CUtensorMap* map, const void* base, long long rows, long lo
 template <int BN, bool SWIGLU>
 static int launch_tcgen05(const CUtensorMap& map_a, const CUtensorMap& map_b, __nv_bfloat16* c, int M, int N, int K, long long ldc,
                           int* error, int sm_count, cudaStream_t stream, float unit_limit = 0.f, float unit_alpha = 1.f,
-                          const int* tile_group = nullptr, int group_rows = 0) {
+                          const int* tile_group = nullptr, int group_rows = 0, const float* unit_row_scale = nullptr) {
   auto kernel = gemm_tcgen05_kernel<BN, SWIGLU ? TC_SWIGLU : TC_PLAIN, 128>;
   static bool configured_on[pylon::MAX_DEVICES] = {};   // function attributes belong to a device
   bool& configured = configured_on[pylon::current_device_slot()];
@@ -523,6 +525,7 @@ static int launch_tcgen05(const CUtensorMap& map_a, const CUtensorMap& map_b, __
   RotateArgs unit{};
   unit.unit_limit = unit_limit;
   unit.unit_alpha = unit_alpha;
+  unit.unit_row_scale = unit_row_scale;
   launch_dependent<LAUNCH_GEMM>(kernel, dim3(blocks), dim3(TC_THREADS), TcShared<BN>::BYTES, stream, map_a, map_b, map_c, M, N, K, error, unit, tile_group, group_rows);
   PYLON_CHECK_LAUNCH("gemm_tcgen05");
 }
@@ -561,7 +564,7 @@ extern "C" int pylon_gemm_tcgen05_force_tile(int columns) {
 // error: one int in device memory; the kernel sets it non-zero if one of its waits ran out (the result is then void).
 static int gemm_tcgen05_entry(const void* x, const void* w, void* y, int M, int N, int K, long long ldx, long long ldw,
                              long long ldy, int swiglu, float unit_limit, float unit_alpha, int* error, int sm_count, cudaStream_t stream,
-                             const int* tile_group = nullptr, int groups = 1) {
+                             const int* tile_group = nullptr, int groups = 1, const float* unit_row_scale = nullptr) {
   using namespace pylon;
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8 || ldx % 8 || ldw % 8 || ldy % 8) PYLON_REFUSE("gemm_tcgen05: K = %d and the row strides must be multiples of 8", K);
@@ -592,14 +595,14 @@ static int gemm_tcgen05_entry(const void* x, const void* w, void* y, int M, int 
   __nv_bfloat16* out = (__nv_bfloat16*)y;
 #define PYLON_TC_CASE(BN_)                                                                                          \
   if (bn == BN_) {                                                                                                  \
-    if (swiglu) return launch_tcgen05<BN_, true>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream, unit_limit, unit_alpha, tile_group, N); \
+    if (swiglu) return launch_tcgen05<BN_, true>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream, unit_limit, unit_alpha, tile_group, N, unit_row_scale); \
     return launch_tcgen05<BN_, false>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream, 0.f, 1.f, tile_group, N);                          \
   }
   PYLON_TC_CASE(256) PYLON_TC_CASE(192)
 #undef PYLON_TC_CASE
   if (bn == 288) return launch_tcgen05<288, false>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream);
   if (bn == 160) return launch_tcgen05<160, false>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream);
-  if (swiglu) return launch_tcgen05<128, true>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream, unit_limit, unit_alpha, tile_group, N);
+  if (swiglu) return launch_tcgen05<128, true>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream, unit_limit, unit_alpha, tile_group, N, unit_row_scale);
   return launch_tcgen05<128, false>(map_a, map_b, out, M, N, K, ldy, error, sm_count, stream, 0.f, 1.f, tile_group, N);
 }
 
@@ -607,11 +610,14 @@ static int gemm_tcgen05_entry(const void* x, const void* w, void* y, int M, int 
 // x's row tile i are multiplied by group tile_group[i]'s matrix; a tile whose entry is negative is passed over and its rows of y are
 // left as they are.  tile_group: int32 in device memory, one entry per 128 rows of x.  Where N is not a whole number of tile widths
 // the last tile's operand reaches into the next group's rows (or past the end, which reads zeros); those columns are never stored.
+// With swiglu: limit > 0 takes the clamped unit of pylon_gemm_tcgen05_glu_clamped, and row_scale (float32 [M], or null) multiplies every
+// row's sums before the unit.
 extern "C" int pylon_gemm_tcgen05_grouped(const void* x, const void* w, void* y, int M, int N, int K, long long ldx, long long ldw,
-                                          long long ldy, int swiglu, const int* tile_group, int groups, int* error, int sm_count,
-                                          cudaStream_t stream) {
+                                          long long ldy, int swiglu, float limit, float alpha, const float* row_scale, const int* tile_group,
+                                          int groups, int* error, int sm_count, cudaStream_t stream) {
+  if (limit < 0.f || (row_scale && !swiglu)) PYLON_REFUSE("gemm_tcgen05_grouped: limit %f, or row factors without a gated unit", limit);
   if (!tile_group || groups < 1) PYLON_REFUSE("gemm_tcgen05_grouped: the row tiles' groups are needed");
-  return gemm_tcgen05_entry(x, w, y, M, N, K, ldx, ldw, ldy, swiglu, 0.f, 1.f, error, sm_count, stream, tile_group, groups);
+  return gemm_tcgen05_entry(x, w, y, M, N, K, ldx, ldw, ldy, swiglu, limit, alpha, error, sm_count, stream, tile_group, groups, row_scale);
 }
 
 extern "C" int pylon_gemm_tcgen05_bf16(const void* x, const void* w, void* y, int M, int N, int K, long long ldx, long long ldw,

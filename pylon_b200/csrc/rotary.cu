@@ -25,11 +25,11 @@ __device__ __forceinline__ void rotate_pairs(float* buf, const float* __restrict
   }
 }
 
-// buf[0 .. n) divided by its root mean square, times weight (or 1).
-__device__ __forceinline__ void unit_rms(float* buf, int n, const float* __restrict__ weight, float eps, int lane) {
+// buf[0 .. n) divided by its root mean square, times weight (or 1).  `size`: how many of the n elements are the vector's own; the rest are zeros.
+__device__ __forceinline__ void unit_rms(float* buf, int n, int size, const float* __restrict__ weight, float eps, int lane) {
   float squares = 0.f;
   for (int e = lane; e < n; e += 32) squares = fmaf(buf[e], buf[e], squares);
-  const float inv = rsqrtf(warp_sum(squares) / n + eps);
+  const float inv = rsqrtf(warp_sum(squares) / size + eps);
   for (int e = lane; e < n; e += 32) buf[e] *= weight ? inv * weight[e] : inv;
 }
 
@@ -41,7 +41,7 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
     T* __restrict__ qkv, long long ld, const float* __restrict__ bias, const float* __restrict__ cos_table, const float* __restrict__ sin_table,
     int rot, int layout, int table_positions, int norm_mode, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
     const int* __restrict__ positions, const int* __restrict__ token_row, const int* __restrict__ block_table, int table_width, int page_size,
-    T* __restrict__ k_pages, T* __restrict__ v_pages, int num_pages, int nq, int nkv, int d, int dv, int num_tokens, int* __restrict__ error_word) {
+    T* __restrict__ k_pages, T* __restrict__ v_pages, int num_pages, int nq, int nkv, int d, int dv, int norm_size, int num_tokens, int* __restrict__ error_word) {
   extern __shared__ float rotary_shared[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int widest = d > dv ? d : dv;
@@ -62,7 +62,7 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
   if (!is_v) {
     const float* weight = is_q ? q_weight : k_weight;
     if (norm_mode == 1) {
-      unit_rms(buf, d, weight, eps, lane);
+      unit_rms(buf, d, norm_size, weight, eps, lane);
       __syncwarp();
     }
     if (rot > 0 && pos < table_positions) {
@@ -70,7 +70,7 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
       __syncwarp();
     }
     if (norm_mode == 2) {
-      unit_rms(buf, d, weight, eps, lane);
+      unit_rms(buf, d, norm_size, weight, eps, lane);
       __syncwarp();
     }
   }
@@ -86,6 +86,102 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
     dst = (is_v ? v_pages : k_pages) + (((size_t)page * nkv + head) * page_size + pos % page_size) * width;
   }
   for (int e = lane; e < width; e += 32) dst[e] = from_float<T>(buf[e]);
+}
+
+// The same for bfloat16 rows without biases whose pairs lie rot / 2 apart, rot a multiple of 16: `lanes` (a power of two) lanes share a
+// head, each with 8 neighbouring elements as one 16-byte piece; the rotation partners of a lane's elements are all in one other lane.
+__device__ __forceinline__ void unpack_8(float (&x)[8], const uint4& raw) {
+  const unsigned words[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 pair = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&words[i]));
+    x[2 * i] = pair.x; x[2 * i + 1] = pair.y;
+  }
+}
+__device__ __forceinline__ void load_8(float (&x)[8], const float* from) {
+  const float4 low = *reinterpret_cast<const float4*>(from), high = *reinterpret_cast<const float4*>(from + 4);
+  x[0] = low.x; x[1] = low.y; x[2] = low.z; x[3] = low.w; x[4] = high.x; x[5] = high.y; x[6] = high.z; x[7] = high.w;
+}
+
+__global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_vec_kernel(
+    __nv_bfloat16* __restrict__ qkv, long long ld, const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot, int table_positions,
+    int norm_mode, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps, const int* __restrict__ positions,
+    const int* __restrict__ token_row, const int* __restrict__ block_table, int table_width, int page_size, __nv_bfloat16* __restrict__ k_pages,
+    __nv_bfloat16* __restrict__ v_pages, int num_pages, int nq, int nkv, int d, int dv, int norm_size, int lanes, long long items,
+    int* __restrict__ error_word) {
+  const long long thread = (long long)blockIdx.x * ROTARY_THREADS + threadIdx.x;
+  const long long item = thread / lanes;
+  const int mine = (int)(thread % lanes) * 8;   // this lane's first element
+  const int per_token = nq + 2 * nkv;
+  const bool there = item < items;
+  const int t = there ? (int)(item / per_token) : 0, hh = there ? (int)(item % per_token) : 0;
+  const int row = there ? token_row[t] : -1;    // negative: a padding token, nothing of it is kept
+  const int pos = row >= 0 ? positions[t] : 0;
+  const bool is_q = hh < nq, is_v = hh >= nq + nkv;
+  const int width = is_v ? dv : d, half = rot >> 1;
+  const bool turned = !is_v && mine < rot && pos < table_positions;
+  float c[8], s[8], x[8];
+  if (turned) {   // position, page and angles do not depend on the kernel ahead
+    const size_t angle = (size_t)pos * half + (mine < half ? mine : mine - half);
+    load_8(c, cos_table + angle);
+    load_8(s, sin_table + angle);
+  }
+  int page = -1;
+  if (row >= 0 && !is_q) {
+    const int logical = pos / page_size;
+    page = logical < table_width ? block_table[(size_t)row * table_width + logical] : -1;
+  }
+  const bool live = row >= 0 && mine < width;
+  __nv_bfloat16* src = qkv + (size_t)t * ld + (is_v ? (nq + nkv) * d + (hh - nq - nkv) * dv : hh * d) + mine;
+  grid_dependency_wait();
+  allow_dependents();
+  const uint4 raw = live ? *reinterpret_cast<const uint4*>(src) : make_uint4(0u, 0u, 0u, 0u);
+  uint4 result = raw;
+  unpack_8(x, raw);
+  auto unit = [&]() {   // every lane of a warp comes here; a value head keeps what it has
+    float squares = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) squares = fmaf(x[i], x[i], squares);
+    for (int offset = lanes >> 1; offset > 0; offset >>= 1) squares += __shfl_xor_sync(0xffffffffu, squares, offset);
+    if (is_v || mine >= width) return;
+    const float inv = rsqrtf(squares / norm_size + eps);
+    const float* weight = is_q ? q_weight : k_weight;
+    float w[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+    if (weight) load_8(w, weight + mine);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] *= inv * w[i];
+  };
+  if (norm_mode == 1) unit();
+  if (rot > 0) {
+    const int apart = half >> 3;   // lanes between the two elements of a pair
+    const int lane = threadIdx.x & 31, partner = mine < half ? lane + apart : lane - apart;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float other = __shfl_sync(0xffffffffu, x[i], partner & 31);
+      if (turned) x[i] = mine < half ? x[i] * c[i] - other * s[i] : x[i] * c[i] + other * s[i];
+    }
+  }
+  if (norm_mode == 2) unit();
+  if (!live) return;
+  if (!is_v) {
+    unsigned words[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const __nv_bfloat162 pair = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+      words[i] = *reinterpret_cast<const unsigned*>(&pair);
+    }
+    result = make_uint4(words[0], words[1], words[2], words[3]);
+  }
+  if (is_q) {
+    *reinterpret_cast<uint4*>(src) = result;
+    return;
+  }
+  if (page < 0 || page >= num_pages) {
+    if (mine == 0 && error_word) atomicMax(error_word, PYLON_ERROR_BAD_PAGE);
+    return;
+  }
+  const int head = is_v ? hh - nq - nkv : hh - nq;
+  *reinterpret_cast<uint4*>((is_v ? v_pages : k_pages) + (((size_t)page * nkv + head) * page_size + pos % page_size) * width + mine) = result;
 }
 
 // One block per token.  down [T, ld] holds [query latent: q_rank | key/value latent: kv_rank | shared rotated key part: rot_dim].
@@ -159,8 +255,9 @@ using namespace pylon;
 extern "C" int pylon_qkv_rotate_write(void* qkv, long long ld, const float* bias, const float* cos_table, const float* sin_table, int rot, int layout,
                                       int table_positions, int norm_mode, const float* q_weight, const float* k_weight, float eps, const int* positions,
                                       const int* token_row, const int* block_table, int table_width, int page_size, void* k_pages, void* v_pages,
-                                      int num_pages, int nq, int nkv, int d, int dv, int num_tokens, int dtype, int* error_word, cudaStream_t stream) {
+                                      int num_pages, int nq, int nkv, int d, int dv, int norm_size, int num_tokens, int dtype, int* error_word, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
+  if (norm_size < 1 || norm_size > d) PYLON_REFUSE("qkv_rotate_write: a norm over %d of %d elements", norm_size, d);
   if (nq < 1 || nkv < 1 || d < 1 || dv < 1 || d > 2048 || dv > 2048) PYLON_REFUSE("qkv_rotate_write: %d / %d heads of %d and %d", nq, nkv, d, dv);
   if (rot < 0 || rot > d || rot % 2 || (rot > 0 && (!cos_table || !sin_table))) PYLON_REFUSE("qkv_rotate_write: %d rotated elements of %d", rot, d);
   if (norm_mode < 0 || norm_mode > 2 || page_size < 1 || table_width < 1) PYLON_REFUSE("qkv_rotate_write: norm mode %d, page size %d, table width %d", norm_mode, page_size, table_width);
@@ -170,11 +267,20 @@ extern "C" int pylon_qkv_rotate_write(void* qkv, long long ld, const float* bias
   if (dtype == PYLON_DTYPE_F32)
     qkv_rotate_write_kernel<float><<<blocks, ROTARY_THREADS, smem, stream>>>(
         (float*)qkv, ld, bias, cos_table, sin_table, rot, layout, table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row, block_table,
-        table_width, page_size, (float*)k_pages, (float*)v_pages, num_pages, nq, nkv, d, dv, num_tokens, error_word);
-  else if (dtype == PYLON_DTYPE_BF16)
+        table_width, page_size, (float*)k_pages, (float*)v_pages, num_pages, nq, nkv, d, dv, norm_size, num_tokens, error_word);
+  else if (dtype == PYLON_DTYPE_BF16 && !bias && layout == 0 && rot % 16 == 0 && d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && ld % 8 == 0 &&
+           (uintptr_t)qkv % 16 == 0 && (uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0 && (uintptr_t)cos_table % 16 == 0 && (uintptr_t)sin_table % 16 == 0 &&
+           (uintptr_t)q_weight % 16 == 0 && (uintptr_t)k_weight % 16 == 0) {
+    int lanes = 1;
+    while (lanes * 8 < (d > dv ? d : dv)) lanes *= 2;
+    const unsigned vector_blocks = (unsigned)((items * lanes + ROTARY_THREADS - 1) / ROTARY_THREADS);
+    launch_dependent(qkv_rotate_write_vec_kernel, dim3(vector_blocks), dim3(ROTARY_THREADS), 0, stream, (__nv_bfloat16*)qkv, ld, cos_table, sin_table, rot,
+                     table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row, block_table, table_width, page_size, (__nv_bfloat16*)k_pages,
+                     (__nv_bfloat16*)v_pages, num_pages, nq, nkv, d, dv, norm_size, lanes, items, error_word);
+  } else if (dtype == PYLON_DTYPE_BF16)
     qkv_rotate_write_kernel<__nv_bfloat16><<<blocks, ROTARY_THREADS, smem, stream>>>(
         (__nv_bfloat16*)qkv, ld, bias, cos_table, sin_table, rot, layout, table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row,
-        block_table, table_width, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages, nq, nkv, d, dv, num_tokens, error_word);
+        block_table, table_width, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages, nq, nkv, d, dv, norm_size, num_tokens, error_word);
   else
     PYLON_REFUSE("qkv_rotate_write: unknown dtype %d", dtype);
   PYLON_CHECK_LAUNCH("qkv_rotate_write");

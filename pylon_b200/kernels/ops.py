@@ -204,6 +204,12 @@ _SIGNATURES = {
                                          c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                          c_int, c_void_p, c_int, c_void_p],
     },
+    "min_gru.cu": {
+        "pylon_min_gru": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_int, c_int, c_void_p],
+    },
+    "output_norm.cu": {
+        "pylon_output_norm": [c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
+    },
     "matrix_memory.cu": {
         "pylon_matrix_memory_scan": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -220,10 +226,10 @@ _SIGNATURES = {
     "experts.cu": {
         "pylon_experts_row_tile": [],
         "pylon_experts_route": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
-                                c_float, c_int, c_void_p, c_void_p],
-        "pylon_experts_plan": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                                c_float, c_int, c_int, c_void_p, c_void_p],
+        "pylon_experts_plan": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
         "pylon_experts_product": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_int, c_void_p],
+                                  c_int, c_void_p, c_float, c_float, c_void_p],
         "pylon_experts_sort_rows": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "pylon_experts_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p],
     },
@@ -244,7 +250,7 @@ _SIGNATURES = {
     },
     "rotary.cu": {
         "pylon_qkv_rotate_write": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
-                                   c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+                                   c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "pylon_latent_norm_rotate_write": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int,
                                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "pylon_rotate_heads": [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
@@ -265,7 +271,7 @@ _SIGNATURES = {
         "pylon_gemm_tcgen05_glu_clamped": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_float, c_float,
                                            c_void_p, c_int, c_void_p],
         "pylon_gemm_tcgen05_force_tile": [c_int],
-        "pylon_gemm_tcgen05_grouped": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int, c_void_p, c_int,
+        "pylon_gemm_tcgen05_grouped": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_int, c_float, c_float, c_void_p, c_void_p, c_int,
                                        c_void_p, c_int, c_void_p],
         "pylon_gemm_tcgen05_qkv_rotate": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_longlong, c_longlong, c_longlong, c_void_p, c_void_p, c_float,
                                           c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
@@ -274,7 +280,8 @@ _SIGNATURES = {
     "attention_simple.cu": {
         "pylon_paged_attention_simple": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
-                                         c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_void_p],
+                                         c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_longlong, c_float,
+                                         c_longlong, c_void_p],
     },
     "attention_window.cu": {
         "pylon_window_attention": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
@@ -418,6 +425,39 @@ def add_rmsnorm(
     _check(library, library.pylon_add_rmsnorm(_ptr(residual), _ptr(delta), _ptr(weight), _ptr(rows), _ptr(out), n_rows, width,
                                               float(eps), 0 if rows is not None else 1, _dtype_code(out_dtype), _stream()))
     return out
+
+
+def output_norm(residual: torch.Tensor, output: torch.Tensor, weight: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """``residual += rmsnorm(output) * weight`` in float32, in place, for a norm that stands on a sublayer's output: ``[T, width]`` in ``dtype``
+    or float32 partial sums ``[parts, T, width]`` whose sum it is.  Returns the new sum in ``dtype`` (``residual`` itself in float32)."""
+    _need_cuda(residual, output, weight)
+    _need(residual.dtype == torch.float32 and residual.dim() == 2 and residual.is_contiguous(), "output_norm: residual must be contiguous float32 [T, width]")
+    tokens, width = residual.shape
+    parts = output.shape[0] if output.dim() == 3 else 0
+    _need(output.shape[-2:] == residual.shape and output.is_contiguous() and output.dtype == (torch.float32 if parts else dtype),
+          "output_norm: output must be contiguous [T, width] in the compute dtype or float32 [parts, T, width]")
+    _need(weight.dtype == torch.float32 and weight.shape == (width,) and weight.is_contiguous(), "output_norm: weight must be float32 [width]")
+    copy = None if dtype == torch.float32 else torch.empty((tokens, width), dtype=dtype, device=residual.device)
+    library = _library("output_norm.cu")
+    _check(library, library.pylon_output_norm(_ptr(output), parts, None, 0, 1.0, _ptr(residual), _ptr(copy), _ptr(weight), tokens, width, float(eps), 1,
+                                              _dtype_code(dtype), _stream()))
+    return residual if copy is None else copy
+
+
+def embedding_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float, dtype: torch.dtype, scale: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """``rmsnorm(table[ids] * scale) * weight``: the stream a model starts with whose embedding is normed, float32 ``[T, width]``, and the same in
+    ``dtype`` (``table``'s dtype; in float32 one tensor serves as both)."""
+    _need_cuda(ids, table, weight)
+    _need(ids.dtype == torch.int32 and ids.dim() == 1 and ids.is_contiguous(), "embedding_norm: ids must be contiguous int32 [T]")
+    _need(table.dim() == 2 and table.is_contiguous() and table.dtype == dtype, "embedding_norm: table must be contiguous [vocab, width] in the compute dtype")
+    tokens, (vocab, width) = ids.shape[0], table.shape
+    _need(weight.dtype == torch.float32 and weight.shape == (width,) and weight.is_contiguous(), "embedding_norm: weight must be float32 [width]")
+    residual = torch.empty((tokens, width), dtype=torch.float32, device=table.device)
+    copy = None if dtype == torch.float32 else torch.empty((tokens, width), dtype=dtype, device=table.device)
+    library = _library("output_norm.cu")
+    _check(library, library.pylon_output_norm(_ptr(table), 0, _ptr(ids), vocab, float(scale), _ptr(residual), _ptr(copy), _ptr(weight), tokens, width, float(eps), 0,
+                                              _dtype_code(dtype), _stream()))
+    return residual, residual if copy is None else copy
 
 
 def residual_add(residual: torch.Tensor, delta: torch.Tensor) -> None:
@@ -870,11 +910,21 @@ def paged_attention(
     keep_first: int = 0,
     distance_bias: Optional[torch.Tensor] = None,
     split_weights: bool = False,
+    weighting: str = "softmax",
+    score_bias: Optional[torch.Tensor] = None,
+    head_gate: Optional[torch.Tensor] = None,
+    out_factor: float = 1.0,
 ) -> torch.Tensor:
     """Causal attention of every token of a step over its request's pages.
 
     ``split_weights`` (latent rows on the tensor cores): a softmax weight enters the weighted sum as two bfloat16 numbers, the rounded
     weight and what the rounding dropped, so that it counts with 16 bits instead of 8, at twice the products over the values.
+
+    ``weighting="sigmoid"``: the weight of a visible key is ``sigmoid(score + score_bias[h])`` (float32 ``[nq]``, or None) and nothing is
+    divided by a sum over the keys.  Then ``head_gate`` (``[T, nq]`` in the cache dtype, any row stride) multiplies head h of token t by
+    ``sigmoid(head_gate[t, h])``, ``out_factor`` multiplies everything, and ``out`` may be a slice of wider rows.  On the tensor cores
+    (values as wide as the keys, a multiple of 16 up to 256) the same kernels run as for the softmax, built for sigmoid weights; a
+    weight enters the weighted sum as two bfloat16 numbers, the rounded weight and what the rounding dropped.
 
     ``keep_first`` n: a window never hides the keys at positions below n (a token sees ``j <= p`` with ``p - j < window`` or
     ``j < n``).  ``distance_bias``: float32 ``[rows, nq]``; the scaled score of the key ``p - j`` positions back gets
@@ -943,10 +993,17 @@ def paged_attention(
     _need(kv_len.dtype == torch.int32 and kv_len.is_contiguous() and kv_len.shape[0] >= rows, "paged_attention: kv_len must be int32 [rows]")
     if out is None:
         out = torch.empty((tokens, nq * dv), dtype=q.dtype, device=q.device)
-    _need(out.shape == (tokens, nq * dv) and out.dtype == q.dtype and out.is_contiguous(), "paged_attention: out has the wrong shape or dtype")
+    sigmoid = weighting == "sigmoid"
+    _need(weighting in ("softmax", "sigmoid"), f"paged_attention: unknown weighting {weighting!r}")
+    _need(out.shape == (tokens, nq * dv) and out.dtype == q.dtype and out.stride(1) == 1 and (sigmoid or out.is_contiguous()), "paged_attention: out has the wrong shape or dtype")
+    _need(sigmoid or (score_bias is None and head_gate is None and out_factor == 1.0), "paged_attention: a number per head on the scores, gated heads and a factor go with sigmoid weights")
+    _need(not sigmoid or (sinks is None and not plain_only), "paged_attention: no sink, kept first keys and bias by distance with sigmoid weights")
+    _need_cuda(score_bias, head_gate)
+    _need(score_bias is None or (score_bias.dtype == torch.float32 and score_bias.shape == (nq,) and score_bias.is_contiguous()), "paged_attention: score_bias must be float32 [nq]")
+    _need(head_gate is None or (head_gate.dtype == q.dtype and head_gate.shape == (tokens, nq) and head_gate.stride(1) == 1), "paged_attention: head_gate must be [T, nq] in the cache dtype")
     scale = 1.0 / math.sqrt(d) if scale is None else float(scale)
-    _need(scale > 0, "paged_attention: the softmax scale must be positive")
-    if q.dtype == torch.bfloat16 and d % 16 == 0 and d <= 256 and not force_simple and same_width and sinks is None and not plain_only:
+    _need(scale > 0 or sigmoid, "paged_attention: the softmax scale must be positive")
+    if q.dtype == torch.bfloat16 and d % 16 == 0 and d <= 256 and not force_simple and same_width and sinks is None and not plain_only and not sigmoid:
         library = _library("attention_mma.cu", {"PYLON_HEAD_DIM": d})
         group = nq // nkv
         any_large = max_q * group > 16
@@ -1010,7 +1067,8 @@ def paged_attention(
     _check(library, library.pylon_paged_attention_simple(
         _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(positions), _ptr(token_row), _ptr(block_table),
         block_table.shape[1], page_size, num_pages, nq, nkv, d, dv, int(window or 0), int(chunk or 0), float(softcap or 0.0), scale,
-        _ptr(sinks), 0, 0, tokens, _dtype_code(q.dtype), int(keep_first), _ptr(distance_bias), 0 if distance_bias is None else distance_bias.shape[0], _stream()))
+        _ptr(sinks), 0, 0, tokens, _dtype_code(q.dtype), int(keep_first), _ptr(distance_bias), 0 if distance_bias is None else distance_bias.shape[0],
+        int(sigmoid), _ptr(score_bias), _ptr(head_gate), 0 if head_gate is None else head_gate.stride(0), float(out_factor), out.stride(0), _stream()))
     return out
 
 
@@ -1073,7 +1131,7 @@ def _latent_attention(q, pages, dv, positions, token_row, q_start, kv_len, block
     _check(library, library.pylon_paged_attention_simple(
         _ptr(q), q.stride(0), _ptr(pages), _ptr(pages), _ptr(out), _ptr(positions), _ptr(token_row), _ptr(block_table),
         block_table.shape[1], page_size, num_pages, nq, 1, d, dv, int(window or 0), 0, 0.0, float(scale),
-        _ptr(sinks), d, d, tokens, _dtype_code(q.dtype), 0, None, 0, _stream()))
+        _ptr(sinks), d, d, tokens, _dtype_code(q.dtype), 0, None, 0, 0, None, None, 0, 1.0, 0, _stream()))
     return out
 
 
@@ -1395,6 +1453,27 @@ def linear_recurrence(proj: torch.Tensor, bias: torch.Tensor, conv_weight: torch
     return out
 
 
+def min_gru(proj: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, num_rows: int, max_q: int,
+            out: torch.Tensor, factor: float = 1.0) -> torch.Tensor:
+    """A minimal gated recurrence per channel over the tokens of a step (``csrc/min_gru.cu`` has the equations).
+
+    ``proj [T, 3 C]``: the projection of the layer's input, columns ``[z | x | g]``, and ``bias`` float32 ``[2, C]`` (z, x); ``state`` float32
+    ``[slots, C]``, read at ``state[slots[row]]`` and advanced in place by the row's tokens; ``max_q``: the most tokens a row brings (an upper
+    bound is fine).  ``out [T, C]`` in ``proj``'s dtype receives ``factor`` times state times ``silu(g)``, ready for the output projection.
+    ``proj`` and ``out`` may be slices of wider rows."""
+    _need_cuda(proj, bias, state, q_start, slots, out)
+    tokens, channels = proj.shape[0], proj.shape[1] // 3
+    _need(proj.dim() == 2 and proj.stride(1) == 1 and proj.shape[1] == 3 * channels, "min_gru: proj must be [T, 3 C]")
+    _need(bias.dtype == torch.float32 and bias.shape == (2, channels) and bias.is_contiguous(), "min_gru: bias must be float32 [2, C]")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.is_contiguous() and state.shape[1] == channels, "min_gru: state must be contiguous float32 [slots, C]")
+    _need(out.shape == (tokens, channels) and out.dtype == proj.dtype and out.stride(1) == 1, "min_gru: out must be [T, C] in proj's dtype")
+    _rows_meta("min_gru", tokens, num_rows, q_start=q_start, slots=slots)
+    library = _library("min_gru.cu")
+    _check(library, library.pylon_min_gru(_ptr(proj), proj.stride(0), _ptr(bias), _ptr(state), _ptr(q_start), _ptr(slots), _ptr(out), out.stride(0), channels,
+                                          float(factor), num_rows, min(tokens, int(max_q)), _dtype_code(proj.dtype), _stream()))
+    return out
+
+
 def matrix_memory(proj: torch.Tensor, gate_logits: torch.Tensor, gate_bias: torch.Tensor, norm_weight: torch.Tensor, state: torch.Tensor,
                   q_start: torch.Tensor, slots: torch.Tensor, heads: int, dim: int, vdim: int, cap: float, norm_eps: float, read_eps: float,
                   num_rows: int) -> torch.Tensor:
@@ -1536,7 +1615,8 @@ EXPERT_TILE_ROWS = 128   # the row tile of the grouped tcgen05 product
 def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[torch.Tensor], w_gate_up: torch.Tensor, w_down: torch.Tensor,
                    top: int, activation: str = "silu", interleaved: bool = False, gated: bool = True, routing: str = "softmax",
                    correction: Optional[torch.Tensor] = None, groups: int = 0, groups_keep: int = 0, share_eps: float = 0.0,
-                   common_up: Optional[torch.Tensor] = None, common_down: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   common_up: Optional[torch.Tensor] = None, common_down: Optional[torch.Tensor] = None, share_normalized: bool = True,
+                   weigh: str = "output", limit: Optional[float] = None, alpha: float = 1.702) -> torch.Tensor:
     """``sum over a token's top experts e of share_e * W_down,e (act(W_gate,e h) * (W_up,e h))`` (``csrc/experts.cu``).
 
     ``h [T, width]``; ``router`` float32 ``[experts, width]`` and ``router_bias`` float32 ``[experts]`` (or None): the logits are
@@ -1551,13 +1631,20 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     an ungated expert that every token goes through, added times ``sigmoid(w h)`` with ``w`` the row that ``router`` then holds behind
     the experts' rows (``[experts + 1, width]``).
 
+    ``share_normalized=False``: the shares are the chosen experts' scores as they are.  ``weigh="input"`` (gated experts): the result is
+    ``sum expert_e(share_e * h)``; an expert's first product is linear in its input, so the share multiplies its float32 sums.
+    ``activation="clamped"`` with a ``limit``: the clamped gated unit of :func:`swiglu`.
+
     The tokens are sorted by expert on the device.  A step of few tokens runs the experts' products from row tiles of 32 slots that
     gather their rows themselves (``mma.sync``, bound by the matrices coming from memory); a bfloat16 step with about half a
     128-row tile or more per expert (gated: interleaved weights and ``silu``) copies the rows into their sorted order and runs both
     products on the grouped form of the tcgen05 kernel (the gated unit in the first one's epilogue; an ungated expert's activation
     is a pass of its own between the two)."""
     _need_cuda(h, router, router_bias, w_gate_up, w_down, correction, common_up, common_down)
-    _need(activation in ACTIVATIONS, f"expert_mixture: activation {activation!r}")
+    clamped = activation == "clamped"
+    _need(activation in ACTIVATIONS or clamped, f"expert_mixture: activation {activation!r}")
+    _need(clamped == (limit is not None) and (not clamped or (gated and limit > 0)), "expert_mixture: a clamped unit is gated and has a positive limit")
+    _need(weigh in ("output", "input") and (weigh == "output" or gated), "expert_mixture: shares weigh a gated expert's output or its input")
     _need(routing in ("softmax", "sigmoid"), f"expert_mixture: routing {routing!r}")
     _need(h.dim() == 2 and h.stride(1) == 1, "expert_mixture: h must be [T, width]")
     tokens, width = h.shape
@@ -1567,6 +1654,7 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
           and w_gate_up.dtype == h.dtype and w_down.dtype == h.dtype, "expert_mixture: w_gate_up [experts, 2 F, width] (ungated: [experts, F, width]) and w_down [experts, width, F] in h's dtype")
     scored = routing == "sigmoid"
     extra = 1 if common_up is not None else 0
+    _need(scored or share_normalized, "expert_mixture: shares that do not add up to one go with sigmoid routing")
     _need(scored or (correction is None and not groups and not extra), "expert_mixture: a correction, groups and a common expert go with sigmoid routing")
     _need(router.dtype == torch.float32 and router.shape == (experts + extra, width) and router.is_contiguous(), "expert_mixture: router must be float32 [experts (+ 1), width]")
     _need(router_bias is None or (router_bias.dtype == torch.float32 and router_bias.shape == (experts,)), "expert_mixture: router_bias must be float32 [experts]")
@@ -1576,7 +1664,7 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     _need((common_up is None) == (common_down is None), "expert_mixture: a common expert has both its matrices")
     library = _library("experts.cu")
     pairs = tokens * top
-    grouped = ((not gated or (interleaved and activation == "silu")) and h.dtype == torch.bfloat16 and pairs * 2 >= EXPERT_TILE_ROWS * experts and width % 8 == 0
+    grouped = ((not gated or (interleaved and activation in ("silu", "clamped"))) and h.dtype == torch.bfloat16 and pairs * 2 >= EXPERT_TILE_ROWS * experts and width % 8 == 0
                and inner % 8 == 0 and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0)
     tile = EXPERT_TILE_ROWS if grouped else library.pylon_experts_row_tile()
     max_tiles = min(pairs, experts) + pairs // tile    # every expert with tokens ends in at most one partly filled tile
@@ -1588,11 +1676,14 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     source = torch.empty((max_slots,), dtype=torch.int32, device=device)
     tile_expert = torch.empty((max_tiles,), dtype=torch.int32, device=device)
     common_gate = torch.empty((tokens,), dtype=torch.float32, device=device) if extra else None
-    code, kind = _dtype_code(h.dtype), ACTIVATIONS[activation]
+    code, kind = _dtype_code(h.dtype), 4 if clamped else ACTIVATIONS[activation]
+    slot_share = torch.empty((max_slots,), dtype=torch.float32, device=device) if weigh == "input" else None
+    limit, out_share = float(limit or 0.0), share if slot_share is None else None
     _check(library, library.pylon_experts_route(_ptr(h), h.stride(0), _ptr(router), _ptr(router_bias), _ptr(chosen), _ptr(share), width, experts, top,
-                                                tokens, code, int(scored), _ptr(correction), int(groups or 0), int(groups_keep or 0), float(share_eps), extra,
+                                                tokens, code, int(scored), _ptr(correction), int(groups or 0), int(groups_keep or 0), float(share_eps), int(bool(share_normalized)), extra,
                                                 _ptr(common_gate), _stream()))
-    _check(library, library.pylon_experts_plan(_ptr(chosen), _ptr(slot_of), _ptr(source), _ptr(tile_expert), pairs, experts, max_slots, max_tiles, tile, _stream()))
+    _check(library, library.pylon_experts_plan(_ptr(chosen), _ptr(slot_of), _ptr(source), _ptr(tile_expert), pairs, experts, max_slots, max_tiles, tile,
+                                               _ptr(share), _ptr(slot_share), _stream()))
     common, common_code = None, F32
     if extra:   # the expert of every token: two plain products around the activation
         common = linear(activation_in_place(linear(h, common_up), activation), common_down)
@@ -1605,22 +1696,22 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
         _check(library, library.pylon_experts_sort_rows(_ptr(h), h.stride(0), _ptr(source), _ptr(rows), width, top, max_slots, code, _stream()))
         act = torch.empty((max_slots, inner), dtype=h.dtype, device=device)
         _check(product, product.pylon_gemm_tcgen05_grouped(_ptr(rows), _ptr(w_gate_up), _ptr(act), max_slots, halves * inner, width, width, width, inner,
-                                                           1 if gated else 0, _ptr(tile_expert), experts, error, sms, _stream()))
+                                                           1 if gated else 0, limit, float(alpha), _ptr(slot_share), _ptr(tile_expert), experts, error, sms, _stream()))
         if not gated:
             activation_in_place(act, activation)   # (rows of empty slots hold act(0) of zeros: they are never gathered)
         y = torch.empty((max_slots, width), dtype=h.dtype, device=device)
-        _check(product, product.pylon_gemm_tcgen05_grouped(_ptr(act), _ptr(w_down), _ptr(y), max_slots, width, inner, inner, inner, width, 0,
+        _check(product, product.pylon_gemm_tcgen05_grouped(_ptr(act), _ptr(w_down), _ptr(y), max_slots, width, inner, inner, inner, width, 0, 0.0, 1.0, None,
                                                            _ptr(tile_expert), experts, error, sms, _stream()))
-        _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(share), _ptr(out), tokens, width, top, code, _ptr(common), _ptr(common_gate),
+        _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, top, code, _ptr(common), _ptr(common_gate),
                                                      common_code, _stream()))
         return out
     act = torch.empty((max_slots, inner), dtype=h.dtype, device=device)
     _check(library, library.pylon_experts_product(_ptr(h), h.stride(0), _ptr(w_gate_up), _ptr(source), _ptr(tile_expert), 1, top, _ptr(act), inner, width,
-                                                  max_tiles, 1 if gated else 2, kind, int(interleaved), code, _stream()))
+                                                  max_tiles, 1 if gated else 2, kind, int(interleaved), code, _ptr(slot_share), limit, float(alpha), _stream()))
     y = torch.empty((max_slots, width), dtype=torch.float32, device=device)
     _check(library, library.pylon_experts_product(_ptr(act), inner, _ptr(w_down), _ptr(source), _ptr(tile_expert), 0, 1, _ptr(y), width, inner,
-                                                  max_tiles, 0, kind, 0, code, _stream()))
-    _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(share), _ptr(out), tokens, width, top, _dtype_code(torch.float32), _ptr(common),
+                                                  max_tiles, 0, kind, 0, code, None, 0.0, 1.0, _stream()))
+    _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, top, _dtype_code(torch.float32), _ptr(common),
                                                  _ptr(common_gate), common_code, _stream()))
     return out
 
@@ -1678,9 +1769,10 @@ def qkv_rotate_write(
     qkv: torch.Tensor, bias: Optional[torch.Tensor], cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rotary_dim: int, layout: str,
     norm: Optional[str], q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
     token_row: torch.Tensor, block_table: torch.Tensor, page_size: int, k_pages: torch.Tensor, v_pages: torch.Tensor, nq: int, nkv: int,
-    head_dim: int, value_dim: int,
+    head_dim: int, value_dim: int, norm_size: Optional[int] = None,
 ) -> torch.Tensor:
-    """On ``qkv [T, nq * d + nkv * d + nkv * dv]``: add ``bias`` (float32, one number per column), rotate the first
+    """``norm_size``: how many elements of a q or k head are its own (default: all ``d``; the rest are zeros, and the mean of the norm's
+    squares is over its own).  On ``qkv [T, nq * d + nkv * d + nkv * dv]``: add ``bias`` (float32, one number per column), rotate the first
     ``rotary_dim`` elements of every q and k head by the tables (``layout``: ``"halves"`` pairs element i with i + rotary_dim / 2,
     ``"neighbours"`` element 2 i with 2 i + 1), divide every q and k head by its root mean square (``norm``: ``"before"`` or
     ``"after"`` the rotation, ``None``: not at all; times ``q_weight`` / ``k_weight [d]`` where given), write q back in place and
@@ -1703,8 +1795,8 @@ def qkv_rotate_write(
     _check(library, library.pylon_qkv_rotate_write(
         _ptr(qkv), qkv.stride(0), _ptr(bias), _ptr(cos), _ptr(sin), rotary_dim if cos is not None else 0, ROTARY_LAYOUTS[layout], table_positions,
         {None: 0, "before": 1, "after": 2}[norm], _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(positions), _ptr(token_row), _ptr(block_table),
-        block_table.shape[1], page_size, _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], nq, nkv, head_dim, value_dim, tokens, _dtype_code(qkv.dtype),
-        _ptr(cache_write_error_word(k_pages.device)), _stream()))
+        block_table.shape[1], page_size, _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], nq, nkv, head_dim, value_dim,
+        head_dim if norm_size is None else int(norm_size), tokens, _dtype_code(qkv.dtype), _ptr(cache_write_error_word(k_pages.device)), _stream()))
     return qkv
 
 

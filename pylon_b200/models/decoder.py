@@ -25,6 +25,7 @@ class DecoderModel:
         self.spec = spec
         self.blocks = [BLOCKS.build(layer.block) for layer in spec.layers]
         self.final_norm = NORMS.build(spec.final_norm)
+        self.embedding_norm = None if spec.embedding_norm is None else NORMS.build(spec.embedding_norm)
         self.embedding: Optional[torch.Tensor] = None
         self.lm_head: Optional[torch.Tensor] = None
         self.position_table: Optional[torch.Tensor] = None   # learnt vectors per position, added to the embedding rows
@@ -46,6 +47,10 @@ class DecoderModel:
         for decl in self.final_norm.tensors():
             name = spec.final_norm_prefix + decl.name
             decls[name] = TensorDecl(name, decl.shape, decl.role, decl.init)
+        if self.embedding_norm is not None:
+            for decl in self.embedding_norm.tensors():
+                name = spec.embedding_norm_prefix + decl.name
+                decls[name] = TensorDecl(name, decl.shape, decl.role, decl.init)
         for layer, block in zip(spec.layers, self.blocks):
             for decl in block.tensors():
                 name = layer.prefix + decl.name
@@ -74,6 +79,10 @@ class DecoderModel:
         self.final_norm.load(
             {decl.name: place(decls[spec.final_norm_prefix + decl.name]) for decl in self.final_norm.tensors()}, dtype, self.device
         )
+        if self.embedding_norm is not None:
+            self.embedding_norm.load(
+                {decl.name: place(decls[spec.embedding_norm_prefix + decl.name]) for decl in self.embedding_norm.tensors()}, dtype, self.device
+            )
         for layer, block in zip(spec.layers, self.blocks):
             block.load({decl.name: place(decls[layer.prefix + decl.name]) for decl in block.tensors()}, dtype, self.device)
 
@@ -107,11 +116,14 @@ class DecoderModel:
         ``taps``: a list that receives the residual stream after every run, float32 ``[T, width]``
         (the sum of the copies where the model keeps several) - for looking at a model layer by layer."""
         step.carry = {}
-        residual = ops.embed_gather(step.token_ids, self.embedding, scale=self.spec.embedding_scale, copies=self.spec.streams)
+        if self.embedding_norm is not None:   # the normed rows are the stream: one kernel, which leaves it in the compute dtype as well
+            stream = self.embedding_norm.enter(step.token_ids, self.embedding, self.spec.embedding_scale)
+        else:
+            stream = ResidualStream(ops.embed_gather(step.token_ids, self.embedding, scale=self.spec.embedding_scale, copies=self.spec.streams))
+        residual = stream.residual
         if self.position_table is not None:   # the learnt vector of each token's position joins its embedding row, in 32-bit like the sum
             ops.embed_gather(step.positions, self.position_table, out=residual, copies=self.spec.streams, accumulate=True)
         entered = residual.clone() if self.reentry is not None else None   # the embedding output, for the runs that re-enter
-        stream = ResidualStream(residual)
         for position, run in enumerate(self.spec.order):
             if run.reenter:
                 # x <- W [x; x0]: what is pending joins the sum, both halves are laid side by side in the compute dtype, and the

@@ -25,6 +25,13 @@ the per-head norm of q and k behind the rotation instead of before it (``qk_norm
 (``qk_norm_weight=False``), an encoding that rotates only part of a head or pairs neighbouring elements, and any of these
 together with values of their own width, chunks or a soft cap: one kernel for bias, rotation, norm and cache write
 (``ops.qkv_rotate_write``) then stands between the product and the attention.
+
+``weighting="sigmoid"``: a visible key's weight is ``sigmoid(score + b_h)``, not a softmax: nothing is divided by a sum over the keys
+(``score_bias``: b, a learnt number per head; without it zero).  It goes with every option of the paragraph above and with windows, chunks
+and a soft cap.  ``head_gate``: head h's output is multiplied by ``sigmoid((W_g x)_h)``, ``W_g [heads, width]`` reading the mixer's input; its
+rows ride in the projections' product and the attention kernels multiply as they write.  In bfloat16 such a mixer keeps keys and
+values at one width, the larger of the two rounded up to a multiple of 16 (zero rows and columns of the weights fill it), so that
+every size up to 256 has the tensor-core kernels.
 """
 from __future__ import annotations
 
@@ -78,6 +85,9 @@ class GroupedQueryAttention(Mixer):
         keep_first: int = 0,
         distance_bias: Optional[Mapping[str, float]] = None,
         sink: bool = False,
+        weighting: str = "softmax",
+        score_bias: bool = False,
+        head_gate: bool = False,
     ) -> None:
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads cannot be grouped over {n_kv_heads} KV heads")
@@ -106,6 +116,14 @@ class GroupedQueryAttention(Mixer):
             raise ValueError(f"the q/k norm stands 'before' or 'after' the rotation or runs over the 'whole' rows, not {qk_norm!r}")
         if plain_scores and (position is not None or value_mix is not None or bias):
             raise NotImplementedError("whole-row norms, kept first positions, a bias by distance and a sink: without rotation, value mixing and projection biases")
+        if weighting not in ("softmax", "sigmoid"):
+            raise ValueError(f"the weights of the keys are a 'softmax' or each a 'sigmoid', not {weighting!r}")
+        self.weighting, self.has_score_bias, self.has_head_gate = weighting, bool(score_bias), bool(head_gate)
+        self.splits_products = weighting == "sigmoid"
+        if weighting == "sigmoid" and (plain_scores or value_mix is not None or bias):
+            raise NotImplementedError("sigmoid weights: without whole-row norms, kept first positions, a bias by distance, a sink, value mixing and projection biases")
+        if weighting != "sigmoid" and (score_bias or head_gate):
+            raise NotImplementedError("a number per head added to the scores and a gate per head go with sigmoid weights")
         self.bias, self.bias_suffix, self.qk_norm_place, self.qk_norm_weight = bool(bias), bias_suffix, qk_norm, bool(qk_norm_weight)
         self.window = None if window is None else int(window)
         self.scale = 1.0 / math.sqrt(self.head_dim) if scale is None else float(scale)
@@ -113,13 +131,17 @@ class GroupedQueryAttention(Mixer):
         self.names = {
             "q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "value_mix": "vmix", "distance_bias": "distance_bias", "sink": "sink",
+            "score_bias": "score_bias", "head_gate": "g_proj.weight",
             **(names or {}),
         }
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.mix_weight = self.b_qkv = self.bias_table = self.sink = None
+        self.score_bias = None
+        self.kept_head_dim = self.head_dim     # the width keys have in the cache, and queries in the product: wider than head_dim when they are kept padded
         self.kept_value_dim = self.value_dim   # the width values have in the cache: wider than value_dim when they are kept padded
         # what the kernels that fuse norm, rotation and cache write do not take goes through the kernel that takes everything
         self.rotary_general = self.bias or self.qk_norm_place == "after" or (self.qk_norm_eps is not None and not self.qk_norm_weight) \
             or (self.position is not None and (self.general or getattr(self.position, "layout", "halves") != "halves"))
+        self.rotary_general = self.rotary_general or weighting == "sigmoid"
         if self.rotary_general and (value_mix is not None or (self.position is not None and not hasattr(self.position, "tables"))):
             raise NotImplementedError("biases, a norm behind the rotation or a rotation beside values of their own width: not with value mixing, and "
                                       "only with an encoding that rotates by tables of cos and sin")
@@ -142,6 +164,10 @@ class GroupedQueryAttention(Mixer):
             decls.append(TensorDecl(n["distance_bias"], (self.bias_rows, self.n_heads), "vector", (0.0, 0.5)))
         if self.has_sink:
             decls.append(TensorDecl(n["sink"], (self.n_heads,), "vector", (0.0, 1.0)))
+        if self.has_score_bias:
+            decls.append(TensorDecl(n["score_bias"], (self.n_heads,), "vector", (-7.0, 0.5)))   # about minus the logarithm of a context's length
+        if self.has_head_gate:
+            decls.append(TensorDecl(n["head_gate"], (self.n_heads, self.width)))
         if self.bias:
             decls += [TensorDecl(n[key] + self.bias_suffix, (size,), "vector", (0.0, 0.02))
                       for key, size in (("q", self.q_size), ("k", self.kv_size), ("v", self.v_size))]
@@ -149,6 +175,9 @@ class GroupedQueryAttention(Mixer):
 
     def load(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> None:
         n = self.names
+        if self.weighting == "sigmoid":
+            self._load_sigmoid(tensors, dtype)
+            return
         w_v, w_o = tensors[n["v"]], tensors[n["o"]]
         b_v = tensors[n["v"] + self.bias_suffix] if self.bias else None
         # The tensor-core attention kernels take values as wide as the keys.  Narrower values are kept padded to the keys'
@@ -182,16 +211,48 @@ class GroupedQueryAttention(Mixer):
         if self.has_sink:
             self.sink = tensors[n["sink"]].contiguous()
 
+    def _load_sigmoid(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype) -> None:
+        n = self.names
+        if dtype == torch.bfloat16 and max(self.head_dim, self.value_dim) <= 256:
+            self.kept_head_dim = self.kept_value_dim = -(-max(self.head_dim, self.value_dim) // 16) * 16
+
+        def wider(weight: torch.Tensor, heads: int, width: int, kept: int) -> torch.Tensor:   # [heads * width, columns] -> [heads * kept, columns]
+            if kept == width:
+                return weight
+            padded = weight.new_zeros((heads, kept, weight.shape[1]))
+            padded[:, :width] = weight.view(heads, width, -1)
+            return padded.view(heads * kept, -1)
+
+        rows = [wider(tensors[n["q"]], self.n_heads, self.head_dim, self.kept_head_dim), wider(tensors[n["k"]], self.n_kv_heads, self.head_dim, self.kept_head_dim),
+                wider(tensors[n["v"]], self.n_kv_heads, self.value_dim, self.kept_value_dim)]
+        if self.has_head_gate:
+            rows.append(tensors[n["head_gate"]])
+        filled = sum(part.shape[0] for part in rows)
+        if filled % 8:   # the gate's rows fill up whole 16-byte pieces of the product's rows
+            rows.append(rows[0].new_zeros((-filled % 8, self.width)))
+        self.input_rows = torch.cat(rows, dim=0).contiguous()
+        self.output_columns = wider(tensors[n["o"]].t(), self.n_heads, self.value_dim, self.kept_value_dim).t().contiguous()
+        if self.qk_norm_eps is not None and self.qk_norm_weight:
+            fill = self.kept_head_dim - self.head_dim
+            self.q_norm, self.k_norm = (torch.nn.functional.pad(tensors[n[key]], (0, fill)).contiguous() for key in ("q_norm", "k_norm"))
+        self.score_bias = tensors[n["score_bias"]].contiguous() if self.has_score_bias else None
+
     def weight_bytes(self) -> int:
+        if self.weighting == "sigmoid":
+            return (self.input_rows.numel() + self.output_columns.numel()) * self.input_rows.element_size() + (0 if self.q_norm is None else 8 * self.head_dim)
         return (self.w_qkv.numel() + self.w_o.numel()) * self.w_qkv.element_size() + (0 if self.q_norm is None else 8 * self.head_dim)
 
     # -- cache ---------------------------------------------------------------------------
     def cache_need(self) -> CacheNeed:
-        value_dim = None if self.kept_value_dim == self.head_dim else self.kept_value_dim   # as kept: known once the weights are loaded
-        return CacheNeed(kv=KVNeed(self.n_kv_heads, self.head_dim, self.window, value_dim, self.chunk, self.keep_first))
+        value_dim = None if self.kept_value_dim == self.kept_head_dim else self.kept_value_dim   # as kept: known once the weights are loaded
+        return CacheNeed(kv=KVNeed(self.n_kv_heads, self.kept_head_dim, self.window, value_dim, self.chunk, self.keep_first))
 
     # -- run -----------------------------------------------------------------------------
     def forward(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> torch.Tensor:
+        if self.weighting == "sigmoid":
+            context = torch.empty((h.shape[0], self.output_columns.shape[1]), dtype=h.dtype, device=h.device)
+            self.middle(ops.linear(h, self.input_rows), step, cache, context, 1.0)
+            return ops.linear_for_residual(context, self.output_columns)
         if self.rotary_general:
             return self._forward_rotary_general(h, step, cache)
         if self.general:
@@ -269,3 +330,21 @@ class GroupedQueryAttention(Mixer):
             rows_alike=step.rows_alike, chunk=self.chunk, softcap=self.softcap,
         )
         return ops.linear_for_residual(context, self.w_o)
+
+    def middle(self, proj: torch.Tensor, step: StepView, cache: LayerCache, out: torch.Tensor, factor: float) -> None:
+        """Sigmoid weights: one kernel for norms, rotation and cache write on the projections, then the attention, which gates its heads
+        and multiplies them by ``factor`` as it writes them."""
+        cos, sin, rotary_dim, layout = self.position.tables(proj.device) if self.position is not None else (None, None, 0, "halves")
+        columns = (self.n_heads + self.n_kv_heads) * self.kept_head_dim + self.n_kv_heads * self.kept_value_dim
+        qkv = proj[:, :columns]
+        ops.qkv_rotate_write(
+            qkv, None, cos, sin, rotary_dim, layout, None if self.qk_norm_eps is None else self.qk_norm_place, self.q_norm, self.k_norm,
+            self.qk_norm_eps or 0.0, step.positions, step.token_row, cache.block_table, cache.page_size, cache.k_pages, cache.v_pages,
+            self.n_heads, self.n_kv_heads, self.kept_head_dim, self.kept_value_dim, norm_size=self.head_dim,
+        )
+        ops.paged_attention(
+            qkv, cache.k_pages, cache.v_pages, step.positions, step.token_row, step.q_start, step.kv_len, cache.block_table,
+            self.n_heads, step.max_q, step.max_kv, window=self.window, scale=self.scale, out=out, row_tokens=step.row_tokens,
+            rows_alike=step.rows_alike, chunk=self.chunk, softcap=self.softcap, weighting="sigmoid", score_bias=self.score_bias,
+            head_gate=proj[:, columns: columns + self.n_heads] if self.has_head_gate else None, out_factor=factor,
+        )

@@ -203,6 +203,15 @@ class Norm(Part):
         normalised (``None``: their plain sum)."""
         raise NotImplementedError
 
+    def join(self, stream: "ResidualStream", output: torch.Tensor) -> None:
+        """For a norm that stands on a sublayer's output: ``stream += norm(output)``.  ``output`` comes in either form of a
+        delta (see :class:`ResidualStream`)."""
+        raise NotImplementedError(f"{type(self).__name__} is not built to stand on a sublayer's output")
+
+    def enter(self, token_ids: torch.Tensor, table: torch.Tensor, scale: float) -> "ResidualStream":
+        """The stream that starts as the norm of the tokens' rows of ``table`` times ``scale``."""
+        raise NotImplementedError(f"{type(self).__name__} is not built to stand on the embedding")
+
 
 class PositionEncoding(Part):
     def rotary_table(self, device: torch.device) -> Optional[tuple[torch.Tensor, torch.Tensor, int]]:
@@ -222,6 +231,17 @@ class Mixer(Part):
     # row.  A mixer that indexes its cache or state by ``token_row`` has to look at this; so the default is False, and
     # a model with such a mixer is never padded.
     takes_padding = False
+    # True for a mixer that is one product of its input, a middle and one product of what the middle gives, and that runs the
+    # middle alone when asked: ``input_rows`` [n, width] and ``output_columns`` [width, k] are then its two matrices once it is
+    # loaded, and a container that holds several such mixers may stack the matrices and run each product once.
+    splits_products = False
+    input_rows: Optional[torch.Tensor] = None
+    output_columns: Optional[torch.Tensor] = None
+
+    def middle(self, proj: torch.Tensor, step: StepView, cache: "LayerCache", out: torch.Tensor, factor: float) -> None:
+        """From ``proj [T, n]`` (the input times ``input_rows``) to ``factor`` times what ``output_columns`` take, ``out [T, k]``; both
+        may be slices of wider rows that start at 16-byte addresses."""
+        raise NotImplementedError
 
     def cache_need(self) -> CacheNeed:
         return CacheNeed()
@@ -279,6 +299,7 @@ class ResidualStream:
         self.pending: Optional[torch.Tensor] = None
         self.pending_scale = 1.0
         self.pending_route: Optional[StreamRoute] = None
+        self.activation: Optional[torch.Tensor] = None   # the sum in the compute dtype, where the last kernel that wrote the sum left it
 
     @property
     def plain(self) -> bool:
@@ -289,6 +310,14 @@ class ResidualStream:
         if self.pending is not None:
             self.flush()
         self.pending, self.pending_scale, self.pending_route = delta, float(scale), route
+        self.activation = None
+
+    def read(self, dtype: torch.dtype) -> torch.Tensor:
+        """The sum as it is (nothing pending, no norm) in ``dtype``: what a sublayer reads whose norm stands on its output."""
+        self.flush()
+        if self.activation is None or self.activation.dtype != dtype:
+            self.activation = self.residual.to(dtype)
+        return self.activation
 
     def take_pending(self) -> tuple[Optional[torch.Tensor], float, Optional[StreamRoute]]:
         pending = (self.pending, self.pending_scale, self.pending_route)

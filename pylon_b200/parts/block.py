@@ -177,3 +177,41 @@ class ParallelSublayers(Block):
         stream.add(self.mixer.forward(h, step, cache))
         if self.feed_forward is not None:
             stream.add(self.feed_forward.forward(h, step))
+
+
+@BLOCKS.register("output_norm")
+class OutputNormBlock(Block):
+    """The norms stand on the sublayers' outputs only: ``x = x + norm1(mixer(x))``, then ``x = x + norm2(feed_forward(x))``; a sublayer
+    reads the sum itself in the compute dtype.  Norm, add and the next sublayer's copy of the sum are one kernel.
+    ``feed_forward=None`` leaves the second sublayer (and its norm) out."""
+
+    def __init__(self, mixer: PartSpec, feed_forward: Optional[PartSpec], mixer_norm: PartSpec, ffn_norm: Optional[PartSpec], mixer_prefix: str = "mix.",
+                 ffn_prefix: str = "mlp.", mixer_norm_prefix: str = "norm1", ffn_norm_prefix: str = "norm2") -> None:
+        self.mixer = MIXERS.build(mixer)
+        self.feed_forward = FEED_FORWARDS.build(feed_forward) if feed_forward is not None else None
+        self.mixer_norm = NORMS.build(mixer_norm)
+        self.ffn_norm = NORMS.build(ffn_norm) if feed_forward is not None else None
+        self._children = [(mixer_prefix, self.mixer), (mixer_norm_prefix, self.mixer_norm)]
+        if self.feed_forward is not None:
+            self._children += [(ffn_prefix, self.feed_forward), (ffn_norm_prefix, self.ffn_norm)]
+        self.dtype: Optional[torch.dtype] = None
+
+    @property
+    def takes_padding(self) -> bool:
+        return bool(self.mixer.takes_padding and (self.feed_forward is None or self.feed_forward.takes_padding))
+
+    def tensors(self) -> Sequence[TensorDecl]:
+        return [decl for prefix, part in self._children for decl in _prefixed(prefix, part.tensors())]
+
+    def load(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> None:
+        self.dtype = dtype
+        for prefix, part in self._children:
+            part.load(_strip(prefix, tensors), dtype, device)
+
+    def weight_bytes(self) -> int:
+        return sum(part.weight_bytes() for _, part in self._children)
+
+    def forward(self, stream: ResidualStream, step: StepView, cache: LayerCache) -> None:
+        self.mixer_norm.join(stream, self.mixer.forward(stream.read(self.dtype), step, cache))
+        if self.feed_forward is not None:
+            self.ffn_norm.join(stream, self.feed_forward.forward(stream.read(self.dtype), step))

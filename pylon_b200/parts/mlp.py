@@ -130,14 +130,26 @@ class ExpertMixture(FeedForward):
     ``correction [experts]``), with ``groups`` only among the experts of the ``groups_keep`` groups of neighbours whose two largest
     choice scores add up to most; the weights are the chosen experts' scores, without the correction, divided by their sum plus
     ``share_eps``.  ``shared_intermediate`` F: one more ungated expert ``shared.up [F, width]`` / ``shared.down`` that every token goes
-    through, added times ``sigmoid(w x)``, ``w`` the tensor ``shared.sg [1, width]`` (it rides in the router's product)."""
+    through, added times ``sigmoid(w x)``, ``w`` the tensor ``shared.sg [1, width]`` (it rides in the router's product).
+    ``share_normalized=False`` (sigmoid routing): the weights are the chosen experts' scores as they are.  ``weigh="input"``: an expert's
+    weight multiplies what it reads, not what it gives: the output is ``sum_e expert_e(weight_e * x)``.  ``activation="clamped"`` with
+    ``limit`` and ``alpha``: the clamped gated unit of :class:`ClampedGLU` in every expert."""
 
     def __init__(self, width: int, intermediate: int, experts: int, top: int, activation: str = "silu", router_bias: bool = False,
                  names: Optional[Mapping[str, str]] = None, gated: bool = True, routing: str = "softmax", correction: bool = False,
                  groups: Optional[int] = None, groups_keep: Optional[int] = None, share_eps: float = 0.0,
-                 shared_intermediate: Optional[int] = None) -> None:
-        if activation not in ops.ACTIVATIONS:
-            raise ValueError(f"unknown activation {activation!r} (known: {', '.join(ops.ACTIVATIONS)})")
+                 shared_intermediate: Optional[int] = None, share_normalized: bool = True, weigh: str = "output", limit: Optional[float] = None,
+                 alpha: float = 1.702) -> None:
+        if activation not in ops.ACTIVATIONS and activation != "clamped":
+            raise ValueError(f"unknown activation {activation!r} (known: {', '.join(ops.ACTIVATIONS)}, clamped)")
+        if (activation == "clamped") != (limit is not None) or (limit is not None and not (limit > 0 and gated)):
+            raise ValueError("a clamped unit has a gate and a positive limit, and no other activation has a limit")
+        if weigh not in ("output", "input") or (weigh == "input" and not gated):
+            raise ValueError(f"the weights multiply a gated expert's 'output' or its 'input', not {weigh!r}")
+        if not share_normalized and routing != "sigmoid":
+            raise ValueError("weights that do not add up to one go with sigmoid routing")
+        self.share_normalized, self.weigh = bool(share_normalized), weigh
+        self.limit, self.alpha = (None if limit is None else float(limit)), float(alpha)
         self.width, self.intermediate, self.experts, self.top = int(width), int(intermediate), int(experts), int(top)
         if not 1 <= self.top <= self.experts:
             raise ValueError(f"a token cannot use {top} of {experts} experts")
@@ -177,9 +189,9 @@ class ExpertMixture(FeedForward):
         return decls
 
     def load(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> None:
-        # In bfloat16 with silu an expert's gate and up rows alternate in groups of 8, the layout the tcgen05 product's gated epilogue
+        # In bfloat16 with silu or the clamped unit an expert's gate and up rows alternate in groups of 8, the layout the tcgen05 product's gated epilogue
         # takes (the products for few tokens read either layout); otherwise the two halves lie one after the other.
-        self.interleaved = self.gated and dtype == torch.bfloat16 and self.activation == "silu" and self.intermediate % 8 == 0
+        self.interleaved = self.gated and dtype == torch.bfloat16 and self.activation in ("silu", "clamped") and self.intermediate % 8 == 0
         if self.gated:
             pair = ops.interleave_gate_up if self.interleaved else (lambda gate, up: torch.cat((gate, up), dim=0))
             self.w_gate_up = torch.stack([pair(tensors[self._expert(e, "gate")], tensors[self._expert(e, "up")]) for e in range(self.experts)]).contiguous()
@@ -201,4 +213,5 @@ class ExpertMixture(FeedForward):
     def forward(self, h: torch.Tensor, step: StepView) -> torch.Tensor:
         return ops.expert_mixture(h, self.w_router, self.b_router, self.w_gate_up, self.w_down, self.top, self.activation, self.interleaved,
                                   gated=self.gated, routing=self.routing, correction=self.correction, groups=self.groups, groups_keep=self.groups_keep,
-                                  share_eps=self.share_eps, common_up=self.w_shared_up, common_down=self.w_shared_down)
+                                  share_eps=self.share_eps, common_up=self.w_shared_up, common_down=self.w_shared_down, share_normalized=self.share_normalized,
+                                  weigh=self.weigh, limit=self.limit, alpha=self.alpha)

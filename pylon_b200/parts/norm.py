@@ -46,6 +46,16 @@ class RMSNorm(Norm):
         # With a row selection the residual stays untouched and the delta is added on the fly.
         return ops.add_rmsnorm(stream.residual, delta, self.weight, self.eps, self.dtype, rows=rows)
 
+    def join(self, stream: ResidualStream, output: torch.Tensor) -> None:
+        stream.flush()
+        stream.activation = ops.output_norm(stream.residual, output, self.weight, self.eps, self.dtype)
+
+    def enter(self, token_ids: torch.Tensor, table: torch.Tensor, scale: float) -> ResidualStream:
+        residual, activation = ops.embedding_norm(token_ids, table, self.weight, self.eps, self.dtype, scale)
+        stream = ResidualStream(residual)
+        stream.activation = activation
+        return stream
+
 
 def _apply_to_streams(norm, kind: str, stream: ResidualStream, rows: Optional[torch.Tensor], read: Optional[torch.Tensor]) -> torch.Tensor:
     """The general form: one or several copies of the stream, a factor on the pending delta, a route by which it enters

@@ -63,7 +63,11 @@ class ParallelMixers(Mixer):
 @MIXERS.register("weighted_mixers")
 class WeightedMixers(ParallelMixers):
     """Mixers side by side whose outputs are added, each times a fixed factor: ``y = sum_i scale_i * mixer_i(h)``, one float32
-    kernel whose result enters the residual sum in 32-bit.  No norms, so no tensors beyond the mixers' own."""
+    kernel whose result enters the residual sum in 32-bit.  No norms, so no tensors beyond the mixers' own.
+
+    Where every mixer splits off its products (``Mixer.splits_products``) the layer has one product in and one out: the mixers' first
+    matrices are stacked by rows, their last ones side by side by columns, each mixer's middle reads its slice of the one row and leaves
+    its slice of the other times its factor, and the sum over the mixers is the last product's own."""
 
     def __init__(self, mixers: Sequence[PartSpec], prefixes: Sequence[str], scales: Sequence[float]) -> None:
         if not 1 <= len(mixers) <= 4 or len(prefixes) != len(mixers) or len(scales) != len(mixers):
@@ -71,6 +75,9 @@ class WeightedMixers(ParallelMixers):
         self.mixers = [MIXERS.build(spec) for spec in mixers]
         self.prefixes, self.norm_names = tuple(prefixes), ()
         self.scales = tuple(float(scale) for scale in scales)
+        self.w_in = self.w_out = None            # the stacked matrices, where the mixers split off their products
+        self.in_slices: list = []                # per mixer: its columns of the product's row, of the last product's operand
+        self.out_slices: list = []
 
     def tensors(self) -> Sequence[TensorDecl]:
         return [TensorDecl(prefix + d.name, d.shape, d.role, d.init) for prefix, mixer in zip(self.prefixes, self.mixers) for d in mixer.tensors()]
@@ -79,10 +86,38 @@ class WeightedMixers(ParallelMixers):
         for prefix, mixer in zip(self.prefixes, self.mixers):
             mixer.load({name[len(prefix):]: tensor for name, tensor in tensors.items() if name.startswith(prefix)}, dtype, device)
         self.dtype = dtype
+        if all(mixer.splits_products for mixer in self.mixers):
+            self._stack()
+
+    def _stack(self) -> None:
+        def slices(sizes):   # every mixer's slice starts at a multiple of 8 numbers: a 16-byte address in either dtype
+            starts = [0]
+            for size in sizes:
+                starts.append(starts[-1] + -(-size // 8) * 8)
+            return [slice(start, start + size) for start, size in zip(starts, sizes)], starts[-1]
+
+        first = self.mixers[0]
+        width = first.input_rows.shape[1]
+        self.in_slices, rows = slices([mixer.input_rows.shape[0] for mixer in self.mixers])
+        self.out_slices, columns = slices([mixer.output_columns.shape[1] for mixer in self.mixers])
+        self.w_in = first.input_rows.new_zeros((rows, width))
+        self.w_out = first.output_columns.new_zeros((width, columns))
+        for mixer, into, out_of in zip(self.mixers, self.in_slices, self.out_slices):
+            self.w_in[into] = mixer.input_rows
+            self.w_out[:, out_of] = mixer.output_columns
+            mixer.input_rows, mixer.output_columns = self.w_in[into], self.w_out[:, out_of]   # no second copy
+        self.filled = columns == sum(part.stop - part.start for part in self.out_slices)
 
     def weight_bytes(self) -> int:
         return sum(mixer.weight_bytes() for mixer in self.mixers)
 
     def forward(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> torch.Tensor:
+        if self.w_in is not None:
+            proj = ops.linear(h, self.w_in)
+            # columns between the slices meet zeros of the last product's matrix, so they must hold numbers
+            middle = (torch.empty if self.filled else torch.zeros)((h.shape[0], self.w_out.shape[1]), dtype=h.dtype, device=h.device)
+            for mixer, scale, into, out_of in zip(self.mixers, self.scales, self.in_slices, self.out_slices):
+                mixer.middle(proj[:, into], step, cache, middle[:, out_of], scale)
+            return ops.linear_for_residual(middle, self.w_out)
         outputs = [mixer.forward(h, step, cache) for mixer in self.mixers]
         return ops.weighted_sum(outputs, self.scales, self.dtype)

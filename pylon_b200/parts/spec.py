@@ -76,6 +76,8 @@ class ModelSpec:
     position_name: Optional[str] = None     # checkpoint name of a learnt table [position_rows, width]: row p is added to the embedding of the token at position p
     position_rows: int = 0
     reentry_name: Optional[str] = None      # checkpoint name of the [width, 2 width] matrix that runs with ``reenter`` go through
+    embedding_norm: Optional[PartSpec] = None   # the embedding rows go through this norm, and what it gives is the stream they start
+    embedding_norm_prefix: str = ""
 
     def __post_init__(self) -> None:
         runs = tuple(run if isinstance(run, RunSpec) else RunSpec(int(run)) for run in self.order)
@@ -85,6 +87,8 @@ class ModelSpec:
             raise ValueError("a model must run at least one layer")
         if any(run.reenter for run in runs) and (self.reentry_name is None or self.streams != 1):
             raise ValueError("a run that re-enters needs the model's reentry matrix and a residual stream of one copy")
+        if self.embedding_norm is not None and (self.streams != 1 or self.position_name is not None or any(run.add_embedding for run in runs)):
+            raise ValueError("a norm on the embedding goes with a residual stream of one copy, without learnt positions and rows added again")
         if self.position_name is not None and not 0 < self.max_positions <= self.position_rows:
             raise ValueError(f"{self.max_positions} positions, but the table of learnt positions has {self.position_rows} rows")
         for position, run in enumerate(runs):
