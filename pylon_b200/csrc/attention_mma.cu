@@ -16,6 +16,12 @@
 // Semantics as raun6k/Pylon's attention call (src/pylon/kv/cache.py:462-476, restated
 // 483-491): key j of the same request is visible to the token at position p iff j <= p
 // (and j > p - window when a window is set); softmax scale 1/sqrt(d) unless given.
+//
+// Built with -DPYLON_SIGMOID_WEIGHTS=1 the library is another attention over the same tiles: the weight of a visible key is
+// sigmoid(score + b_h) with b a number per head, and nothing is divided by a sum over the keys.  There is no maximum to keep and
+// nothing to rescale, and partial results simply add up.  A weight enters the weighted sum as two bfloat16 numbers, the rounded
+// weight and what the rounding dropped, so that it counts with 16 of its 24 bits: a long row adds up many small weights, and no
+// sum of weights divides their common rounding out.  Head h of token t may be multiplied by sigmoid(gate[t, h]) as it is written.
 #include "common.cuh"
 
 #include <cuda.h>
@@ -25,8 +31,21 @@
 #ifndef PYLON_HEAD_DIM
 #define PYLON_HEAD_DIM 128
 #endif
+#ifndef PYLON_SIGMOID_WEIGHTS
+#define PYLON_SIGMOID_WEIGHTS 0
+#endif
 
 namespace pylon {
+
+constexpr bool SIGMOID = PYLON_SIGMOID_WEIGHTS != 0;
+
+// What goes with sigmoid weights (all unused with a softmax).
+struct HeadOptions {
+  const float* score_bias;       // [nq] or null: added to the scaled scores
+  const __nv_bfloat16* gate;     // [tokens, >= nq], rows gate_stride apart, or null
+  long long gate_stride;
+  float factor;                  // on every output
+};
 
 constexpr int D = PYLON_HEAD_DIM;
 static_assert(D % 16 == 0 && D >= 16 && D <= 256, "head size must be a multiple of 16 in 16..256");
@@ -57,6 +76,8 @@ struct AttentionParams {
   unsigned* counters;         // [rows * nkv], zero between launches: the last block of a decoded (row, KV head) combines its segments
   int* error;                 // set non-zero when a bounded wait for a TMA copy ran out (the output is then void)
   float scale_log2;     // softmax scale * log2(e)
+  long long out_stride; // elements between the output rows of two tokens
+  HeadOptions heads;
 };
 
 // The first key that the token at position pos sees (a window, a chunk of positions, both or neither); it never decreases with pos.
@@ -106,6 +127,18 @@ __device__ __forceinline__ float soft_tanh(float x) {
 __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<unsigned*>(&v);
+}
+// sigmoid(x) for x in log2 units; exactly 0 for -infinity.
+__device__ __forceinline__ float sigmoid_exp2(float x) { return __fdividef(1.f, 1.f + fast_exp2(-x)); }
+// What pack_bf16 dropped of its two numbers, packed.
+__device__ __forceinline__ unsigned pack_dropped(float lo, float hi, unsigned packed) {
+  return pack_bf16(lo - __uint_as_float(packed << 16), hi - __uint_as_float(packed & 0xffff0000u));
+}
+__device__ __forceinline__ float head_score_bias(const HeadOptions& o, int head) { return SIGMOID && o.score_bias ? o.score_bias[head] * 1.4426950408889634f : 0.f; }
+// What an output of this head is multiplied by.
+__device__ __forceinline__ float head_factor(const HeadOptions& o, size_t token, int head) {
+  if (!SIGMOID) return 1.f;
+  return o.gate ? o.factor * sigmoid_exp2(1.4426950408889634f * __bfloat162float(o.gate[token * o.gate_stride + head])) : o.factor;
 }
 
 // Gathers keys [tile * 64, tile * 64 + 64) of one KV head into a padded shared tile.  Keys
@@ -186,6 +219,7 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
   int row_pos[MT][2], row_token[MT][2], row_head[MT][2], row_lo[MT][2];
   const bool bounded = p.window > 0 || p.chunk > 0;
   bool row_valid[MT][2];
+  float row_bias[MT][2];
   int warp_min_pos = 0x7fffffff;
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
@@ -197,6 +231,7 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
       row_head[mt][h] = kv_head * G + (row_valid[mt][h] ? m % G : 0);
       row_pos[mt][h] = pos0 + row_token[mt][h];
       row_lo[mt][h] = first_visible(p, row_pos[mt][h]);
+      row_bias[mt][h] = head_score_bias(p.heads, row_head[mt][h]);
     }
   }
   // Smallest position among the warp's rows (rows past the end count as the first row): tiles
@@ -306,11 +341,19 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
           }
         }
 
-        // Online softmax in float32 (base 2).
+        // Online softmax in float32 (base 2), or a sigmoid of every score.
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
           for (int h = 0; h < 2; ++h) {
+            if (SIGMOID) {
+#pragma unroll
+              for (int n = 0; n < BLOCK_N / 8; ++n) {
+                s[mt][n][2 * h] = sigmoid_exp2(fmaf(s[mt][n][2 * h], p.scale_log2, row_bias[mt][h]));
+                s[mt][n][2 * h + 1] = sigmoid_exp2(fmaf(s[mt][n][2 * h + 1], p.scale_log2, row_bias[mt][h]));
+              }
+              continue;
+            }
             float mx = -INFINITY;
 #pragma unroll
             for (int n = 0; n < BLOCK_N / 8; ++n) mx = fmaxf(mx, fmaxf(s[mt][n][2 * h], s[mt][n][2 * h + 1]));
@@ -343,13 +386,15 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
         // O += P V
 #pragma unroll
         for (int kk = 0; kk < BLOCK_N / 16; ++kk) {
-          unsigned a[MT][4];
+          unsigned a[MT][4], dropped[MT][4];
 #pragma unroll
           for (int mt = 0; mt < MT; ++mt) {
-            a[mt][0] = pack_bf16(s[mt][2 * kk][0], s[mt][2 * kk][1]);
-            a[mt][1] = pack_bf16(s[mt][2 * kk][2], s[mt][2 * kk][3]);
-            a[mt][2] = pack_bf16(s[mt][2 * kk + 1][0], s[mt][2 * kk + 1][1]);
-            a[mt][3] = pack_bf16(s[mt][2 * kk + 1][2], s[mt][2 * kk + 1][3]);
+#pragma unroll
+            for (int f = 0; f < 4; ++f) {
+              const float low = s[mt][2 * kk + (f >> 1)][2 * (f & 1)], high = s[mt][2 * kk + (f >> 1)][2 * (f & 1) + 1];
+              a[mt][f] = pack_bf16(low, high);
+              if (SIGMOID) dropped[mt][f] = pack_dropped(low, high, a[mt][f]);
+            }
           }
 #pragma unroll
           for (int d2 = 0; d2 < D / 16; ++d2) {
@@ -359,6 +404,10 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
             for (int mt = 0; mt < MT; ++mt) {
               mma_bf16(o[mt][2 * d2], a[mt], b[0], b[1]);
               mma_bf16(o[mt][2 * d2 + 1], a[mt], b[2], b[3]);
+              if (SIGMOID) {
+                mma_bf16(o[mt][2 * d2], dropped[mt], b[0], b[1]);
+                mma_bf16(o[mt][2 * d2 + 1], dropped[mt], b[2], b[3]);
+              }
             }
           }
         }
@@ -376,10 +425,10 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
       sum += __shfl_xor_sync(0xffffffffu, sum, 1);
       sum += __shfl_xor_sync(0xffffffffu, sum, 2);
       if (!row_valid[mt][h]) continue;
-      const float inv = sum > 0.f ? 1.f / sum : 0.f;
       const size_t token = (size_t)q0 + row_token[mt][h];
+      const float inv = SIGMOID ? (p.num_splits == 1 ? head_factor(p.heads, token, row_head[mt][h]) : 1.f) : (sum > 0.f ? 1.f / sum : 0.f);
       if (p.num_splits == 1) {
-        __nv_bfloat16* dst = p.out + (token * p.nq + row_head[mt][h]) * D;
+        __nv_bfloat16* dst = p.out + token * p.out_stride + (size_t)row_head[mt][h] * D;
 #pragma unroll
         for (int i = 0; i < D / 8; ++i)
           *reinterpret_cast<__nv_bfloat162*>(dst + i * 8 + 2 * tq) = __floats2bfloat162_rn(o[mt][i][2 * h] * inv, o[mt][i][2 * h + 1] * inv);
@@ -389,7 +438,7 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
 #pragma unroll
         for (int i = 0; i < D / 8; ++i)
           *reinterpret_cast<float2*>(dst + i * 8 + 2 * tq) = make_float2(o[mt][i][2 * h] * inv, o[mt][i][2 * h + 1] * inv);
-        if (tq == 0) p.partial_lse[slot] = sum > 0.f ? row_max[mt][h] * p.scale_log2 + log2f(sum) : -INFINITY;
+        if (tq == 0 && !SIGMOID) p.partial_lse[slot] = sum > 0.f ? row_max[mt][h] * p.scale_log2 + log2f(sum) : -INFINITY;
       }
     }
   }
@@ -766,10 +815,11 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
           }
           run_max = new_max;
         }
-        const float inv = run_total > 0.f ? 1.f / run_total : 0.f;
         const size_t token = (size_t)q0 + r / G;
         const int head = kv_head * G + r % G;
-        __nv_bfloat16* dst = p.out + (token * p.nq + head) * D + col;
+        // with sigmoid weights every segment's log-sum-exp is written as 0: the parts have been added up with weights of one
+        const float inv = SIGMOID ? head_factor(p.heads, token, head) : (run_total > 0.f ? 1.f / run_total : 0.f);
+        __nv_bfloat16* dst = p.out + token * p.out_stride + (size_t)head * D + col;
         *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(sum.x * inv, sum.y * inv), pack_bf16(sum.z * inv, sum.w * inv));
       }
       if (threadIdx.x == 0) p.counters[pair] = 0u;   // ready for the next launch
@@ -791,10 +841,12 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
 
     int row_pos[2], row_lo[2];
     bool row_valid[2];
+    float row_bias[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int m = g + 8 * h;
       row_valid[h] = m < packed_rows;
+      row_bias[h] = head_score_bias(p.heads, kv_head * G + (row_valid[h] ? m % G : 0));
       row_pos[h] = pos0 + (row_valid[h] ? m / G : 0);
       row_lo[h] = first_visible(p, row_pos[h]);
     }
@@ -928,6 +980,14 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
         // One decoded token times a group of up to 8 fills rows 0..7 only: rows 8..15 hold zero
         // queries, their scores stay zero and nothing of them is stored.
         if (h == 1 && upper_rows_unused) continue;
+        if (SIGMOID) {
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            s[n][2 * h] = sigmoid_exp2(fmaf(s[n][2 * h], p.scale_log2, row_bias[h]));
+            s[n][2 * h + 1] = sigmoid_exp2(fmaf(s[n][2 * h + 1], p.scale_log2, row_bias[h]));
+          }
+          continue;
+        }
         float mx = fmaxf(fmaxf(s[0][2 * h], s[0][2 * h + 1]), fmaxf(s[1][2 * h], s[1][2 * h + 1]));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
@@ -954,12 +1014,21 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
       a[1] = pack_bf16(s[0][2], s[0][3]);
       a[2] = pack_bf16(s[1][0], s[1][1]);
       a[3] = pack_bf16(s[1][2], s[1][3]);
+      unsigned dropped[4];
+      if (SIGMOID) {
+#pragma unroll
+        for (int f = 0; f < 4; ++f) dropped[f] = pack_dropped(s[f >> 1][2 * (f & 1)], s[f >> 1][2 * (f & 1) + 1], a[f]);
+      }
 #pragma unroll
       for (int d2 = 0; d2 < D / 16; ++d2) {
         unsigned b[4];
         ldmatrix_x4_trans(b, vs + Tiles::offset(key_row + 8 * ((lane >> 3) & 1), d2 * 2 + (lane >> 4)));
         mma_bf16(o[2 * d2], a, b[0], b[1]);
         mma_bf16(o[2 * d2 + 1], a, b[2], b[3]);
+        if (SIGMOID) {
+          mma_bf16(o[2 * d2], dropped, b[0], b[1]);
+          mma_bf16(o[2 * d2 + 1], dropped, b[2], b[3]);
+        }
       }
       __syncthreads();   // everyone is done with this stage before it is loaded again
     }
@@ -998,7 +1067,12 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
     }
     __syncthreads();
     // Per row, once: the warps' weights 2^(max_w - max) over the total, and the log-sum-exp.
-    if (threadIdx.x < packed_rows) {
+    if (SIGMOID && threadIdx.x < packed_rows) {   // the warps' results add up as they are
+#pragma unroll
+      for (int w = 0; w < 4; ++w) merge_max[w * SMALL_ROWS + threadIdx.x] = 1.f;
+      row_lse[threadIdx.x] = 0.f;
+    }
+    if (!SIGMOID && threadIdx.x < packed_rows) {
       const int r = threadIdx.x;
       float mx = -INFINITY;
 #pragma unroll
@@ -1052,7 +1126,8 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
       if (segments == 1) {
         const size_t token = (size_t)q0 + r / G;
         const int head = kv_head * G + r % G;
-        p.out[(token * p.nq + head) * D + col] = __float2bfloat16_rn(value);
+        if (SIGMOID) value *= head_factor(p.heads, token, head);
+        p.out[token * p.out_stride + (size_t)head * D + col] = __float2bfloat16_rn(value);
       } else {
         p.decode_out[(slot * SMALL_ROWS + r) * D + col] = value;
         if (col == 0) p.decode_lse[slot * SMALL_ROWS + r] = row_lse[r];
@@ -1119,7 +1194,7 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
       }
       const size_t token = (size_t)q0 + r / G;
       const int head = kv_head * G + r % G;
-      p.out[(token * p.nq + head) * D + col] = __float2bfloat16_rn(total > 0.f ? sum / total : 0.f);
+      p.out[token * p.out_stride + (size_t)head * D + col] = __float2bfloat16_rn(SIGMOID ? sum * head_factor(p.heads, token, head) : (total > 0.f ? sum / total : 0.f));
     }
   }
 }
@@ -1130,7 +1205,7 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
 // kernel wrote them).
 __global__ void combine_splits_kernel(const float* __restrict__ partial_out, const float* __restrict__ partial_lse,
                                       __nv_bfloat16* __restrict__ out, int num_splits, long long items, const int* __restrict__ q_start,
-                                      int num_rows, int nq, int group, int skip_small) {
+                                      int num_rows, int nq, int group, int skip_small, long long out_stride, HeadOptions heads) {
   grid_dependency_wait();
   allow_dependents();   // only now: a kernel that is itself still waiting must not pull the next one onto the SMs
   const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -1146,15 +1221,15 @@ __global__ void combine_splits_kernel(const float* __restrict__ partial_out, con
   }
   const int lane = threadIdx.x & 31;
   float mx = -INFINITY;
-  for (int s = 0; s < num_splits; ++s) mx = fmaxf(mx, partial_lse[(size_t)s * items + item]);
+  for (int s = 0; !SIGMOID && s < num_splits; ++s) mx = fmaxf(mx, partial_lse[(size_t)s * items + item]);
   float acc[(D + 31) / 32];
 #pragma unroll
   for (int i = 0; i < (D + 31) / 32; ++i) acc[i] = 0.f;
   float total = 0.f;
   for (int s = 0; s < num_splits; ++s) {
-    const float lse = partial_lse[(size_t)s * items + item];
+    const float lse = SIGMOID ? 0.f : partial_lse[(size_t)s * items + item];
     if (lse == -INFINITY) continue;
-    const float w = exp2f(lse - mx);
+    const float w = SIGMOID ? 1.f : exp2f(lse - mx);
     total += w;
     const float* src = partial_out + ((size_t)s * items + item) * D;
 #pragma unroll
@@ -1163,11 +1238,11 @@ __global__ void combine_splits_kernel(const float* __restrict__ partial_out, con
       if (e < D) acc[i] += w * src[e];
     }
   }
-  const float inv = total > 0.f ? 1.f / total : 0.f;
+  const float inv = SIGMOID ? head_factor(heads, (size_t)(item / nq), (int)(item % nq)) : (total > 0.f ? 1.f / total : 0.f);
 #pragma unroll
   for (int i = 0; i < (D + 31) / 32; ++i) {
     const int e = lane + 32 * i;
-    if (e < D) out[(size_t)item * D + e] = __float2bfloat16_rn(acc[i] * inv);
+    if (e < D) out[(size_t)(item / nq) * out_stride + (size_t)(item % nq) * D + e] = __float2bfloat16_rn(acc[i] * inv);
   }
 }
 
@@ -1314,13 +1389,14 @@ extern "C" long long pylon_attention_scratch_floats(int num_splits, int total_to
 // thread-block cluster of its own (with rows of very different lengths that would leave most blocks idle: the result is
 // right either way).
 // chunk > 0: attention inside chunks of positions (see AttentionParams); softcap c > 0: scaled scores go through c * tanh(s / c).
-extern "C" int pylon_paged_attention_mma_masked(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
+static int attention_mma_entry(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                 void* out, float* scratch, unsigned* counters, const int* q_start, const int* kv_len,
                                                 const int* block_table, int table_width, int page_size, int num_pages,
                                                 int nq, int nkv, int window, int chunk, float softcap, float scale, int num_rows,
                                                 int total_tokens, int max_q, int num_splits, int decode_blocks, int skip_large,
-                                                int rows_alike, int* error, cudaStream_t stream) {
+                                                int rows_alike, int* error, cudaStream_t stream, long long out_stride, const HeadOptions& heads) {
   if (num_rows <= 0 || total_tokens <= 0) return 0;
+  if (out_stride < (long long)nq * D || out_stride % 4) PYLON_REFUSE("paged_attention_mma: output rows of %d elements %lld apart (a multiple of 4)", nq * D, out_stride);
   if (chunk < 0 || softcap < 0.f) PYLON_REFUSE("paged_attention_mma: chunk %d, soft cap %f", chunk, softcap);
   if (nkv < 1 || nq < 1 || nq % nkv) PYLON_REFUSE("paged_attention_mma: %d query heads over %d KV heads", nq, nkv);
   if (page_size < 1 || table_width < 1 || window < 0 || max_q < 1 || num_splits < 1)
@@ -1370,6 +1446,8 @@ extern "C" int pylon_paged_attention_mma_masked(const void* q, long long q_strid
   p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride;
   p.k_pages = (const __nv_bfloat16*)k_pages; p.v_pages = (const __nv_bfloat16*)v_pages;
   p.out = (__nv_bfloat16*)out;
+  p.out_stride = out_stride;
+  p.heads = heads;
   const long long items = (long long)total_tokens * nq;
   float* decode_scratch = scratch;
   p.partial_out = p.partial_lse = nullptr;
@@ -1440,12 +1518,39 @@ extern "C" int pylon_paged_attention_mma_masked(const void* q, long long q_strid
     const int warps = 4;
     launch_dependent(combine_splits_kernel, dim3((unsigned)((items + warps - 1) / warps)), dim3(warps * 32), 0, stream,
                      (const float*)p.partial_out, (const float*)p.partial_lse, p.out, num_splits, items, q_start, num_rows, nq, group,
-                     maybe_small ? 1 : 0);
+                     maybe_small ? 1 : 0, out_stride, heads);
   }
   PYLON_CHECK_LAUNCH("paged_attention_mma");
 }
 
-// The same without chunks and soft cap.
+extern "C" int pylon_paged_attention_mma_masked(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
+                                                void* out, float* scratch, unsigned* counters, const int* q_start, const int* kv_len,
+                                                const int* block_table, int table_width, int page_size, int num_pages,
+                                                int nq, int nkv, int window, int chunk, float softcap, float scale, int num_rows,
+                                                int total_tokens, int max_q, int num_splits, int decode_blocks, int skip_large,
+                                                int rows_alike, int* error, cudaStream_t stream) {
+  if (SIGMOID) PYLON_REFUSE("paged_attention_mma: this library is built for sigmoid weights");
+  return attention_mma_entry(q, q_stride, k_pages, v_pages, out, scratch, counters, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv,
+                             window, chunk, softcap, scale, num_rows, total_tokens, max_q, num_splits, decode_blocks, skip_large, rows_alike, error, stream,
+                             (long long)nq * D, HeadOptions{nullptr, nullptr, 0, 1.f});
+}
+
+// Sigmoid weights (a library built for them): score_bias float32 [nq] or null; gate bfloat16 [tokens, >= nq] with rows gate_stride elements
+// apart, or null; factor on every output; out's rows out_stride elements apart.
+extern "C" int pylon_paged_attention_mma_sigmoid(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
+                                                 void* out, float* scratch, unsigned* counters, const int* q_start, const int* kv_len,
+                                                 const int* block_table, int table_width, int page_size, int num_pages,
+                                                 int nq, int nkv, int window, int chunk, float softcap, float scale, int num_rows,
+                                                 int total_tokens, int max_q, int num_splits, int decode_blocks, int skip_large,
+                                                 int rows_alike, int* error, const float* score_bias, const void* gate, long long gate_stride, float factor,
+                                                 long long out_stride, cudaStream_t stream) {
+  if (!SIGMOID) PYLON_REFUSE("paged_attention_mma: this library is built for a softmax");
+  return attention_mma_entry(q, q_stride, k_pages, v_pages, out, scratch, counters, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv,
+                             window, chunk, softcap, scale, num_rows, total_tokens, max_q, num_splits, decode_blocks, skip_large, rows_alike, error, stream,
+                             out_stride, HeadOptions{score_bias, (const __nv_bfloat16*)gate, gate_stride, factor});
+}
+
+// The softmax without chunks and soft cap.
 extern "C" int pylon_paged_attention_mma(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                          void* out, float* scratch, unsigned* counters, const int* q_start, const int* kv_len,
                                          const int* block_table, int table_width, int page_size, int num_pages,

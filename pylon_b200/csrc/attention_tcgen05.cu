@@ -33,6 +33,12 @@
 // Semantics as raun6k/Pylon's attention call (src/pylon/kv/cache.py:462-476, restated
 // 483-491): key j of the same request is visible to the token at position p iff j <= p (and
 // j > p - window when a window is set); softmax scale 1/sqrt(d) unless given.
+//
+// Built with -DPYLON_SIGMOID_WEIGHTS=1 the library is another attention over the same tiles: the weight of a visible key is
+// sigmoid(score + b_h) with b a number per head, and nothing is divided by a sum over the keys.  No maximum is kept and no output
+// rescaled.  A weight is two bfloat16 numbers, the rounded weight and what the rounding dropped (it counts with 16 of its 24 bits):
+// the two halves fill exactly the columns of the scores they replace, and the weighted sum is two products over one tile of values.
+// Two sigmoids share a reciprocal: with a = 1 + 2^-x and b = 1 + 2^-y, 1 / (a b) times b and times a.
 #include "common.cuh"
 
 #include <cuda.h>
@@ -42,10 +48,14 @@
 #ifndef PYLON_HEAD_DIM
 #define PYLON_HEAD_DIM 128
 #endif
+#ifndef PYLON_SIGMOID_WEIGHTS
+#define PYLON_SIGMOID_WEIGHTS 0
+#endif
 
 namespace pylon {
 
 constexpr int D = PYLON_HEAD_DIM;
+constexpr bool SIGMOID = PYLON_SIGMOID_WEIGHTS != 0;
 static_assert(D == 64 || D == 128, "the tcgen05 attention is built for head sizes 64 and 128");
 constexpr int FA_BM = 128, FA_BN = 64, FA_STAGES = 2, FA_THREADS = 192;
 constexpr int FA_SMALL_ROWS = 16;                  // rows with at most this many packed query rows belong to the decode kernel
@@ -74,6 +84,12 @@ struct FaParams {
                       // scale_log2 is c * log2(e), so that the softmax is that of c * tanh(scale * s / c)
   float scale_log2;
   int* error;
+  long long out_stride;            // elements between the output rows of two tokens
+  // with sigmoid weights
+  const float* score_bias;         // [nq] or null
+  const __nv_bfloat16* gate;       // [tokens, >= nq] with rows gate_stride elements apart, or null: head h of token t is multiplied by its sigmoid
+  long long gate_stride;
+  float factor;                    // on every output
 };
 
 // The first key that the token at position pos sees (a window, a chunk of positions, both or neither); it never decreases with pos.
@@ -166,6 +182,11 @@ __device__ __forceinline__ void fa_tmem_wait_stores() { asm volatile("tcgen05.wa
 __device__ __forceinline__ float fa_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float fa_reciprocal(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
 __device__ __forceinline__ unsigned fa_pack(float lo, float hi) {
@@ -321,6 +342,7 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
         for (int kk = 0; kk < FA_BN / 16; ++kk) {   // 16 keys: 32 bytes along a row of P, two 8-key groups (2048 bytes) down V
           const uint64_t b = fa_desc(v_tile + kk * 2048, FA_BN * 128, 1024);
           fa_mma_a_tmem(tmem_base + FA_O_COLUMN, tmem_base + (t & 1) * FA_S_COLUMNS + kk * 8, b, idesc_o, (t | kk) != 0 ? 1u : 0u);
+          if (SIGMOID) fa_mma_a_tmem(tmem_base + FA_O_COLUMN, tmem_base + (t & 1) * FA_S_COLUMNS + FA_BN / 2 + kk * 8, b, idesc_o, 1u);   // what the rounding dropped
         }
         fa_commit(&v_empty[t & 1]);
         fa_commit(&pv_done[t & 1]);
@@ -364,6 +386,7 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
     const unsigned lane_base = tmem_base + ((unsigned)(warp * 32) << 16);
     float reference = -INFINITY;   // the maximum the weights refer to (log2 units, scaled)
     float sum = 0.f;
+    const float bias_log2 = SIGMOID && p.score_bias ? p.score_bias[head] * 1.4426950408889634f : 0.f;
     bool alive = true;
     for (int t = 0; t < num_tiles; ++t) {
       if (!fa_mbar_wait(&s_full[t & 1], (t >> 1) & 1)) { atomicExch(p.error, 3); alive = false; break; }
@@ -385,7 +408,8 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
 #pragma unroll
         for (int j = 0; j < FA_BN; ++j) s[j] = 1.f - __fdividef(2.f, fa_exp2(s[j] * (p.cap_pre * 2.8853900817779268f)) + 1.f);
       }
-      if (p.window > 0 || p.chunk > 0 || key0 + FA_BN - 1 > pos0 + token_lo || !valid) {
+      const bool masked = p.window > 0 || p.chunk > 0 || key0 + FA_BN - 1 > pos0 + token_lo || !valid;
+      if (masked) {
 #pragma unroll
         for (int j = 0; j < FA_BN; ++j) {
           const int key = key0 + j;
@@ -393,44 +417,64 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
           if (!visible) s[j] = -INFINITY;
         }
       }
-      // Eight chains side by side: one chain of 63 dependent comparisons would cost more than the exponentials.
-      float lane_max[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) lane_max[j] = s[j];
-#pragma unroll
-      for (int j = 8; j < FA_BN; ++j) lane_max[j & 7] = fmaxf(lane_max[j & 7], s[j]);
-      float tile_max = fmaxf(fmaxf(fmaxf(lane_max[0], lane_max[1]), fmaxf(lane_max[2], lane_max[3])),
-                             fmaxf(fmaxf(lane_max[4], lane_max[5]), fmaxf(lane_max[6], lane_max[7])));
-      tile_max *= p.scale_log2;   // the scale is positive: the largest score stays the largest
-      // The reference moves only when the maximum has grown by more than the step (or was not set yet).
-      const bool move = tile_max > reference + FA_RESCALE_STEP || (reference == -INFINITY && tile_max > -INFINITY);
-      const float alpha = move ? (reference == -INFINITY ? 0.f : fa_exp2(reference - tile_max)) : 1.f;
-      if (move) reference = tile_max;
-      const float use = reference == -INFINITY ? 0.f : reference;
-      // The weights first, in registers: the product of the tile before this one may still be running.
-      sum *= alpha;
-      float part_sum[4] = {0.f, 0.f, 0.f, 0.f};   // four chains, for the same reason
       unsigned packed[FA_BN / 2];
+      if constexpr (SIGMOID) {
+        unsigned dropped[FA_BN / 2];
 #pragma unroll
-      for (int j = 0; j < FA_BN; j += 2) {
-        const float w0 = fa_exp2(fmaf(s[j], p.scale_log2, -use)), w1 = fa_exp2(fmaf(s[j + 1], p.scale_log2, -use));   // 0 for masked keys
-        part_sum[(j >> 1) & 3] += w0 + w1;
-        packed[j / 2] = fa_pack(w0, w1);
-      }
-      sum += (part_sum[0] + part_sum[1]) + (part_sum[2] + part_sum[3]);
-      // The weights go into tensor memory over this tile's scores, two to a column (this lane's scores are in registers
-      // and nothing else reads these columns before the weighted sum).  The output may be rescaled once the tile before
-      // this one is added up: only then is that product waited for.
-      if (t > 0 && __any_sync(0xffffffffu, move)) {   // tcgen05.ld/st are warp-wide: rows that stay multiply by one
-        if (!fa_mbar_wait(&pv_done[(t - 1) & 1], ((t - 1) >> 1) & 1)) { atomicExch(p.error, 3); alive = false; break; }
-        fa_fence_after();
+        for (int j = 0; j < FA_BN; j += 2) {
+          // 2^-x up to 2^60: the product of two stays in range, and a weight below 2^-60 is no weight
+          const float a = 1.f + fminf(fa_exp2(fmaf(s[j], -p.scale_log2, -bias_log2)), 1.152921504606847e18f);
+          const float b = 1.f + fminf(fa_exp2(fmaf(s[j + 1], -p.scale_log2, -bias_log2)), 1.152921504606847e18f);
+          const float shared = fa_reciprocal(a * b);
+          float w0 = shared * b, w1 = shared * a;
+          if (masked) {   // a key that is not seen weighs exactly nothing
+            if (s[j] == -INFINITY) w0 = 0.f;
+            if (s[j + 1] == -INFINITY) w1 = 0.f;
+          }
+          packed[j / 2] = fa_pack(w0, w1);
+          dropped[j / 2] = fa_pack(w0 - __uint_as_float(packed[j / 2] << 16), w1 - __uint_as_float(packed[j / 2] & 0xffff0000u));
+        }
+        fa_tmem_store_16(lane_base + (t & 1) * FA_S_COLUMNS + FA_BN / 2, dropped);
+        fa_tmem_store_16(lane_base + (t & 1) * FA_S_COLUMNS + FA_BN / 2 + 16, dropped + 16);
+      } else {
+        // Eight chains side by side: one chain of 63 dependent comparisons would cost more than the exponentials.
+        float lane_max[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) lane_max[j] = s[j];
+#pragma unroll
+        for (int j = 8; j < FA_BN; ++j) lane_max[j & 7] = fmaxf(lane_max[j & 7], s[j]);
+        float tile_max = fmaxf(fmaxf(fmaxf(lane_max[0], lane_max[1]), fmaxf(lane_max[2], lane_max[3])),
+                               fmaxf(fmaxf(lane_max[4], lane_max[5]), fmaxf(lane_max[6], lane_max[7])));
+        tile_max *= p.scale_log2;   // the scale is positive: the largest score stays the largest
+        // The reference moves only when the maximum has grown by more than the step (or was not set yet).
+        const bool move = tile_max > reference + FA_RESCALE_STEP || (reference == -INFINITY && tile_max > -INFINITY);
+        const float alpha = move ? (reference == -INFINITY ? 0.f : fa_exp2(reference - tile_max)) : 1.f;
+        if (move) reference = tile_max;
+        const float use = reference == -INFINITY ? 0.f : reference;
+        // The weights first, in registers: the product of the tile before this one may still be running.
+        sum *= alpha;
+        float part_sum[4] = {0.f, 0.f, 0.f, 0.f};   // four chains, for the same reason
+#pragma unroll
+        for (int j = 0; j < FA_BN; j += 2) {
+          const float w0 = fa_exp2(fmaf(s[j], p.scale_log2, -use)), w1 = fa_exp2(fmaf(s[j + 1], p.scale_log2, -use));   // 0 for masked keys
+          part_sum[(j >> 1) & 3] += w0 + w1;
+          packed[j / 2] = fa_pack(w0, w1);
+        }
+        sum += (part_sum[0] + part_sum[1]) + (part_sum[2] + part_sum[3]);
+        // The weights go into tensor memory over this tile's scores, two to a column (this lane's scores are in registers
+        // and nothing else reads these columns before the weighted sum).  The output may be rescaled once the tile before
+        // this one is added up: only then is that product waited for.
+        if (t > 0 && __any_sync(0xffffffffu, move)) {   // tcgen05.ld/st are warp-wide: rows that stay multiply by one
+          if (!fa_mbar_wait(&pv_done[(t - 1) & 1], ((t - 1) >> 1) & 1)) { atomicExch(p.error, 3); alive = false; break; }
+          fa_fence_after();
 #pragma unroll 1
-        for (int c = 0; c < D / 32; ++c) {
-          unsigned raw[32];
-          fa_tmem_load_32(lane_base + FA_O_COLUMN + c * 32, raw);
+          for (int c = 0; c < D / 32; ++c) {
+            unsigned raw[32];
+            fa_tmem_load_32(lane_base + FA_O_COLUMN + c * 32, raw);
 #pragma unroll
-          for (int j = 0; j < 32; ++j) raw[j] = __float_as_uint(__uint_as_float(raw[j]) * alpha);
-          fa_tmem_store_32(lane_base + FA_O_COLUMN + c * 32, raw);
+            for (int j = 0; j < 32; ++j) raw[j] = __float_as_uint(__uint_as_float(raw[j]) * alpha);
+            fa_tmem_store_32(lane_base + FA_O_COLUMN + c * 32, raw);
+          }
         }
       }
       fa_tmem_store_16(lane_base + (t & 1) * FA_S_COLUMNS, packed);
@@ -455,8 +499,12 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
     if (alive && !fa_mbar_wait(&pv_done[(num_tiles - 1) & 1], ((num_tiles - 1) >> 1) & 1)) { atomicExch(p.error, 3); alive = false; }
     if (alive) {
       fa_fence_after();
-      const float inv = sum > 0.f ? 1.f / sum : 0.f;
-      __nv_bfloat16* dst = p.out + ((size_t)(q0 + token) * p.nq + head) * D;
+      float inv = sum > 0.f ? 1.f / sum : 0.f;
+      if (SIGMOID) {
+        inv = p.factor;
+        if (p.gate && valid) inv *= __fdividef(1.f, 1.f + fa_exp2(-1.4426950408889634f * __bfloat162float(p.gate[(size_t)(q0 + token) * p.gate_stride + head])));
+      }
+      __nv_bfloat16* dst = p.out + (size_t)(q0 + token) * p.out_stride + (size_t)head * D;
 #pragma unroll 1
       for (int c = 0; c < D / 32; ++c) {
         unsigned raw[32];
@@ -537,12 +585,14 @@ extern "C" int pylon_attention_tcgen05_head_dim() { return D; }
 // with at most 16 packed query rows (tokens x group) are left alone (another kernel writes them).  error: one int in device memory that the kernel sets
 // non-zero when one of its bounded waits ran out (the output is then void).
 // chunk > 0: attention inside chunks of positions; softcap c > 0: scaled scores go through c * tanh(s / c) (see FaParams).
-extern "C" int pylon_paged_attention_tcgen05_masked(const void* q, long long q_stride, const void* k_pages, const void* v_pages, void* out,
+static int attention_tcgen05_entry(const void* q, long long q_stride, const void* k_pages, const void* v_pages, void* out,
                                                     const int* q_start, const int* kv_len, const int* block_table, int table_width,
                                                     int page_size, int num_pages, int nq, int nkv, int window, int chunk, float softcap,
                                                     float scale, int first_row, int num_rows, int max_q, int skip_small, int* error,
-                                                    cudaStream_t stream) {
+                                                    cudaStream_t stream, long long out_stride, const float* score_bias, const void* gate,
+                                                    long long gate_stride, float factor) {
   if (num_rows <= 0) return 0;
+  if (out_stride < (long long)nq * D || out_stride % 8) PYLON_REFUSE("paged_attention_tcgen05: output rows of %d elements %lld apart (a multiple of 8)", nq * D, out_stride);
   if (chunk < 0 || softcap < 0.f) PYLON_REFUSE("paged_attention_tcgen05: chunk %d, soft cap %f", chunk, softcap);
   if (nkv < 1 || nq < 1 || nq % nkv) PYLON_REFUSE("paged_attention_tcgen05: %d query heads over %d KV heads", nq, nkv);
   if (page_size < 64 || page_size % 64) PYLON_REFUSE("paged_attention_tcgen05: pages of %d keys; a multiple of 64 is needed", page_size);
@@ -573,13 +623,37 @@ extern "C" int pylon_paged_attention_tcgen05_masked(const void* q, long long q_s
   p.chunk = chunk;
   p.cap_pre = softcap > 0.f ? scale / softcap : 0.f;
   p.error = error;
+  p.out_stride = out_stride; p.score_bias = score_bias; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride; p.factor = factor;
   const long long q_tiles = ((long long)max_q * p.group + FA_BM - 1) / FA_BM;
   if (q_tiles > 65535) PYLON_REFUSE("paged_attention_tcgen05: too many query tiles");
   launch_dependent(attention_tcgen05_kernel, dim3(nkv, num_rows, (unsigned)q_tiles), dim3(FA_THREADS), FA_SMEM, stream, p, map_k, map_v);
   PYLON_CHECK_LAUNCH("paged_attention_tcgen05");
 }
 
-// The same without chunks and soft cap.
+extern "C" int pylon_paged_attention_tcgen05_masked(const void* q, long long q_stride, const void* k_pages, const void* v_pages, void* out,
+                                                    const int* q_start, const int* kv_len, const int* block_table, int table_width,
+                                                    int page_size, int num_pages, int nq, int nkv, int window, int chunk, float softcap,
+                                                    float scale, int first_row, int num_rows, int max_q, int skip_small, int* error,
+                                                    cudaStream_t stream) {
+  if (SIGMOID) PYLON_REFUSE("paged_attention_tcgen05: this library is built for sigmoid weights");
+  return attention_tcgen05_entry(q, q_stride, k_pages, v_pages, out, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv, window, chunk,
+                                 softcap, scale, first_row, num_rows, max_q, skip_small, error, stream, (long long)nq * D, nullptr, nullptr, 0, 1.f);
+}
+
+// Sigmoid weights (a library built for them): score_bias float32 [nq] or null; gate bfloat16 [tokens, >= nq] with rows gate_stride elements
+// apart, or null; factor on every output; out's rows out_stride elements apart.
+extern "C" int pylon_paged_attention_tcgen05_sigmoid(const void* q, long long q_stride, const void* k_pages, const void* v_pages, void* out,
+                                                     const int* q_start, const int* kv_len, const int* block_table, int table_width,
+                                                     int page_size, int num_pages, int nq, int nkv, int window, int chunk, float softcap,
+                                                     float scale, int first_row, int num_rows, int max_q, int skip_small, int* error,
+                                                     const float* score_bias, const void* gate, long long gate_stride, float factor, long long out_stride,
+                                                     cudaStream_t stream) {
+  if (!SIGMOID) PYLON_REFUSE("paged_attention_tcgen05: this library is built for a softmax");
+  return attention_tcgen05_entry(q, q_stride, k_pages, v_pages, out, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv, window, chunk,
+                                 softcap, scale, first_row, num_rows, max_q, skip_small, error, stream, out_stride, score_bias, gate, gate_stride, factor);
+}
+
+// The softmax without chunks and soft cap.
 extern "C" int pylon_paged_attention_tcgen05(const void* q, long long q_stride, const void* k_pages, const void* v_pages, void* out,
                                              const int* q_start, const int* kv_len, const int* block_table, int table_width,
                                              int page_size, int num_pages, int nq, int nkv, int window, float scale, int first_row,

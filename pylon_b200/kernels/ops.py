@@ -296,6 +296,9 @@ _SIGNATURES = {
         "pylon_paged_attention_mma_masked": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int,
                                              c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+        "pylon_paged_attention_mma_sigmoid": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int,
+                                              c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_float, c_longlong, c_void_p],
         "pylon_attention_scratch_floats": [c_int, c_int, c_int, c_int, c_int, c_int],
         "pylon_attention_decode_blocks": [],
     },
@@ -304,6 +307,9 @@ _SIGNATURES = {
                                           c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "pylon_paged_attention_tcgen05_masked": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                                  c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+        "pylon_paged_attention_tcgen05_sigmoid": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                                  c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                                                  c_void_p, c_longlong, c_float, c_longlong, c_void_p],
     },
     "sampling.cu": {
         "pylon_sample": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
@@ -1003,8 +1009,11 @@ def paged_attention(
     _need(head_gate is None or (head_gate.dtype == q.dtype and head_gate.shape == (tokens, nq) and head_gate.stride(1) == 1), "paged_attention: head_gate must be [T, nq] in the cache dtype")
     scale = 1.0 / math.sqrt(d) if scale is None else float(scale)
     _need(scale > 0 or sigmoid, "paged_attention: the softmax scale must be positive")
-    if q.dtype == torch.bfloat16 and d % 16 == 0 and d <= 256 and not force_simple and same_width and sinks is None and not plain_only and not sigmoid:
-        library = _library("attention_mma.cu", {"PYLON_HEAD_DIM": d})
+    if q.dtype == torch.bfloat16 and d % 16 == 0 and d <= 256 and not force_simple and same_width and sinks is None and not plain_only \
+            and (not sigmoid or (scale > 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)):
+        defines = {"PYLON_HEAD_DIM": d, **({"PYLON_SIGMOID_WEIGHTS": 1} if sigmoid else {})}
+        extra = (_ptr(score_bias), _ptr(head_gate), 0 if head_gate is None else head_gate.stride(0), float(out_factor), out.stride(0)) if sigmoid else ()
+        library = _library("attention_mma.cu", defines)
         group = nq // nkv
         any_large = max_q * group > 16
         # Rows of decoded tokens can occur unless the step is one long row.
@@ -1018,17 +1027,18 @@ def paged_attention(
         use_tcgen05 = any_large and prefill_kernel == "tcgen05"
         if use_tcgen05:
             _need(d in (64, 128) and page_size % 64 == 0, "paged_attention: the tcgen05 kernel needs head size 64 or 128 and pages of a multiple of 64 keys")
-            fast = _library("attention_tcgen05.cu", {"PYLON_HEAD_DIM": d})
+            fast = _library("attention_tcgen05.cu", defines)
             first_row, row_count = 0, rows
             if row_tokens is not None and len(row_tokens) == rows:
                 large = [index for index, count in enumerate(row_tokens) if count * group > 16]
                 if large and large[-1] - large[0] + 1 == len(large):   # one run of rows: the scheduler puts decoded rows first
                     first_row, row_count = large[0], len(large)
-            _check(fast, fast.pylon_paged_attention_tcgen05_masked(
+            entry = fast.pylon_paged_attention_tcgen05_sigmoid if sigmoid else fast.pylon_paged_attention_tcgen05_masked
+            _check(fast, entry(
                 _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(q_start), _ptr(kv_len), _ptr(block_table),
                 block_table.shape[1], page_size, num_pages, nq, nkv, int(window or 0), int(chunk or 0), float(softcap or 0.0), scale,
                 first_row, row_count, int(max_q), int(maybe_small),
-                _ptr(attention_error_word(q.device)), _stream()))
+                _ptr(attention_error_word(q.device)), *extra, _stream()))
             if not maybe_small:
                 return out
         splits = 1 if use_tcgen05 else (attention_splits(rows, nkv, group, max_q, max_kv, _multiprocessors(q.device)) if num_splits is None else int(num_splits))
@@ -1042,11 +1052,12 @@ def paged_attention(
             scratch = torch.empty((floats,), dtype=torch.float32, device=q.device)
         if blocks:
             counters = _zeroed_counters(q.device, "attention", rows * nkv)
-        _check(library, library.pylon_paged_attention_mma_masked(
+        entry = library.pylon_paged_attention_mma_sigmoid if sigmoid else library.pylon_paged_attention_mma_masked
+        _check(library, entry(
             _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(scratch), _ptr(counters), _ptr(q_start), _ptr(kv_len),
             _ptr(block_table), block_table.shape[1], page_size, num_pages, nq, nkv, int(window or 0), int(chunk or 0), float(softcap or 0.0),
             scale, rows, tokens,
-            int(max_q), splits, blocks, int(use_tcgen05), int(bool(rows_alike)), _ptr(attention_error_word(q.device)), _stream()))
+            int(max_q), splits, blocks, int(use_tcgen05), int(bool(rows_alike)), _ptr(attention_error_word(q.device)), *extra, _stream()))
         return out
     if ((plain_only or sinks is not None) and q.dtype == torch.bfloat16 and not force_simple and chunk is None and softcap is None and d % 16 == 0 and d <= 256 and dv % 8 == 0 and dv <= 256
             and nq // nkv <= 8 and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0):
