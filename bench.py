@@ -483,7 +483,7 @@ DESIGN_SIZES = {
     "4k": dict(width=4_096, layers=8, heads=32, kv_heads=8, head_dim=128, ff=12_288, vocab=32_768),
 }
 DESIGN_CONTEXT = 2_048
-_TIMED_OPS = ("linear", "linear_for_residual", "linear_swiglu", "linear_for_rotation", "linear_qkv_rotated", "paged_attention", "gated_delta_rule",
+_TIMED_OPS = ("linear", "linear_stacked", "linear_for_residual", "linear_swiglu", "linear_for_rotation", "linear_qkv_rotated", "paged_attention", "gated_delta_rule",
               "streams_update_norm", "add_rmsnorm", "swiglu", "qk_norm_mix_kv_write", "qk_norm_rope_kv_write", "embed_gather", "lightning_attention",
               "qkv_rotate_write", "latent_norm_rotate_write", "rotate_heads", "linear_heads", "state_space", "expert_mixture", "mean_of_normed",
               "gated_unit", "add_bias", "concat_cast", "linear_recurrence", "matrix_memory", "weighted_sum", "residual_add",

@@ -20,7 +20,7 @@
 // padded to whole tiles, and the grouped products run over the most tiles there can be; a tile beyond the last one, and
 // a slot of padding inside a tile, is skipped.
 //
-//   experts_route     router logits, the top choices, their shares: a block per token in a step of few tokens, else a warp per four
+//   experts_route     router logits, the top choices, their shares: a block per token in a step of few tokens, else a block per four
 //   experts_plan      one block: tokens per expert, the experts' first tiles, a slot for every pair
 //   experts_product   a block per (row tile, column tile): rows gathered by slot, the expert's matrix, float32 sums in a
 //                     fixed order of k; with GLU the gate and up tiles side by side and act(gate) * up written
@@ -173,107 +173,78 @@ __device__ __forceinline__ void route_choose_scored(float* logits, float* choice
 }
 
 // h [T, width] in T; router float32 [experts, width]; bias float32 [experts] or null.  chosen int32 [T, top], share float32 [T, top].
-// A logit is summed in one order whatever the kernel form: the columns fall into four classes by (c mod 128) / 32; within class k
-// lane l adds the columns 128 i + 32 k + l in order of i, the 32 lanes' sums are added up by the same butterfly, and the four class
-// sums are added in order of k.  So a token's choice does not depend on how many tokens the step has.
-//
-// Many tokens: a warp takes TOKENS tokens side by side, so that a router value it has loaded serves all of them, and walks the four
-// classes one after the other.  Shared memory: warps * TOKENS * experts floats.
-template <typename T, int TOKENS>
-__global__ void experts_route_kernel(const T* __restrict__ h, long long ld, const float* __restrict__ router, const float* __restrict__ bias,
-                                     int* __restrict__ chosen, float* __restrict__ share, int width, int experts, int top, int num_tokens,
-                                     RouteScored mode) {
-  extern __shared__ float logits_all[];
+// A block of four warps takes TOKENS tokens, so that a router value it has loaded serves all of them; a warp takes a quarter of the
+// columns.  A thread takes V neighbouring columns at a time (V 4 where the rows are whole pieces of it, else 1; by the sizes alone): warp k's
+// lane l adds up the columns V (128 i + 32 k + l) .. + V - 1 in order of i, its 32 lanes' sums are added by a butterfly, and the four warps'
+// sums in order of k.  So a token's logits, and with them its choice, do not depend on how many tokens the step has.
+// Shared memory: TOKENS * (4 * 8 + what a token takes) floats.
+template <typename T, int V>
+__device__ __forceinline__ void route_load(float (&x)[V], const T* from) {
+  if constexpr (V == 1) x[0] = to_float<T>(from[0]);
+  else if constexpr (sizeof(T) == 4) {
+    const float4 raw = *reinterpret_cast<const float4*>(from);
+    x[0] = raw.x; x[1] = raw.y; x[2] = raw.z; x[3] = raw.w;
+  } else {
+    const uint2 raw = *reinterpret_cast<const uint2*>(from);
+    const float2 low = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), high = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    x[0] = low.x; x[1] = low.y; x[2] = high.x; x[3] = high.y;
+  }
+}
+
+template <typename T, int TOKENS, int V>
+__global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict__ h, long long ld, const float* __restrict__ router, const float* __restrict__ bias,
+                                                            int* __restrict__ chosen, float* __restrict__ share, int width, int experts, int top, int num_tokens,
+                                                            RouteScored mode) {
+  extern __shared__ float route_shared[];
+  constexpr int SIDE = 8;   // experts side by side: the tokens' rows are read once per eight experts
   const int rows = experts + mode.extra;                                        // rows of the router
-  const int per_token = rows + (mode.on ? experts + mode.groups : 0);           // floats of shared memory a token takes
+  const int per_token = rows + (mode.on ? experts + mode.groups : 0);           // logits, then with mode.on choice scores and the groups' worths
+  float* parts = route_shared;                                                  // [4][TOKENS][SIDE]
+  float* logits = route_shared + 4 * TOKENS * SIDE;                             // [TOKENS][per_token]
   grid_dependency_wait();
   allow_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t0 = (blockIdx.x * (blockDim.x >> 5) + warp) * TOKENS;
-  if (t0 >= num_tokens) return;
-  constexpr int SIDE = 8;   // experts side by side: the tokens' rows are read once per eight experts
+  const int t0 = blockIdx.x * TOKENS;
   for (int e0 = 0; e0 < rows; e0 += SIDE) {
-    float total[TOKENS][SIDE];
-    for (int k = 0; k < 4; ++k) {
-      float acc[TOKENS][SIDE];
+    float acc[TOKENS][SIDE];
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i)
+#pragma unroll
+      for (int j = 0; j < SIDE; ++j) acc[i][j] = 0.f;
+#pragma unroll 2
+    for (int c = V * threadIdx.x; c < width; c += V * 128) {
+      float x[TOKENS][V], r[SIDE][V];
+#pragma unroll
+      for (int i = 0; i < TOKENS; ++i) route_load<T, V>(x[i], h + (long long)(t0 + i < num_tokens ? t0 + i : t0) * ld + c);
+#pragma unroll
+      for (int j = 0; j < SIDE; ++j) route_load<float, V>(r[j], router + (long long)(e0 + j < rows ? e0 + j : e0) * width + c);
 #pragma unroll
       for (int i = 0; i < TOKENS; ++i)
 #pragma unroll
-        for (int j = 0; j < SIDE; ++j) acc[i][j] = 0.f;
-#pragma unroll 4
-      for (int c = 32 * k + lane; c < width; c += 128) {   // unrolled, so that several columns' loads are on their way at once
-        float x[TOKENS], r[SIDE];
+        for (int j = 0; j < SIDE; ++j)
 #pragma unroll
-        for (int i = 0; i < TOKENS; ++i) x[i] = t0 + i < num_tokens ? to_float<T>(h[(long long)(t0 + i) * ld + c]) : 0.f;
-#pragma unroll
-        for (int j = 0; j < SIDE; ++j) r[j] = e0 + j < rows ? router[(long long)(e0 + j) * width + c] : 0.f;
-#pragma unroll
-        for (int i = 0; i < TOKENS; ++i)
-#pragma unroll
-          for (int j = 0; j < SIDE; ++j) acc[i][j] = fmaf(x[i], r[j], acc[i][j]);
-      }
-#pragma unroll
-      for (int i = 0; i < TOKENS; ++i)
-#pragma unroll
-        for (int j = 0; j < SIDE; ++j) {
-          const float z = warp_sum(acc[i][j]);
-          total[i][j] = k == 0 ? z : total[i][j] + z;
-        }
+          for (int v = 0; v < V; ++v) acc[i][j] = fmaf(x[i][v], r[j][v], acc[i][j]);
     }
 #pragma unroll
     for (int i = 0; i < TOKENS; ++i)
 #pragma unroll
-      for (int j = 0; j < SIDE; ++j)
-        if (lane == 0 && e0 + j < rows)
-          logits_all[(warp * TOKENS + i) * per_token + e0 + j] = total[i][j] + (bias != nullptr && e0 + j < experts ? bias[e0 + j] : 0.f);
+      for (int j = 0; j < SIDE; ++j) {
+        const float z = warp_sum(acc[i][j]);
+        if (lane == 0) parts[(warp * TOKENS + i) * SIDE + j] = z;
+      }
+    __syncthreads();
+    if (threadIdx.x < TOKENS * SIDE) {
+      const int i = threadIdx.x / SIDE, j = threadIdx.x % SIDE;
+      if (e0 + j < rows)
+        logits[i * per_token + e0 + j] = ((parts[i * SIDE + j] + parts[(TOKENS + i) * SIDE + j]) + parts[(2 * TOKENS + i) * SIDE + j]) + parts[(3 * TOKENS + i) * SIDE + j] +
+                                         (bias != nullptr && e0 + j < experts ? bias[e0 + j] : 0.f);
+    }
+    __syncthreads();
   }
-  __syncwarp();
-  for (int i = 0; i < TOKENS && t0 + i < num_tokens; ++i) {
-    float* mine = logits_all + (warp * TOKENS + i) * per_token;
+  for (int i = warp; i < TOKENS && t0 + i < num_tokens; i += 4) {
+    float* mine = logits + i * per_token;
     if (mode.on) route_choose_scored(mine, mine + rows, mine + rows + experts, chosen, share, t0 + i, experts, top, lane, mode);
     else route_choose(mine, chosen, share, t0 + i, experts, top, lane);
-  }
-}
-
-// Few tokens: a block of four warps per token, warp k takes class k.  Shared memory: (4 * 8 + experts) floats.
-template <typename T>
-__global__ void __launch_bounds__(128) experts_route_block_kernel(const T* __restrict__ h, long long ld, const float* __restrict__ router,
-                                                                  const float* __restrict__ bias, int* __restrict__ chosen, float* __restrict__ share,
-                                                                  int width, int experts, int top, RouteScored mode) {
-  extern __shared__ float route_shared[];
-  constexpr int SIDE = 8;
-  float* parts = route_shared;               // [4][SIDE]
-  float* logits = route_shared + 4 * SIDE;   // [experts + extra], then with mode.on [experts] choice scores and [groups] groups' worths
-  const int rows = experts + mode.extra;
-  grid_dependency_wait();
-  allow_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long t = blockIdx.x;
-  for (int e0 = 0; e0 < rows; e0 += SIDE) {
-    float acc[SIDE];
-#pragma unroll
-    for (int j = 0; j < SIDE; ++j) acc[j] = 0.f;
-#pragma unroll 4
-    for (int c = threadIdx.x; c < width; c += 128) {
-      const float x = to_float<T>(h[t * ld + c]);
-#pragma unroll
-      for (int j = 0; j < SIDE; ++j) acc[j] = fmaf(x, e0 + j < rows ? router[(long long)(e0 + j) * width + c] : 0.f, acc[j]);
-    }
-#pragma unroll
-    for (int j = 0; j < SIDE; ++j) {
-      const float z = warp_sum(acc[j]);
-      if (lane == 0) parts[warp * SIDE + j] = z;
-    }
-    __syncthreads();
-    if (threadIdx.x < SIDE && e0 + threadIdx.x < rows) {
-      const int j = threadIdx.x;
-      logits[e0 + j] = ((parts[j] + parts[SIDE + j]) + parts[2 * SIDE + j]) + parts[3 * SIDE + j] + (bias != nullptr && e0 + j < experts ? bias[e0 + j] : 0.f);
-    }
-    __syncthreads();
-  }
-  if (warp == 0) {
-    if (mode.on) route_choose_scored(logits, logits + rows, logits + rows + experts, chosen, share, t, experts, top, lane, mode);
-    else route_choose(logits, chosen, share, t, experts, top, lane);
   }
 }
 
@@ -421,7 +392,8 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
                                                                   const __nv_bfloat16* __restrict__ w, const int* __restrict__ source,
                                                                   const int* __restrict__ tile_expert, int gathered, int divide,
                                                                   void* __restrict__ out_v, int n_out, int k_size, int kind, int interleaved, int act_out,
-                                                                  const float* __restrict__ slot_share, float limit, float alpha) {
+                                                                  const float* __restrict__ slot_share, float limit, float alpha,
+                                                                  int k_each, long long part_stride) {
   constexpr int TN = MMA_TN, TK = MMA_TK, LD = MMA_TK + MMA_PAD, G = GLU ? 2 : 1, MMA_STAGES = mma_stages(GLU);
   constexpr int A_ELEMENTS = EXPERT_ROWS * LD, STAGE_ELEMENTS = mma_stage_elements(GLU);
   extern __shared__ __align__(16) unsigned char mma_shared[];
@@ -451,22 +423,24 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
       for (int j = 0; j < 2; ++j)
 #pragma unroll
         for (int f = 0; f < 4; ++f) acc[g][i][j][f] = 0.f;
-  const int steps = (k_size + TK - 1) / TK;
+  const int k_first = blockIdx.z * k_each;                                            // this block's share of k (all of it for a gated product)
+  const int k_last = k_first + k_each < k_size ? k_first + k_each : k_size;
+  const int steps = (k_last - k_first + TK - 1) / TK;
   auto fill = [&](int step) {   // every thread commits one group a call, also an empty one, so that the groups count the steps
     if (step < steps) {
-      const int k0 = step * TK;
+      const int k0 = k_first + step * TK;
       __nv_bfloat16* a_stage = ring + (size_t)(step % MMA_STAGES) * STAGE_ELEMENTS;
       __nv_bfloat16* b_stage = a_stage + A_ELEMENTS;
       for (int x = threadIdx.x; x < EXPERT_ROWS * (TK / 8); x += 128) {
         const int r = x / (TK / 8), c = (x % (TK / 8)) * 8;
         const int row = rows[r];
-        const bool real = row >= 0 && k0 + c < k_size;
+        const bool real = row >= 0 && k0 + c < k_last;
         copy_16_or_zeros(a_stage + r * LD + c, real ? a + (long long)row * lda + k0 + c : a, real);
       }
       for (int x = threadIdx.x; x < G * TN * (TK / 8); x += 128) {
         const int g = x / (TN * (TK / 8)), y = x % (TN * (TK / 8));
         const int r = y / (TK / 8), c = (y % (TK / 8)) * 8;
-        const bool real = n0 + r < n_out && k0 + c < k_size;
+        const bool real = n0 + r < n_out && k0 + c < k_last;
         copy_16_or_zeros(b_stage + (g * TN + r) * LD + c, real ? w_mine + glu_row(n0 + r, g, n_out, GLU && interleaved) * k_size + k0 + c : w_mine, real);
       }
     }
@@ -523,7 +497,7 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
           const float value = acc[0][i][j][2 * half + e];
           if (GLU) ((__nv_bfloat16*)out_v)[slot * n_out + n] = __float2bfloat16_rn(expert_unit(reads * value, reads * acc[G - 1][i][j][2 * half + e], kind, limit, alpha));
           else if (act_out) ((__nv_bfloat16*)out_v)[slot * n_out + n] = __float2bfloat16_rn(expert_activation(value, kind));
-          else ((float*)out_v)[slot * n_out + n] = value;
+          else ((float*)out_v)[blockIdx.z * part_stride + slot * n_out + n] = value;
         }
     }
 }
@@ -534,7 +508,7 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
 template <typename Y, typename C>
 __global__ void experts_gather_kernel(const Y* __restrict__ y, const int* __restrict__ slot_of, const float* __restrict__ share,
                                       float* __restrict__ out, int width, int top, long long total, const C* __restrict__ common,
-                                      const float* __restrict__ gate) {
+                                      const float* __restrict__ gate, int parts, long long part_stride) {
   grid_dependency_wait();
   allow_dependents();
   const long long item = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -542,7 +516,12 @@ __global__ void experts_gather_kernel(const Y* __restrict__ y, const int* __rest
   const long long t = item / width;
   const int c = (int)(item % width);
   float acc = 0.f;
-  for (int k = 0; k < top; ++k) acc = fmaf(share ? share[t * top + k] : 1.f, to_float<Y>(y[(long long)slot_of[t * top + k] * width + c]), acc);
+  for (int k = 0; k < top; ++k) {
+    const Y* row = y + (long long)slot_of[t * top + k] * width + c;
+    float value = to_float<Y>(row[0]);
+    for (int part = 1; part < parts; ++part) value += to_float<Y>(row[part * part_stride]);
+    acc = fmaf(share ? share[t * top + k] : 1.f, value, acc);
+  }
   if (common != nullptr) acc = fmaf(gate[t], to_float<C>(common[item]), acc);
   out[item] = acc;
 }
@@ -579,23 +558,20 @@ extern "C" int pylon_experts_route(const void* h, long long ld, const float* rou
     PYLON_REFUSE("experts_route: %d groups of which %d are kept for %d of %d experts, %d extra rows", groups, keep, top, experts, extra);
   const RouteScored mode{scored ? 1 : 0, correction, groups, keep, share_eps, normalize, extra, extra_out};
   const int per_token = experts + extra + (scored ? experts + groups : 0);
-  if (num_tokens < 512) {   // a step of few tokens wants many threads a token
-    const size_t smem = (size_t)(4 * 8 + per_token) * sizeof(float);
-    if (dtype == PYLON_DTYPE_F32)
-      launch_dependent(experts_route_block_kernel<float>, dim3((unsigned)num_tokens), dim3(128), smem, stream, (const float*)h, ld, router, bias, chosen, share, width, experts, top, mode);
-    else if (dtype == PYLON_DTYPE_BF16)
-      launch_dependent(experts_route_block_kernel<__nv_bfloat16>, dim3((unsigned)num_tokens), dim3(128), smem, stream, (const __nv_bfloat16*)h, ld, router, bias, chosen, share, width, experts, top, mode);
-    else PYLON_REFUSE("experts_route: unknown dtype %d", dtype);
-  } else {
-    constexpr int warps = 4, side = 4;   // tokens a warp takes side by side (57 us for 2,048 tokens of 2,048 columns and 8 experts; two a warp took 73 us)
-    const dim3 grid((unsigned)((num_tokens + warps * side - 1) / (warps * side)));
-    const size_t smem = (size_t)warps * side * per_token * sizeof(float);
-    if (dtype == PYLON_DTYPE_F32)
-      launch_dependent(experts_route_kernel<float, side>, grid, dim3(warps * 32), smem, stream, (const float*)h, ld, router, bias, chosen, share, width, experts, top, num_tokens, mode);
-    else if (dtype == PYLON_DTYPE_BF16)
-      launch_dependent(experts_route_kernel<__nv_bfloat16, side>, grid, dim3(warps * 32), smem, stream, (const __nv_bfloat16*)h, ld, router, bias, chosen, share, width, experts, top, num_tokens, mode);
-    else PYLON_REFUSE("experts_route: unknown dtype %d", dtype);
-  }
+  const bool few = num_tokens < 512;   // a step of few tokens: a block each
+  const size_t element = dtype == PYLON_DTYPE_F32 ? 4 : 2;
+  const bool pieces = width % 4 == 0 && ld % 4 == 0 && (uintptr_t)h % (4 * element) == 0 && (uintptr_t)router % 16 == 0;
+#define PYLON_ROUTE(T, TOKENS, V)                                                                                                            \
+  launch_dependent(experts_route_kernel<T, TOKENS, V>, dim3((unsigned)((num_tokens + TOKENS - 1) / TOKENS)), dim3(128),                      \
+                   (size_t)TOKENS * (4 * 8 + per_token) * sizeof(float), stream, (const T*)h, ld, router, bias, chosen, share, width, experts, top, num_tokens, mode)
+#define PYLON_ROUTE_SIZES(T)                                                                                                                 \
+  if (few) { if (pieces) PYLON_ROUTE(T, 1, 4); else PYLON_ROUTE(T, 1, 1); }                                                                  \
+  else { if (pieces) PYLON_ROUTE(T, 4, 4); else PYLON_ROUTE(T, 4, 1); }
+  if (dtype == PYLON_DTYPE_F32) { PYLON_ROUTE_SIZES(float) }
+  else if (dtype == PYLON_DTYPE_BF16) { PYLON_ROUTE_SIZES(__nv_bfloat16) }
+  else PYLON_REFUSE("experts_route: unknown dtype %d", dtype);
+#undef PYLON_ROUTE_SIZES
+#undef PYLON_ROUTE
   PYLON_CHECK_LAUNCH("experts_route");
 }
 
@@ -622,17 +598,22 @@ static void allow_mma_shared_memory() {
 
 // a: [rows, lda] in dtype; w: [experts, (glu ? 2 : 1) * n_out, k] in dtype, contiguous (with glu an expert's gate rows, then its up rows;
 // or, interleaved != 0, alternating in groups of 8); out: [max_tiles * EXPERT_ROWS, n_out], in dtype with glu, else float32.
+// k_parts > 1 (a plain bfloat16 product): k in so many equal parts, out float32 [k_parts, max_tiles * EXPERT_ROWS, n_out] whose sum the product is.
 // glu == 2: no gate, but the activation on the product itself, out in dtype (the first product of an ungated expert).
 extern "C" int pylon_experts_product(const void* a, long long lda, const void* w, const int* source, const int* tile_expert, int gathered,
                                      int divide, void* out, int n_out, int k_size, int max_tiles, int glu, int kind, int interleaved, int dtype,
-                                     const float* slot_share, float limit, float alpha, cudaStream_t stream) {
+                                     const float* slot_share, float limit, float alpha, int k_parts, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
   const int act_out = glu == 2 ? 1 : 0;
   if (act_out) glu = 0;
   if (n_out <= 0 || k_size <= 0 || divide < 1 || kind < 0 || kind > 4 || (kind == 4 && glu && !(limit > 0.f)) || (kind == 4 && act_out)) PYLON_REFUSE("experts_product: n %d, k %d, divide %d, activation %d", n_out, k_size, divide, kind);
   if (max_tiles > 65535) PYLON_REFUSE("experts_product: %d row tiles", max_tiles);
   if (interleaved && (!glu || n_out % 8)) PYLON_REFUSE("experts_product: interleaved rows need a gated product of a multiple of 8 columns, got %d", n_out);
-  const dim3 grid((unsigned)((n_out + 63) / 64), (unsigned)max_tiles);
+  if (k_parts < 1 || k_parts > 16 || (k_parts > 1 && (glu || act_out || dtype != PYLON_DTYPE_BF16 || k_size % (64 * k_parts) || lda % 8 || (uintptr_t)a % 16 || (uintptr_t)w % 16)))
+    PYLON_REFUSE("experts_product: k of %d in %d parts (a plain bfloat16 product over whole steps of 64 only)", k_size, k_parts);
+  const dim3 grid((unsigned)((n_out + 63) / 64), (unsigned)max_tiles, (unsigned)k_parts);
+  const int k_each = k_size / k_parts;
+  const long long part_stride = (long long)max_tiles * EXPERT_ROWS * n_out;
   if (dtype == PYLON_DTYPE_F32) {
     if (glu) launch_dependent(experts_product_kernel<float, true>, grid, dim3(256), 0, stream, (const float*)a, lda, (const float*)w, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
     else launch_dependent(experts_product_kernel<float, false>, grid, dim3(256), 0, stream, (const float*)a, lda, (const float*)w, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
@@ -643,10 +624,10 @@ extern "C" int pylon_experts_product(const void* a, long long lda, const void* w
     if (vectors) {
       if (glu) {
         allow_mma_shared_memory<true>();
-        launch_dependent(experts_product_mma_kernel<true>, grid, dim3(128), mma_shared_bytes(true), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
+        launch_dependent(experts_product_mma_kernel<true>, grid, dim3(128), mma_shared_bytes(true), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha, k_each, part_stride);
       } else {
         allow_mma_shared_memory<false>();
-        launch_dependent(experts_product_mma_kernel<false>, grid, dim3(128), mma_shared_bytes(false), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
+        launch_dependent(experts_product_mma_kernel<false>, grid, dim3(128), mma_shared_bytes(false), stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha, k_each, part_stride);
       }
     } else {
       if (glu) launch_dependent(experts_product_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, stream, ab, lda, wb, source, tile_expert, gathered, divide, out, n_out, k_size, kind, interleaved, act_out, slot_share, limit, alpha);
@@ -670,16 +651,18 @@ extern "C" int pylon_experts_sort_rows(const void* h, long long ld, const int* s
   PYLON_CHECK_LAUNCH("experts_sort_rows");
 }
 
+// parts > 1: y is float32 [parts, slots, width], the rows' partial sums.
 // y: [slots, width] in float32 (y_dtype PYLON_DTYPE_F32) or bfloat16; out float32 [num_tokens, width].
 // common ([num_tokens, width] in common_dtype) and gate (float32 [num_tokens]), both or neither: out += gate[t] * common[t].
 extern "C" int pylon_experts_gather(const void* y, const int* slot_of, const float* share, float* out, int num_tokens, int width, int top, int y_dtype,
-                                    const void* common, const float* gate, int common_dtype, cudaStream_t stream) {
+                                    const void* common, const float* gate, int common_dtype, int parts, long long slots, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
+  if (parts < 1 || (parts > 1 && (y_dtype != PYLON_DTYPE_F32 || slots < 1))) PYLON_REFUSE("experts_gather: %d parts", parts);
   if ((common == nullptr) != (gate == nullptr)) PYLON_REFUSE("experts_gather: a common expert's output and its gate go together");
   const long long total = (long long)num_tokens * width;
   const dim3 grid((unsigned)((total + 255) / 256));
   const bool common_f32 = common == nullptr || common_dtype == PYLON_DTYPE_F32;
-#define PYLON_GATHER(Y, C) launch_dependent(experts_gather_kernel<Y, C>, grid, dim3(256), 0, stream, (const Y*)y, slot_of, share, out, width, top, total, (const C*)common, gate)
+#define PYLON_GATHER(Y, C) launch_dependent(experts_gather_kernel<Y, C>, grid, dim3(256), 0, stream, (const Y*)y, slot_of, share, out, width, top, total, (const C*)common, gate, parts, slots * width)
   if (y_dtype == PYLON_DTYPE_F32) { if (common_f32) PYLON_GATHER(float, float); else PYLON_GATHER(float, __nv_bfloat16); }
   else if (y_dtype == PYLON_DTYPE_BF16) { if (common_f32) PYLON_GATHER(__nv_bfloat16, float); else PYLON_GATHER(__nv_bfloat16, __nv_bfloat16); }
   else PYLON_REFUSE("experts_gather: unknown dtype %d", y_dtype);

@@ -13,26 +13,47 @@
 //
 //   min_gru_walk      a thread per request row and V channels walks the row's tokens: steps of a few tokens a row
 //   min_gru_cluster   prompt portions.  The state enters linearly, so a piece of the row walked from S = 0 gives its own share B, and
-//                     the product A of its (1 - z) is the factor on what enters it: S_out = A S_in + B.  A thread-block cluster takes
-//                     a row's 32 V channels; a warp takes TOKENS neighbouring tokens of them, a block 8 neighbouring warps' pieces,
-//                     the cluster its blocks' pieces one after the other.  Every thread reads its tokens' gates and candidates once
-//                     and keeps them in registers; pieces meet through shared memory inside the block and through the other blocks'
-//                     shared memory across it (one cluster barrier per 8 x 8 x TOKENS tokens); then every thread walks its tokens again
-//                     from the state that really enters them.  The row is read once and written once.
+//                     the product A of its (1 - z) is the factor on what enters it: S_out = A S_in + B.  A thread-block cluster takes a
+//                     row's 32 V channels; its warps take equal pieces of the row, in order.  Every warp walks its piece once for A and
+//                     B; the pieces meet through shared memory inside a block and through the other blocks' shared memory across the
+//                     cluster; then every warp walks its piece again (from L2) from the state that really enters it, and writes.  Two
+//                     cluster barriers however long the row is.
 #include "common.cuh"
 
 namespace pylon {
 
-constexpr int GRU_WARPS = 8, GRU_CLUSTER = 8;
+constexpr int GRU_CLUSTER = 8;
+constexpr int GRU_WALKED = 16;   // up to this many tokens a row is walked by one thread per V channels
+constexpr int GRU_AHEAD = 8;     // tokens whose loads are on their way at once
 
-// The hardware's exponential and division (relative errors of a few 2^-23 for the sizes met here) for bfloat16 rows, the library's for
-// float32 rows.
+// The hardware's exponential and reciprocal (relative errors of a few 2^-23) for bfloat16 rows, the library's for float32 rows.
 template <typename T> __device__ __forceinline__ float gru_sigmoid(float x);
 template <> __device__ __forceinline__ float gru_sigmoid<float>(float x) { return 1.f / (1.f + expf(-x)); }
-template <> __device__ __forceinline__ float gru_sigmoid<__nv_bfloat16>(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+template <> __device__ __forceinline__ float gru_sigmoid<__nv_bfloat16>(float x) {
+  float e, y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(e) : "f"(-1.4426950408889634f * x));
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(1.f + e));   // 0 where e is infinite
+  return y;
+}
 
-template <typename T>
-__device__ __forceinline__ float gru_candidate(float u) { return u >= 0.f ? u + 0.5f : gru_sigmoid<T>(u); }
+// Gate and candidate of a token from z + b_z and u.  (Both sides of the candidate are formed: a branch would split the warp at every token.)
+template <typename T> __device__ __forceinline__ void gru_unit(float z, float u, float& gate, float& candidate);
+template <> __device__ __forceinline__ void gru_unit<float>(float z, float u, float& gate, float& candidate) {
+  const float low = gru_sigmoid<float>(u);
+  gate = gru_sigmoid<float>(z);
+  candidate = u >= 0.f ? u + 0.5f : low;
+}
+template <> __device__ __forceinline__ void gru_unit<__nv_bfloat16>(float z, float u, float& gate, float& candidate) {
+  // The two sigmoids share a reciprocal: with a = 1 + e^-z and b = 1 + e^-u, 1 / (a b) times b and times a.  The exponentials stop at
+  // 2^60, so that the product stays in range: a gate below 2^-60 moves nothing.
+  float ez, eu, shared;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(ez) : "f"(-1.4426950408889634f * z));
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(eu) : "f"(-1.4426950408889634f * u));
+  const float a = 1.f + fminf(ez, 1.152921504606847e18f), b = 1.f + fminf(eu, 1.152921504606847e18f);
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(shared) : "f"(a * b));
+  gate = shared * b;
+  candidate = u >= 0.f ? u + 0.5f : shared * a;
+}
 
 template <typename T, int V> struct GruVector;
 template <typename T> struct GruVector<T, 1> { using Type = T; };
@@ -90,7 +111,9 @@ __global__ void __launch_bounds__(128) min_gru_walk_kernel(const GruParams p) {
     gru_load<T, V>(g, from + 2 * (long long)p.channels);
 #pragma unroll
     for (int v = 0; v < V; ++v) {
-      s[v] = fmaf(gru_sigmoid<T>(z[v] + bz[v]), gru_candidate<T>(x[v] + bx[v]) - s[v], s[v]);
+      float gate, candidate;
+      gru_unit<T>(z[v] + bz[v], x[v] + bx[v], gate, candidate);
+      s[v] = fmaf(gate, candidate - s[v], s[v]);
       y[v] = p.factor * s[v] * g[v] * gru_sigmoid<T>(g[v]);
     }
     gru_store<T, V>(to, y);
@@ -108,12 +131,12 @@ __device__ __forceinline__ void gru_cluster_barrier() {
   asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;\n" ::: "memory");
 }
 
-// Grid (channel groups x GRU_CLUSTER, rows).
-template <typename T, int V, int TOKENS>
-__global__ void __launch_bounds__(GRU_WARPS * 32) min_gru_cluster_kernel(const GruParams p) {
+// Grid (channel groups x GRU_CLUSTER, rows); WARPS x 32 threads.
+template <typename T, int V, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32) min_gru_cluster_kernel(const GruParams p) {
   constexpr int GROUP = 32 * V;                                   // channels of a cluster
-  __shared__ float warp_parts[2][GRU_WARPS][2][GROUP];            // [round parity][warp][A, B][channel]: the warps' pieces
-  __shared__ float block_parts[2][GRU_CLUSTER][2][GROUP];         // the cluster's blocks' pieces, sent by the blocks
+  __shared__ float warp_parts[WARPS][2][GROUP];                   // [warp][A, B][channel]: the warps' pieces
+  __shared__ float block_parts[GRU_CLUSTER][2][GROUP];            // the cluster's blocks' pieces, sent by the blocks
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rank = blockIdx.x % GRU_CLUSTER, c0 = blockIdx.x / GRU_CLUSTER * GROUP, row = blockIdx.y;
   const int mine = lane * V, c = c0 + mine;
@@ -122,110 +145,122 @@ __global__ void __launch_bounds__(GRU_WARPS * 32) min_gru_cluster_kernel(const G
   allow_dependents();
   const int first = p.q_start[row], count = p.q_start[row + 1] - first;
   if (count <= 0) return;                                         // the whole cluster leaves: nobody waits for it
-  const bool one_piece = count <= TOKENS;                         // a decoded row in a step that also brings portions: one warp has it all
+  const bool one_piece = count <= GRU_WALKED;                     // a decoded row in a step that also brings portions: one warp has it all
   if (one_piece && (rank > 0 || warp > 0)) return;                // (the same for the whole cluster: no barrier is met)
+  const int each = one_piece ? count : (count + GRU_CLUSTER * WARPS - 1) / (GRU_CLUSTER * WARPS);
+  const int begin = (rank * WARPS + warp) * each, end = begin + each < count ? begin + each : count;   // this warp's tokens (none where the row is used up)
   float* slot = p.state + (long long)p.slots[row] * p.channels + c;
-  float carry[V], bz[V], bx[V];
+  float s[V], bz[V], bx[V];
 #pragma unroll
   for (int v = 0; v < V; ++v) {
-    carry[v] = real ? slot[v] : 0.f;
+    s[v] = real ? slot[v] : 0.f;
     bz[v] = real ? p.bias[c + v] : 0.f;
     bx[v] = real ? p.bias[p.channels + c + v] : 0.f;
   }
-  if (!one_piece) gru_cluster_barrier();   // every block has started (its shared memory may be written) and has read the slot (rank 0 may write it)
-  constexpr int BLOCK_TOKENS = GRU_WARPS * TOKENS, ROUND_TOKENS = GRU_CLUSTER * BLOCK_TOKENS;
-  for (int round = 0, base = 0; base < count; ++round, base += ROUND_TOKENS) {
-    const int parity = round & 1;
-    const int begin = base + rank * BLOCK_TOKENS + warp * TOKENS;   // this warp's tokens: begin .. begin + TOKENS - 1, as far as the row goes
-    const T* from = (const T*)p.proj + (long long)(first + begin) * p.ld + c;
-    float z[TOKENS][V], cand[TOKENS][V], g[TOKENS][V];
-#pragma unroll
-    for (int n = 0; n < TOKENS; ++n) {
-      if (real && begin + n < count) {
-        gru_load<T, V>(z[n], from + n * p.ld);
-        gru_load<T, V>(cand[n], from + n * p.ld + p.channels);
-        gru_load<T, V>(g[n], from + n * p.ld + 2 * (long long)p.channels);
-      } else {
-#pragma unroll
-        for (int v = 0; v < V; ++v) { z[n][v] = -INFINITY; cand[n][v] = 0.f; g[n][v] = 0.f; }   // a gate that is shut: the state passes unchanged
-      }
-    }
+  const T* proj = (const T*)p.proj + (long long)first * p.ld + c;
+  if (!one_piece) {
     float a[V], b[V];
 #pragma unroll
     for (int v = 0; v < V; ++v) { a[v] = 1.f; b[v] = 0.f; }
+    if (real) {
+      auto take = [&](const float (&z)[V], const float (&x)[V]) {
 #pragma unroll
-    for (int n = 0; n < TOKENS; ++n)
+        for (int v = 0; v < V; ++v) {
+          float gate, candidate;
+          gru_unit<T>(z[v] + bz[v], x[v] + bx[v], gate, candidate);
+          b[v] = fmaf(gate, candidate - b[v], b[v]);
+          a[v] = fmaf(-gate, a[v], a[v]);
+        }
+      };
+      int n = begin;
+      const T* from = proj + n * p.ld;
+      for (; n + GRU_AHEAD <= end; n += GRU_AHEAD) {
+        float z[GRU_AHEAD][V], x[GRU_AHEAD][V];
 #pragma unroll
-      for (int v = 0; v < V; ++v) {
-        z[n][v] = gru_sigmoid<T>(z[n][v] + bz[v]);
-        cand[n][v] = gru_candidate<T>(cand[n][v] + bx[v]);
-        b[v] = fmaf(z[n][v], cand[n][v] - b[v], b[v]);
-        a[v] = fmaf(-z[n][v], a[v], a[v]);
+        for (int k = 0; k < GRU_AHEAD; ++k, from += p.ld) {
+          gru_load<T, V>(z[k], from);
+          gru_load<T, V>(x[k], from + p.channels);
+        }
+#pragma unroll
+        for (int k = 0; k < GRU_AHEAD; ++k) take(z[k], x[k]);
       }
-    float s[V];
-    if (one_piece) {
-#pragma unroll
-      for (int v = 0; v < V; ++v) { s[v] = carry[v]; carry[v] = fmaf(a[v], carry[v], b[v]); }
-    } else {
-#pragma unroll
-      for (int v = 0; v < V; ++v) { warp_parts[parity][warp][0][mine + v] = a[v]; warp_parts[parity][warp][1][mine + v] = b[v]; }
-      __syncthreads();
-      // The block's piece, a thread per channel, into every block of the cluster.
-      if (threadIdx.x < GROUP) {
-        float block_a = 1.f, block_b = 0.f;
-#pragma unroll
-        for (int w = 0; w < GRU_WARPS; ++w) {
-          const float wa = warp_parts[parity][w][0][threadIdx.x];
-          block_b = fmaf(wa, block_b, warp_parts[parity][w][1][threadIdx.x]);
-          block_a *= wa;
-        }
-#pragma unroll
-        for (int r = 0; r < GRU_CLUSTER; ++r) {
-          gru_cluster_store(&block_parts[parity][rank][0][threadIdx.x], r, block_a);
-          gru_cluster_store(&block_parts[parity][rank][1][threadIdx.x], r, block_b);
-        }
-      }
-      // One barrier a round: the buffers of this round are written again two rounds on, behind the next round's barrier, which every block
-      // reaches only after it has read them.
-      gru_cluster_barrier();
-#pragma unroll
-      for (int v = 0; v < V; ++v) {
-        float enters = carry[v];
-#pragma unroll
-        for (int r = 0; r < GRU_CLUSTER; ++r) {
-          if (r == rank) s[v] = enters;
-          enters = fmaf(block_parts[parity][r][0][mine + v], enters, block_parts[parity][r][1][mine + v]);
-        }
-        carry[v] = enters;   // what leaves the round
-        for (int w = 0; w < warp; ++w) s[v] = fmaf(warp_parts[parity][w][0][mine + v], s[v], warp_parts[parity][w][1][mine + v]);
+      for (; n < end; ++n, from += p.ld) {
+        float z[V], x[V];
+        gru_load<T, V>(z, from);
+        gru_load<T, V>(x, from + p.channels);
+        take(z, x);
       }
     }
-    T* to = (T*)p.out + (long long)(first + begin) * p.ld_out + c;
 #pragma unroll
-    for (int n = 0; n < TOKENS; ++n) {
-      float y[V];
+    for (int v = 0; v < V; ++v) { warp_parts[warp][0][mine + v] = a[v]; warp_parts[warp][1][mine + v] = b[v]; }
+    gru_cluster_barrier();   // every block has started (its shared memory may be written) and has read the slot (the last one writes it)
+    // The block's piece, a thread per channel and block of the cluster.
+    for (int x = threadIdx.x; x < GROUP * GRU_CLUSTER; x += WARPS * 32) {
+      const int channel = x % GROUP;
+      float block_a = 1.f, block_b = 0.f;
 #pragma unroll
-      for (int v = 0; v < V; ++v) {
-        s[v] = fmaf(z[n][v], cand[n][v] - s[v], s[v]);
-        y[v] = p.factor * s[v] * g[n][v] * gru_sigmoid<T>(g[n][v]);
+      for (int w = 0; w < WARPS; ++w) {
+        const float wa = warp_parts[w][0][channel];
+        block_b = fmaf(wa, block_b, warp_parts[w][1][channel]);
+        block_a *= wa;
       }
-      if (real && begin + n < count) gru_store<T, V>(to + n * p.ld_out, y);
+      gru_cluster_store(&block_parts[rank][0][channel], x / GROUP, block_a);
+      gru_cluster_store(&block_parts[rank][1][channel], x / GROUP, block_b);
+    }
+    gru_cluster_barrier();   // what every block sent is there
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      for (int r = 0; r < rank; ++r) s[v] = fmaf(block_parts[r][0][mine + v], s[v], block_parts[r][1][mine + v]);
+      for (int w = 0; w < warp; ++w) s[v] = fmaf(warp_parts[w][0][mine + v], s[v], warp_parts[w][1][mine + v]);
     }
   }
-  if (rank == 0 && warp == 0 && real) {
+  if (!real || begin >= end) return;
+  auto give = [&](T* to, const float (&z)[V], const float (&x)[V], const float (&g)[V]) {
+    float y[V];
 #pragma unroll
-    for (int v = 0; v < V; ++v) slot[v] = carry[v];
+    for (int v = 0; v < V; ++v) {
+      float gate, candidate;
+      gru_unit<T>(z[v] + bz[v], x[v] + bx[v], gate, candidate);
+      s[v] = fmaf(gate, candidate - s[v], s[v]);
+      y[v] = p.factor * s[v] * g[v] * gru_sigmoid<T>(g[v]);
+    }
+    gru_store<T, V>(to, y);
+  };
+  int n = begin;
+  const T* from = proj + n * p.ld;
+  T* to = (T*)p.out + (long long)(first + n) * p.ld_out + c;
+  for (; n + GRU_AHEAD <= end; n += GRU_AHEAD) {
+    float z[GRU_AHEAD][V], x[GRU_AHEAD][V], g[GRU_AHEAD][V];
+#pragma unroll
+    for (int k = 0; k < GRU_AHEAD; ++k, from += p.ld) {
+      gru_load<T, V>(z[k], from);
+      gru_load<T, V>(x[k], from + p.channels);
+      gru_load<T, V>(g[k], from + 2 * p.channels);
+    }
+#pragma unroll
+    for (int k = 0; k < GRU_AHEAD; ++k, to += p.ld_out) give(to, z[k], x[k], g[k]);
+  }
+  for (; n < end; ++n, from += p.ld, to += p.ld_out) {
+    float z[V], x[V], g[V];
+    gru_load<T, V>(z, from);
+    gru_load<T, V>(x, from + p.channels);
+    gru_load<T, V>(g, from + 2 * p.channels);
+    give(to, z, x, g);
+  }
+  if (end == count) {   // the warp that has walked the row's last token
+#pragma unroll
+    for (int v = 0; v < V; ++v) slot[v] = s[v];
   }
 }
 
 template <typename T, int V>
 static int launch_min_gru(const GruParams& p, int num_rows, int max_q, cudaStream_t stream) {
-  constexpr int TOKENS = V == 2 ? 8 : 16;
-  if (max_q <= TOKENS) {
+  constexpr int WARPS = 16;
+  if (max_q <= GRU_WALKED) {
     launch_dependent(min_gru_walk_kernel<T, V>, dim3((unsigned)((p.channels / V + 127) / 128), (unsigned)num_rows), dim3(128), 0, stream, p);
   } else {
     const int groups = (p.channels + 32 * V - 1) / (32 * V);
-    launch_dependent_cluster(min_gru_cluster_kernel<T, V, TOKENS>, dim3((unsigned)(groups * GRU_CLUSTER), (unsigned)num_rows), dim3(GRU_WARPS * 32), 0, stream, GRU_CLUSTER, p);
+    launch_dependent_cluster(min_gru_cluster_kernel<T, V, WARPS>, dim3((unsigned)(groups * GRU_CLUSTER), (unsigned)num_rows), dim3(WARPS * 32), 0, stream, GRU_CLUSTER, p);
   }
   PYLON_CHECK_LAUNCH("min_gru");
 }

@@ -88,8 +88,10 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
   for (int e = lane; e < width; e += 32) dst[e] = from_float<T>(buf[e]);
 }
 
-// The same for bfloat16 rows without biases whose pairs lie rot / 2 apart, rot a multiple of 16: `lanes` (a power of two) lanes share a
-// head, each with 8 neighbouring elements as one 16-byte piece; the rotation partners of a lane's elements are all in one other lane.
+// The same for bfloat16 rows without biases whose pairs lie rot / 2 apart, rot a multiple of 16.  A block takes one token; `lanes` (a power
+// of two) lanes share a head, each with 8 neighbouring elements as one 16-byte piece; the rotation partners of a lane's elements are all in
+// one other lane.  A lane meets the same elements of several heads, so it reads its angles once, and four heads' pieces are on their
+// way at once.
 __device__ __forceinline__ void unpack_8(float (&x)[8], const uint4& raw) {
   const unsigned words[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
@@ -103,85 +105,94 @@ __device__ __forceinline__ void load_8(float (&x)[8], const float* from) {
   x[0] = low.x; x[1] = low.y; x[2] = low.z; x[3] = low.w; x[4] = high.x; x[5] = high.y; x[6] = high.z; x[7] = high.w;
 }
 
-__global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_vec_kernel(
+constexpr int ROTARY_VEC_MOST = 512;   // threads of a block at most: a step of few tokens gives every head lanes of its own
+
+__global__ void __launch_bounds__(ROTARY_VEC_MOST, 2) qkv_rotate_write_vec_kernel(
     __nv_bfloat16* __restrict__ qkv, long long ld, const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot, int table_positions,
     int norm_mode, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps, const int* __restrict__ positions,
     const int* __restrict__ token_row, const int* __restrict__ block_table, int table_width, int page_size, __nv_bfloat16* __restrict__ k_pages,
-    __nv_bfloat16* __restrict__ v_pages, int num_pages, int nq, int nkv, int d, int dv, int norm_size, int lanes, long long items,
-    int* __restrict__ error_word) {
-  const long long thread = (long long)blockIdx.x * ROTARY_THREADS + threadIdx.x;
-  const long long item = thread / lanes;
-  const int mine = (int)(thread % lanes) * 8;   // this lane's first element
-  const int per_token = nq + 2 * nkv;
-  const bool there = item < items;
-  const int t = there ? (int)(item / per_token) : 0, hh = there ? (int)(item % per_token) : 0;
-  const int row = there ? token_row[t] : -1;    // negative: a padding token, nothing of it is kept
-  const int pos = row >= 0 ? positions[t] : 0;
-  const bool is_q = hh < nq, is_v = hh >= nq + nkv;
-  const int width = is_v ? dv : d, half = rot >> 1;
-  const bool turned = !is_v && mine < rot && pos < table_positions;
-  float c[8], s[8], x[8];
-  if (turned) {   // position, page and angles do not depend on the kernel ahead
+    __nv_bfloat16* __restrict__ v_pages, int num_pages, int nq, int nkv, int d, int dv, int norm_size, int lanes, int* __restrict__ error_word) {
+  constexpr int SIDE = 4;                              // heads of a lane on their way at once
+  const int t = blockIdx.x, row = token_row[t];        // position, page and angles do not depend on the kernel ahead
+  if (row < 0) {                                       // a padding token: nothing of it is kept
+    grid_dependency_wait();                            // a grid must not end before the grid ahead of it has
+    return;
+  }
+  const int mine = (int)(threadIdx.x % lanes) * 8;     // this lane's first element
+  const int group = threadIdx.x / lanes, groups = blockDim.x / lanes;
+  const int pos = positions[t], half = rot >> 1, heads = nq + 2 * nkv;
+  const bool turned = mine < rot && pos < table_positions;
+  float c[8], s[8];
+  if (turned) {
     const size_t angle = (size_t)pos * half + (mine < half ? mine : mine - half);
     load_8(c, cos_table + angle);
     load_8(s, sin_table + angle);
   }
-  int page = -1;
-  if (row >= 0 && !is_q) {
-    const int logical = pos / page_size;
-    page = logical < table_width ? block_table[(size_t)row * table_width + logical] : -1;
-  }
-  const bool live = row >= 0 && mine < width;
-  __nv_bfloat16* src = qkv + (size_t)t * ld + (is_v ? (nq + nkv) * d + (hh - nq - nkv) * dv : hh * d) + mine;
+  const int logical = pos / page_size;
+  const int page = logical < table_width ? block_table[(size_t)row * table_width + logical] : -1;
+  const bool page_there = page >= 0 && page < num_pages;
+  const size_t slot = (size_t)(page_there ? page : 0) * nkv * page_size + pos % page_size;
+  const int lane = threadIdx.x & 31, apart = half >> 3, partner = (mine < half ? lane + apart : lane - apart) & 31;
   grid_dependency_wait();
   allow_dependents();
-  const uint4 raw = live ? *reinterpret_cast<const uint4*>(src) : make_uint4(0u, 0u, 0u, 0u);
-  uint4 result = raw;
-  unpack_8(x, raw);
-  auto unit = [&]() {   // every lane of a warp comes here; a value head keeps what it has
-    float squares = 0.f;
+  for (int h0 = 0; h0 < heads; h0 += SIDE * groups) {  // the same turns for every lane: all of a warp meet the shuffles
+    uint4 raw[SIDE];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) squares = fmaf(x[i], x[i], squares);
-    for (int offset = lanes >> 1; offset > 0; offset >>= 1) squares += __shfl_xor_sync(0xffffffffu, squares, offset);
-    if (is_v || mine >= width) return;
-    const float inv = rsqrtf(squares / norm_size + eps);
-    const float* weight = is_q ? q_weight : k_weight;
-    float w[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
-    if (weight) load_8(w, weight + mine);
+    for (int k = 0; k < SIDE; ++k) {
+      const int hh = h0 + k * groups + group;
+      const bool is_v = hh >= nq + nkv;
+      const bool live = hh < heads && mine < (is_v ? dv : d);
+      raw[k] = live ? *reinterpret_cast<const uint4*>(qkv + (size_t)t * ld + (is_v ? (nq + nkv) * d + (hh - nq - nkv) * dv : hh * d) + mine) : make_uint4(0u, 0u, 0u, 0u);
+    }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) x[i] *= inv * w[i];
-  };
-  if (norm_mode == 1) unit();
-  if (rot > 0) {
-    const int apart = half >> 3;   // lanes between the two elements of a pair
-    const int lane = threadIdx.x & 31, partner = mine < half ? lane + apart : lane - apart;
+    for (int k = 0; k < SIDE; ++k) {
+      if (h0 + k * groups >= heads) break;               // the same for every lane
+      const int hh = h0 + k * groups + group;
+      const bool is_q = hh < nq, is_v = hh >= nq + nkv;
+      float x[8];
+      unpack_8(x, raw[k]);
+      auto unit = [&]() {
+        float squares = 0.f;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const float other = __shfl_sync(0xffffffffu, x[i], partner & 31);
-      if (turned) x[i] = mine < half ? x[i] * c[i] - other * s[i] : x[i] * c[i] + other * s[i];
+        for (int i = 0; i < 8; ++i) squares = fmaf(x[i], x[i], squares);
+        for (int offset = lanes >> 1; offset > 0; offset >>= 1) squares += __shfl_xor_sync(0xffffffffu, squares, offset);
+        const float inv = rsqrtf(squares / norm_size + eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] *= inv;
+        const float* weight = is_q ? q_weight : k_weight;
+        if (weight && mine < d) {
+          float w[8];
+          load_8(w, weight + mine);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) x[i] *= w[i];
+        }
+      };
+      if (norm_mode == 1) unit();
+      if (rot > 0) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float other = __shfl_sync(0xffffffffu, x[i], partner);
+          if (turned) x[i] = mine < half ? x[i] * c[i] - other * s[i] : x[i] * c[i] + other * s[i];
+        }
+      }
+      if (norm_mode == 2) unit();
+      if (hh >= heads || mine >= (is_v ? dv : d)) continue;
+      uint4 result = raw[k];                             // a value stays what it is
+      if (!is_v) {
+        unsigned words[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const __nv_bfloat162 pair = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
+          words[i] = *reinterpret_cast<const unsigned*>(&pair);
+        }
+        result = make_uint4(words[0], words[1], words[2], words[3]);
+      }
+      if (is_q) *reinterpret_cast<uint4*>(qkv + (size_t)t * ld + hh * d + mine) = result;
+      else if (!page_there) { if (mine == 0 && error_word) atomicMax(error_word, PYLON_ERROR_BAD_PAGE); }
+      else if (is_v) *reinterpret_cast<uint4*>(v_pages + (slot + (size_t)(hh - nq - nkv) * page_size) * dv + mine) = result;
+      else *reinterpret_cast<uint4*>(k_pages + (slot + (size_t)(hh - nq) * page_size) * d + mine) = result;
     }
   }
-  if (norm_mode == 2) unit();
-  if (!live) return;
-  if (!is_v) {
-    unsigned words[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const __nv_bfloat162 pair = __floats2bfloat162_rn(x[2 * i], x[2 * i + 1]);
-      words[i] = *reinterpret_cast<const unsigned*>(&pair);
-    }
-    result = make_uint4(words[0], words[1], words[2], words[3]);
-  }
-  if (is_q) {
-    *reinterpret_cast<uint4*>(src) = result;
-    return;
-  }
-  if (page < 0 || page >= num_pages) {
-    if (mine == 0 && error_word) atomicMax(error_word, PYLON_ERROR_BAD_PAGE);
-    return;
-  }
-  const int head = is_v ? hh - nq - nkv : hh - nq;
-  *reinterpret_cast<uint4*>((is_v ? v_pages : k_pages) + (((size_t)page * nkv + head) * page_size + pos % page_size) * width + mine) = result;
 }
 
 // One block per token.  down [T, ld] holds [query latent: q_rank | key/value latent: kv_rank | shared rotated key part: rot_dim].
@@ -273,10 +284,10 @@ extern "C" int pylon_qkv_rotate_write(void* qkv, long long ld, const float* bias
            (uintptr_t)q_weight % 16 == 0 && (uintptr_t)k_weight % 16 == 0) {
     int lanes = 1;
     while (lanes * 8 < (d > dv ? d : dv)) lanes *= 2;
-    const unsigned vector_blocks = (unsigned)((items * lanes + ROTARY_THREADS - 1) / ROTARY_THREADS);
-    launch_dependent(qkv_rotate_write_vec_kernel, dim3(vector_blocks), dim3(ROTARY_THREADS), 0, stream, (__nv_bfloat16*)qkv, ld, cos_table, sin_table, rot,
+    const int threads = num_tokens <= 148 ? ROTARY_VEC_MOST : ROTARY_THREADS;
+    launch_dependent(qkv_rotate_write_vec_kernel, dim3((unsigned)num_tokens), dim3(threads), 0, stream, (__nv_bfloat16*)qkv, ld, cos_table, sin_table, rot,
                      table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row, block_table, table_width, page_size, (__nv_bfloat16*)k_pages,
-                     (__nv_bfloat16*)v_pages, num_pages, nq, nkv, d, dv, norm_size, lanes, items, error_word);
+                     (__nv_bfloat16*)v_pages, num_pages, nq, nkv, d, dv, norm_size, lanes, error_word);
   } else if (dtype == PYLON_DTYPE_BF16)
     qkv_rotate_write_kernel<__nv_bfloat16><<<blocks, ROTARY_THREADS, smem, stream>>>(
         (__nv_bfloat16*)qkv, ld, bias, cos_table, sin_table, rot, layout, table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row,

@@ -9,7 +9,8 @@ from __future__ import annotations
 import ctypes
 import math
 from ctypes import c_float, c_int, c_longlong, c_void_p
-from typing import Optional, Sequence
+from dataclasses import dataclass
+from typing import Optional, Sequence, Union
 
 import torch
 
@@ -208,7 +209,7 @@ _SIGNATURES = {
         "pylon_min_gru": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_int, c_int, c_void_p],
     },
     "output_norm.cu": {
-        "pylon_output_norm": [c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
+        "pylon_output_norm": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
     },
     "matrix_memory.cu": {
         "pylon_matrix_memory_scan": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p,
@@ -229,9 +230,9 @@ _SIGNATURES = {
                                 c_float, c_int, c_int, c_void_p, c_void_p],
         "pylon_experts_plan": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
         "pylon_experts_product": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_int, c_void_p, c_float, c_float, c_void_p],
+                                  c_int, c_void_p, c_float, c_float, c_int, c_void_p],
         "pylon_experts_sort_rows": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-        "pylon_experts_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p],
+        "pylon_experts_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p],
     },
     "gemm_f32.cu": {
         "pylon_gemm_f32_nt": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_void_p],
@@ -433,19 +434,36 @@ def add_rmsnorm(
     return out
 
 
-def output_norm(residual: torch.Tensor, output: torch.Tensor, weight: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
+@dataclass(frozen=True)
+class ScatteredRows:
+    """A block ``[T, width]`` that is not put together yet: token t's row is the sum over k < ``top`` of the rows ``slot_of[t * top + k]``, each
+    times ``share[t, k]`` (None: as they are).  ``rows``: ``[slots, width]`` in the compute dtype, or float32 ``[parts, slots, width]`` partial sums."""
+
+    rows: torch.Tensor
+    slot_of: torch.Tensor
+    top: int
+    share: Optional[torch.Tensor]
+
+
+def output_norm(residual: torch.Tensor, output: Union[torch.Tensor, ScatteredRows], weight: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
     """``residual += rmsnorm(output) * weight`` in float32, in place, for a norm that stands on a sublayer's output: ``[T, width]`` in ``dtype``
-    or float32 partial sums ``[parts, T, width]`` whose sum it is.  Returns the new sum in ``dtype`` (``residual`` itself in float32)."""
-    _need_cuda(residual, output, weight)
+    or float32 partial sums ``[parts, T, width]`` whose sum it is, or :class:`ScatteredRows`.  Returns the new sum in ``dtype`` (``residual`` itself in float32)."""
+    slot_of = share = None
+    top, slots = 1, 0
+    if isinstance(output, ScatteredRows):
+        slot_of, share, top, slots, output = output.slot_of, output.share, output.top, output.rows.shape[-2], output.rows
+        _need(slot_of.dtype == torch.int32 and slot_of.is_contiguous() and slot_of.numel() == residual.shape[0] * top, "output_norm: slot_of must be int32 [T, top]")
+        _need(share is None or (share.dtype == torch.float32 and share.is_contiguous() and share.numel() == slot_of.numel()), "output_norm: share must be float32 [T, top]")
+    _need_cuda(residual, output, weight, slot_of, share)
     _need(residual.dtype == torch.float32 and residual.dim() == 2 and residual.is_contiguous(), "output_norm: residual must be contiguous float32 [T, width]")
     tokens, width = residual.shape
     parts = output.shape[0] if output.dim() == 3 else 0
-    _need(output.shape[-2:] == residual.shape and output.is_contiguous() and output.dtype == (torch.float32 if parts else dtype),
+    _need(output.shape[-2:] == (slots if slot_of is not None else tokens, width) and output.is_contiguous() and output.dtype == (torch.float32 if parts else dtype),
           "output_norm: output must be contiguous [T, width] in the compute dtype or float32 [parts, T, width]")
     _need(weight.dtype == torch.float32 and weight.shape == (width,) and weight.is_contiguous(), "output_norm: weight must be float32 [width]")
     copy = None if dtype == torch.float32 else torch.empty((tokens, width), dtype=dtype, device=residual.device)
     library = _library("output_norm.cu")
-    _check(library, library.pylon_output_norm(_ptr(output), parts, None, 0, 1.0, _ptr(residual), _ptr(copy), _ptr(weight), tokens, width, float(eps), 1,
+    _check(library, library.pylon_output_norm(_ptr(output), parts, None, 0, _ptr(slot_of), _ptr(share), top, slots, 1.0, _ptr(residual), _ptr(copy), _ptr(weight), tokens, width, float(eps), 1,
                                               _dtype_code(dtype), _stream()))
     return residual if copy is None else copy
 
@@ -461,7 +479,7 @@ def embedding_norm(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor,
     residual = torch.empty((tokens, width), dtype=torch.float32, device=table.device)
     copy = None if dtype == torch.float32 else torch.empty((tokens, width), dtype=dtype, device=table.device)
     library = _library("output_norm.cu")
-    _check(library, library.pylon_output_norm(_ptr(table), 0, _ptr(ids), vocab, float(scale), _ptr(residual), _ptr(copy), _ptr(weight), tokens, width, float(eps), 0,
+    _check(library, library.pylon_output_norm(_ptr(table), 0, _ptr(ids), vocab, None, None, 1, 0, float(scale), _ptr(residual), _ptr(copy), _ptr(weight), tokens, width, float(eps), 0,
                                               _dtype_code(dtype), _stream()))
     return residual, residual if copy is None else copy
 
@@ -620,6 +638,18 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
             return linear_tcgen05(x, w)
         return torch.mm(x, w.t())
     return torch.mm(x, w.t(), out_dtype=torch.float32)
+
+
+def linear_stacked(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """:func:`linear` for many weight rows (projections of several readers stacked): a decode step's few rows go to the TMA-fed kernel, whose
+    blocks of 64 weight rows then fill the device by themselves."""
+    m, k = x.shape
+    n = w.shape[0]
+    if (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.is_cuda and m <= STREAM_MAX_ROWS and k >= 1024 and k % 8 == 0 and n % 8 == 0
+            and 2 * n >= 64 * _multiprocessors(x.device) and x.stride(1) == 1 and w.stride(1) == 1 and x.stride(0) % 8 == 0 and w.stride(0) % 8 == 0
+            and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
+        return linear_stream(x, w)
+    return linear(x, w)
 
 
 def _tcgen05_fills_the_sms(m: int, n: int, sms: int) -> bool:
@@ -1627,7 +1657,7 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
                    top: int, activation: str = "silu", interleaved: bool = False, gated: bool = True, routing: str = "softmax",
                    correction: Optional[torch.Tensor] = None, groups: int = 0, groups_keep: int = 0, share_eps: float = 0.0,
                    common_up: Optional[torch.Tensor] = None, common_down: Optional[torch.Tensor] = None, share_normalized: bool = True,
-                   weigh: str = "output", limit: Optional[float] = None, alpha: float = 1.702) -> torch.Tensor:
+                   weigh: str = "output", limit: Optional[float] = None, alpha: float = 1.702, scattered: bool = False) -> Union[torch.Tensor, "ScatteredRows"]:
     """``sum over a token's top experts e of share_e * W_down,e (act(W_gate,e h) * (W_up,e h))`` (``csrc/experts.cu``).
 
     ``h [T, width]``; ``router`` float32 ``[experts, width]`` and ``router_bias`` float32 ``[experts]`` (or None): the logits are
@@ -1644,7 +1674,8 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
 
     ``share_normalized=False``: the shares are the chosen experts' scores as they are.  ``weigh="input"`` (gated experts): the result is
     ``sum expert_e(share_e * h)``; an expert's first product is linear in its input, so the share multiplies its float32 sums.
-    ``activation="clamped"`` with a ``limit``: the clamped gated unit of :func:`swiglu`.
+    ``activation="clamped"`` with a ``limit``: the clamped gated unit of :func:`swiglu`.  ``scattered=True`` (no common expert): the experts'
+    rows are handed on where they lie, as :class:`ScatteredRows`, for a reader that adds them up itself.
 
     The tokens are sorted by expert on the device.  A step of few tokens runs the experts' products from row tiles of 32 slots that
     gather their rows themselves (``mma.sync``, bound by the matrices coming from memory); a bfloat16 step with about half a
@@ -1673,6 +1704,7 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     _need(1 <= top <= experts, f"expert_mixture: top {top} of {experts} experts")
     _need(not interleaved or (gated and inner % 8 == 0), "expert_mixture: interleaved rows need a gated unit of an inner width that is a multiple of 8")
     _need((common_up is None) == (common_down is None), "expert_mixture: a common expert has both its matrices")
+    _need(not scattered or common_up is None, "expert_mixture: rows cannot stay scattered beside a common expert")
     library = _library("experts.cu")
     pairs = tokens * top
     grouped = ((not gated or (interleaved and activation in ("silu", "clamped"))) and h.dtype == torch.bfloat16 and pairs * 2 >= EXPERT_TILE_ROWS * experts and width % 8 == 0
@@ -1699,7 +1731,6 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     if extra:   # the expert of every token: two plain products around the activation
         common = linear(activation_in_place(linear(h, common_up), activation), common_down)
         common_code = _dtype_code(common.dtype)
-    out = torch.empty((1, tokens, width), dtype=torch.float32, device=device)
     if grouped:
         product = _library("gemm_tcgen05.cu")
         error, sms = _ptr(tcgen05_error_word(device)), _multiprocessors(device)
@@ -1713,18 +1744,35 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
         y = torch.empty((max_slots, width), dtype=h.dtype, device=device)
         _check(product, product.pylon_gemm_tcgen05_grouped(_ptr(act), _ptr(w_down), _ptr(y), max_slots, width, inner, inner, inner, width, 0, 0.0, 1.0, None,
                                                            _ptr(tile_expert), experts, error, sms, _stream()))
+        if scattered:
+            return ScatteredRows(y, slot_of, top, out_share)
+        out = torch.empty((1, tokens, width), dtype=torch.float32, device=device)
         _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, top, code, _ptr(common), _ptr(common_gate),
-                                                     common_code, _stream()))
+                                                     common_code, 1, 0, _stream()))
         return out
     act = torch.empty((max_slots, inner), dtype=h.dtype, device=device)
     _check(library, library.pylon_experts_product(_ptr(h), h.stride(0), _ptr(w_gate_up), _ptr(source), _ptr(tile_expert), 1, top, _ptr(act), inner, width,
-                                                  max_tiles, 1 if gated else 2, kind, int(interleaved), code, _ptr(slot_share), limit, float(alpha), _stream()))
-    y = torch.empty((max_slots, width), dtype=torch.float32, device=device)
+                                                  max_tiles, 1 if gated else 2, kind, int(interleaved), code, _ptr(slot_share), limit, float(alpha), 1, _stream()))
+    parts = _expert_parts(experts, width, inner, _multiprocessors(device)) if h.dtype == torch.bfloat16 else 1
+    y = torch.empty((parts, max_slots, width), dtype=torch.float32, device=device)
     _check(library, library.pylon_experts_product(_ptr(act), inner, _ptr(w_down), _ptr(source), _ptr(tile_expert), 0, 1, _ptr(y), width, inner,
-                                                  max_tiles, 0, kind, 0, code, None, 0.0, 1.0, _stream()))
+                                                  max_tiles, 0, kind, 0, code, None, 0.0, 1.0, parts, _stream()))
+    if scattered:
+        return ScatteredRows(y, slot_of, top, out_share)
+    out = torch.empty((1, tokens, width), dtype=torch.float32, device=device)
     _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, top, _dtype_code(torch.float32), _ptr(common),
-                                                 _ptr(common_gate), common_code, _stream()))
+                                                 _ptr(common_gate), common_code, parts, max_slots, _stream()))
     return out
+
+
+def _expert_parts(experts: int, columns: int, k: int, sms: int) -> int:
+    """In how many parts of k the second product of a step of few tokens is cut: enough that its blocks (64 columns of one expert each) give every SM
+    about four, in whole steps of 64 of at least 512.  By the sizes alone, so that a token's sums do not depend on the step."""
+    blocks = experts * -(-columns // 64)
+    parts = 1
+    while parts < 4 and blocks * parts < 4 * sms and k % (128 * parts) == 0 and k // (2 * parts) >= 512:
+        parts *= 2
+    return parts
 
 
 # ---------------------------------------------------------------------------------------

@@ -251,7 +251,7 @@ class GroupedQueryAttention(Mixer):
     def forward(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> torch.Tensor:
         if self.weighting == "sigmoid":
             context = torch.empty((h.shape[0], self.output_columns.shape[1]), dtype=h.dtype, device=h.device)
-            self.middle(ops.linear(h, self.input_rows), step, cache, context, 1.0)
+            self.middle(ops.linear_stacked(h, self.input_rows), step, cache, context, 1.0)
             return ops.linear_for_residual(context, self.output_columns)
         if self.rotary_general:
             return self._forward_rotary_general(h, step, cache)

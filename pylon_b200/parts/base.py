@@ -205,7 +205,7 @@ class Norm(Part):
 
     def join(self, stream: "ResidualStream", output: torch.Tensor) -> None:
         """For a norm that stands on a sublayer's output: ``stream += norm(output)``.  ``output`` comes in either form of a
-        delta (see :class:`ResidualStream`)."""
+        delta (see :class:`ResidualStream`), or as :class:`ops.ScatteredRows`."""
         raise NotImplementedError(f"{type(self).__name__} is not built to stand on a sublayer's output")
 
     def enter(self, token_ids: torch.Tensor, table: torch.Tensor, scale: float) -> "ResidualStream":
@@ -259,6 +259,10 @@ class FeedForward(Part):
     def forward(self, h: torch.Tensor, step: StepView) -> torch.Tensor:
         """Returns the delta for the residual stream (see :class:`ResidualStream`)."""
         raise NotImplementedError
+
+    def forward_scattered(self, h: torch.Tensor, step: StepView):
+        """The same for a reader that can put the output together itself (:meth:`Norm.join`): may be :class:`ops.ScatteredRows`."""
+        return self.forward(h, step)
 
 
 class Block(Part):

@@ -214,4 +214,4 @@ class OutputNormBlock(Block):
     def forward(self, stream: ResidualStream, step: StepView, cache: LayerCache) -> None:
         self.mixer_norm.join(stream, self.mixer.forward(stream.read(self.dtype), step, cache))
         if self.feed_forward is not None:
-            self.ffn_norm.join(stream, self.feed_forward.forward(stream.read(self.dtype), step))
+            self.ffn_norm.join(stream, self.feed_forward.forward_scattered(stream.read(self.dtype), step))

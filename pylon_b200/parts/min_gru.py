@@ -55,7 +55,7 @@ class MinGRU(Mixer):
 
     def forward(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> torch.Tensor:
         read = torch.empty((h.shape[0], self.channels), dtype=h.dtype, device=h.device)
-        self.middle(ops.linear(h, self.input_rows), step, cache, read, 1.0)
+        self.middle(ops.linear_stacked(h, self.input_rows), step, cache, read, 1.0)
         return ops.linear_for_residual(read, self.output_columns)
 
     def middle(self, proj: torch.Tensor, step: StepView, cache: LayerCache, out: torch.Tensor, factor: float) -> None:

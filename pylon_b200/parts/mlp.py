@@ -210,8 +210,11 @@ class ExpertMixture(FeedForward):
         shared = 0 if self.w_shared_up is None else self.w_shared_up.numel() + self.w_shared_down.numel()
         return (self.w_gate_up.numel() + self.w_down.numel() + shared) * self.w_down.element_size() + self.w_router.numel() * 4
 
-    def forward(self, h: torch.Tensor, step: StepView) -> torch.Tensor:
+    def forward(self, h: torch.Tensor, step: StepView, scattered: bool = False) -> torch.Tensor:
         return ops.expert_mixture(h, self.w_router, self.b_router, self.w_gate_up, self.w_down, self.top, self.activation, self.interleaved,
                                   gated=self.gated, routing=self.routing, correction=self.correction, groups=self.groups, groups_keep=self.groups_keep,
                                   share_eps=self.share_eps, common_up=self.w_shared_up, common_down=self.w_shared_down, share_normalized=self.share_normalized,
-                                  weigh=self.weigh, limit=self.limit, alpha=self.alpha)
+                                  weigh=self.weigh, limit=self.limit, alpha=self.alpha, scattered=scattered)
+
+    def forward_scattered(self, h: torch.Tensor, step: StepView):
+        return self.forward(h, step, scattered=self.shared_intermediate is None)

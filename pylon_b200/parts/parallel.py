@@ -113,7 +113,7 @@ class WeightedMixers(ParallelMixers):
 
     def forward(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> torch.Tensor:
         if self.w_in is not None:
-            proj = ops.linear(h, self.w_in)
+            proj = ops.linear_stacked(h, self.w_in)
             # columns between the slices meet zeros of the last product's matrix, so they must hold numbers
             middle = (torch.empty if self.filled else torch.zeros)((h.shape[0], self.w_out.shape[1]), dtype=h.dtype, device=h.device)
             for mixer, scale, into, out_of in zip(self.mixers, self.scales, self.in_slices, self.out_slices):

@@ -534,8 +534,29 @@ def test_the_norm_on_an_output_and_on_the_embedding(width, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("width,top,parts,shared", [(30, 1, 0, False), (72, 3, 0, True), (200, 2, 2, False), (2048, 2, 5, True)])
+def test_the_norm_on_rows_that_lie_in_slots(width, top, parts, shared, dtype):
+    """An output that is still scattered: the sum of ``top`` rows a token, each times its share, as they lie or as partial sums."""
+    from pylon_b200.kernels import ops
+
+    g = torch.Generator().manual_seed(width)
+    tokens, slots, eps = 7, 40, 1e-4
+    rows = torch.randn(parts, slots, width, generator=g) if parts else torch.randn(slots, width, generator=g).to(dtype)
+    slot_of = torch.randperm(slots, generator=g)[: tokens * top].to(torch.int32)
+    share = torch.rand(tokens, top, generator=g) if shared else None
+    weight, residual = torch.rand(width, generator=g) + 0.5, torch.randn(tokens, width, generator=g)
+    whole = (rows.double().sum(dim=0) if parts else rows.double())[slot_of.long()].view(tokens, top, width)
+    whole = (whole * share.double()[..., None] if shared else whole).sum(dim=1)
+    want = plain.add_normed(residual.double(), whole, weight.double(), eps)
+    held = on(residual.clone())
+    copy = ops.output_norm(held, ops.ScatteredRows(on(rows), on(slot_of), top, None if share is None else on(share)), on(weight), eps, dtype)
+    torch.testing.assert_close(held.double().cpu(), want, rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(copy.double().cpu(), want, **(dict(rtol=2e-2, atol=2e-2) if dtype == torch.bfloat16 else dict(rtol=1e-5, atol=1e-5)))
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("width,ff,experts,top,tokens", [(40, 12, 3, 1, 1), (56, 20, 6, 6, 7), (48, 24, 12, 4, 150), (128, 64, 33, 3, 70), (64, 40, 2, 1, 40),
-                                                         (256, 136, 4, 2, 700), (384, 256, 3, 1, 600), (72, 9, 5, 2, 90)])
+                                                         (256, 136, 4, 2, 700), (384, 256, 3, 1, 600), (72, 9, 5, 2, 90), (64, 1024, 3, 2, 20)])
 def test_the_mixture_whose_scores_weigh_the_experts_input(width, ff, experts, top, tokens, dtype):
     """Sigmoid scores in 32-bit as they are, the clamped unit on both sides of its limits, an expert's input times its score: one token, few and
     many, tiles that are partly filled, an inner width that is no whole piece; two shapes have enough tokens an expert for the grouped
@@ -567,6 +588,10 @@ def test_the_mixture_whose_scores_weigh_the_experts_input(width, ff, experts, to
     spread = float(want.std())
     tolerance = 0.06 * spread if dtype == torch.bfloat16 else 1e-4 * spread
     assert float((got - want)[sure].abs().max()) <= tolerance
+    # the rows where the experts left them, for a reader that adds them up itself
+    loose = part.forward_scattered(on(h), step_view((tokens,), (0,), dtype))
+    rows = (loose.rows.sum(dim=0) if loose.rows.dim() == 3 else loose.rows).double().cpu()[loose.slot_of.long().cpu()].view(tokens, top, width).sum(dim=1)
+    torch.testing.assert_close(rows, got, rtol=1e-5, atol=1e-5)
     # the same tokens in another order and among others: a token's result does not depend on its place in the step
     order = torch.randperm(tokens, generator=g)
     both = torch.cat([h[order], rand(5, width).to(dtype)])
