@@ -56,8 +56,8 @@ CONFIGS = {
         layer((3, 3, 24, 8, 0.2), (24, 10000.0, None), 33, (1.1, 0.6)),
         layer((1, 1, 8, 8, 0.5), None, 16, (0.5, 1.0), dense(40, 1.5)),
     ], logit_scale=0.7),
-    # heads of sizes that are no multiples of 8, one expert a token, experts of an odd width; pages of 4
-    "odd": model(61, 40, [
+    # heads of sizes that are no multiples of 8, one expert a token, experts and a stream of an odd width; pages of 4
+    "odd": model(61, 45, [
         layer((4, 1, 10, 6, 0.4), (6, 50.0, YARN), 7, (1.3, 0.9), moe(9, 3, 1, 1.0)),
         layer((2, 2, 12, 20, 0.3), (4, 300.0, {"factor": 2.0, "original": 64, "fast": 16.0, "slow": 2.0}), 20, (0.8, -0.5), dense(12, 3.0)),
     ], eps=1e-4, logit_scale=1.0),
