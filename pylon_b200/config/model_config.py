@@ -1095,3 +1095,208 @@ class ZabusunConfig:
         if self.eos_token_ids:
             data["eos_token_id"] = list(self.eos_token_ids)
         return data
+
+
+# ---------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class PinedraAttention:
+    """One Pinedra mixer's sizes and constants.  Its kind says what it does: ``attention`` (values are the projected keys, q and k normed
+    over their whole rows, biases on q, k and the output, every output element gated), ``attention_2`` (q and k normed per head, queries
+    times a factor that grows with their position, a slope per head on the distance, one added to the softmax's denominator, every output
+    element gated) or ``attention_3`` (biases on q, k and v, partly rotated heads, soft-capped scores inside chunks of positions, every
+    head gated)."""
+
+    kind: str
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    temperature: Optional[tuple[float, float]] = None   # attention_2: (coef, every)
+    rot: Optional[RotarySpec] = None                    # attention_3
+    softcap: Optional[float] = None                     # attention_3; None: scores as they are
+    chunk: Optional[int] = None                         # attention_3; None: every earlier key
+
+    KINDS: ClassVar[tuple[str, ...]] = ("attention", "attention_2", "attention_3")
+
+    @classmethod
+    def from_dict(cls, kind: str, data: Mapping[str, Any], where: str) -> "PinedraAttention":
+        if kind not in cls.KINDS:
+            raise ConfigError(f"{where}: unknown type {kind!r} ({', '.join(cls.KINDS)})")
+        heads, kv_heads, dim, vdim = (_positive_int(data, key) for key in ("heads", "kv_heads", "dim", "vdim"))
+        if heads % kv_heads:
+            raise ConfigError(f"{where}: {heads} heads cannot be grouped over {kv_heads} kv_heads")
+        scale = _number(data, "scale")
+        if not scale > 0:
+            raise ConfigError(f"{where}: scale must be positive")
+        if kind == "attention":
+            if vdim != dim:
+                raise ConfigError(f"{where}: the values are the keys, so vdim must be dim ({dim}), got {vdim}")
+            return cls(kind, heads, kv_heads, dim, vdim, scale)
+        if kind == "attention_2":
+            temperature = None
+            if data.get("q_temp") is not None:
+                temperature = (_number(_mapping(data, "q_temp"), "coef"), _number(_mapping(data, "q_temp"), "every"))
+                if not temperature[1] > 0:
+                    raise ConfigError(f"{where}: q_temp.every must be positive")
+            return cls(kind, heads, kv_heads, dim, vdim, scale, temperature=temperature)
+        rot = softcap = chunk = None
+        if data.get("rot") is not None:
+            rot = RotarySpec.from_dict(_mapping(data, "rot"), where, ())
+            if rot.scaling is not None:
+                raise ConfigError(f"{where}: the frequencies of the rotation are not scaled in this design")
+            if rot.dims > dim:
+                raise ConfigError(f"{where}: rot.dims {rot.dims} exceeds the head's dim {dim}")
+        if data.get("softcap") is not None:
+            softcap = _number(data, "softcap")
+            if not softcap > 0:
+                raise ConfigError(f"{where}: softcap must be positive")
+        if data.get("mask") is not None:
+            chunk = _positive_int(_mapping(data, "mask"), "size")
+        return cls(kind, heads, kv_heads, dim, vdim, scale, rot=rot, softcap=softcap, chunk=chunk)
+
+    def to_dict(self) -> dict[str, Any]:
+        data: dict[str, Any] = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale}
+        if self.temperature is not None:
+            data["q_temp"] = {"coef": self.temperature[0], "every": self.temperature[1]}
+        if self.rot is not None:
+            data["rot"] = {"dims": self.rot.dims, "base": self.rot.base}
+        if self.softcap is not None:
+            data["softcap"] = self.softcap
+        if self.chunk is not None:
+            data["mask"] = {"size": self.chunk}
+        return data
+
+
+@dataclass(frozen=True)
+class PinedraFeedForward:
+    """A mixture of ``experts`` gated units of inner width ``ff`` beside ``identity`` experts that hand their input back; a token uses
+    ``top`` of them, chosen by softmax scores with a correction among the ``groups_keep`` best of ``groups`` groups and weighted by the scores
+    times ``scale``; plus (``shared_ff``) one gated unit for every token."""
+
+    ff: int
+    experts: int
+    top: int
+    scale: float = 1.0
+    identity: int = 0
+    groups: Optional[int] = None
+    groups_keep: Optional[int] = None
+    shared_ff: Optional[int] = None
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], where: str) -> "PinedraFeedForward":
+        kind = _require(data, "kind", str)
+        if kind != "moe":
+            raise ConfigError(f"{where}: unknown feed-forward kind {kind!r} (moe)")
+        router = _mapping(data, "router")
+        experts, top = _positive_int(router, "experts"), _positive_int(router, "top")
+        identity = 0 if router.get("identity") is None else _require(router, "identity", int)
+        if identity < 0:
+            raise ConfigError(f"{where}: router.identity must not be negative")
+        choices, groups, keep = experts + identity, None, None
+        if router.get("groups") is not None:
+            groups, keep = _positive_int(_mapping(router, "groups"), "count"), _positive_int(_mapping(router, "groups"), "keep")
+            if choices % groups or keep > groups:
+                raise ConfigError(f"{where}: {choices} experts in {groups} groups of which {keep} are kept")
+        if top > (choices if groups is None else keep * (choices // groups)):
+            raise ConfigError(f"{where}: a token cannot use {top} of the experts it may choose from")
+        shared = data.get("shared")
+        return cls(_positive_int(_mapping(data, "expert"), "ff"), experts, top, 1.0 if router.get("scale") is None else _number(router, "scale"), identity,
+                   groups, keep, None if shared is None else _positive_int(_mapping(data, "shared"), "ff"))
+
+    def to_dict(self) -> dict[str, Any]:
+        router: dict[str, Any] = {"experts": self.experts, "top": self.top, "scale": self.scale, "identity": self.identity}
+        if self.groups is not None:
+            router["groups"] = {"count": self.groups, "keep": self.groups_keep}
+        data: dict[str, Any] = {"kind": "moe", "expert": {"ff": self.ff}, "router": router}
+        if self.shared_ff is not None:
+            data["shared"] = {"ff": self.shared_ff}
+        return data
+
+
+@dataclass(frozen=True)
+class PinedraLayer:
+    """One layer: its mixer and its feed-forward (or none), side by side behind one norm."""
+
+    mixer: PinedraAttention
+    mlp: Optional[PinedraFeedForward] = None
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any], index: int) -> "PinedraLayer":
+        where, mlp = f"layer {index}", data.get("mlp")
+        if mlp is not None and not isinstance(mlp, dict):
+            raise ConfigError(f"{where}: 'mlp' must be an object or null")
+        return cls(PinedraAttention.from_dict(_require(data, "type", str), _mapping(data, "mixer"), where),
+                   None if mlp is None else PinedraFeedForward.from_dict(mlp, where))
+
+    def to_dict(self) -> dict[str, Any]:
+        return {"type": self.mixer.kind, "mixer": self.mixer.to_dict(), "mlp": None if self.mlp is None else self.mlp.to_dict()}
+
+
+@dataclass(frozen=True)
+class PinedraConfig:
+    """Pinedra: a decoder whose layers each read one RMS norm (its weight a single number) and add mixer and feed-forward to the stream
+    side by side.  The mixers are three kinds of gated grouped-query attention in an order the configuration lists; the feed-forward is a
+    mixture of experts, some of which hand their input back, with a shared expert.  The embedding is scaled, the head is a tensor of its
+    own, and a span of layers ``loop`` = (start, stop, times) runs several times in a row, the embedding added again before every pass but
+    the first, each pass with caches of its own.
+
+    ``config.json`` names the model by ``"architecture": "Pinedra"``.  Field names follow its keys.
+    """
+
+    architecture: ClassVar[str] = "Pinedra"
+
+    vocab: int
+    width: int
+    layers: tuple[PinedraLayer, ...]
+    norm_eps: float
+    embedding_scale: float = 1.0
+    loop: Optional[tuple[int, int, int]] = None
+    eos_token_ids: tuple[int, ...] = field(default_factory=tuple)
+
+    def __post_init__(self) -> None:
+        if not self.layers:
+            raise ConfigError("a model needs at least one layer")
+        if not self.norm_eps > 0:
+            raise ConfigError(f"norm.eps must be positive, got {self.norm_eps}")
+        if self.loop is not None:
+            start, stop, times = self.loop
+            if not 0 <= start <= stop <= len(self.layers) or times < 1:
+                raise ConfigError(f"loop {start} .. {stop} x {times} does not fit {len(self.layers)} layers")
+
+    @classmethod
+    def from_dict(cls, data: Mapping[str, Any]) -> "PinedraConfig":
+        layers, eos, loop = _require(data, "layers", list), data.get("eos_token_id"), data.get("loop")
+        if loop is not None and not isinstance(loop, dict):
+            raise ConfigError("'loop' must be an object or null")
+        return cls(
+            vocab=_positive_int(data, "vocab"),
+            width=_positive_int(data, "width"),
+            layers=tuple(PinedraLayer.from_dict(layer, index) for index, layer in enumerate(layers)),
+            norm_eps=_number(_mapping(data, "norm"), "eps"),
+            embedding_scale=1.0 if data.get("embedding") is None else _number(_mapping(data, "embedding"), "scale"),
+            loop=None if loop is None else (int(_require(loop, "start", int)), int(_require(loop, "stop", int)), _positive_int(loop, "times")),
+            eos_token_ids=() if eos is None else ((eos,) if isinstance(eos, int) else tuple(int(x) for x in eos)),
+        )
+
+    def to_dict(self) -> dict[str, Any]:
+        data: dict[str, Any] = {
+            "architecture": self.architecture, "vocab": self.vocab, "width": self.width, "embedding": {"scale": self.embedding_scale},
+            "layers": [layer.to_dict() for layer in self.layers], "norm": {"eps": self.norm_eps},
+        }
+        if self.loop is not None:
+            data["loop"] = {"start": self.loop[0], "stop": self.loop[1], "times": self.loop[2]}
+        if self.eos_token_ids:
+            data["eos_token_id"] = list(self.eos_token_ids)
+        return data
+
+    def run_order(self) -> list[tuple[int, bool]]:
+        """(layer, whether the embedding output is added right before it) of every layer run: the layers before the loop, the loop's
+        span ``times`` times, the rest."""
+        if self.loop is None:
+            return [(index, False) for index in range(len(self.layers))]
+        start, stop, times = self.loop
+        order = [(index, False) for index in range(start)]
+        for turn in range(times):
+            order += [(index, turn > 0 and index == start) for index in range(start, stop)]
+        return order + [(index, False) for index in range(stop, len(self.layers))]

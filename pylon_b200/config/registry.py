@@ -11,7 +11,7 @@ from dataclasses import dataclass
 from pathlib import Path
 from typing import Any, Callable, Mapping, Optional
 
-from pylon_b200.config.model_config import ConfigError, FikeraxConfig, Qwen3Config, RirusunConfig, VopepelConfig, ZabusunConfig, ZemavikConfig
+from pylon_b200.config.model_config import ConfigError, FikeraxConfig, PinedraConfig, Qwen3Config, RirusunConfig, VopepelConfig, ZabusunConfig, ZemavikConfig
 from pylon_b200.parts.spec import ModelSpec
 
 
@@ -74,6 +74,9 @@ def _register_builtin() -> None:
     from pylon_b200.models.zabusun import zabusun_spec
 
     register_architecture(ZabusunConfig.architecture, ZabusunConfig, zabusun_spec)
+    from pylon_b200.models.pinedra import pinedra_spec
+
+    register_architecture(PinedraConfig.architecture, PinedraConfig, pinedra_spec)
 
 
 _register_builtin()

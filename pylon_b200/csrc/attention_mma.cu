@@ -22,6 +22,11 @@
 // nothing to rescale, and partial results simply add up.  A weight enters the weighted sum as two bfloat16 numbers, the rounded
 // weight and what the rounding dropped, so that it counts with 16 of its 24 bits: a long row adds up many small weights, and no
 // sum of weights divides their common rounding out.  Head h of token t may be multiplied by sigmoid(gate[t, h]) as it is written.
+//
+// Built with -DPYLON_SOFTMAX_OPTIONS=1 the softmax has what few designs ask for: a slope per head on the distance (the score of the key d
+// positions back loses slopes[h] d), a sink per head (the denominator also holds exp(sinks[h]); met by the part of a row's keys that comes
+// first in the tiled kernel, and by one segment of a pair in the decode kernel), outputs times a factor and the sigmoid of a gate per head or per
+// element, rows of the output in a wider row; and its weights enter the weighted sum as two bfloat16 numbers, as the sigmoid ones do.
 #include "common.cuh"
 
 #include <cuda.h>
@@ -34,17 +39,25 @@
 #ifndef PYLON_SIGMOID_WEIGHTS
 #define PYLON_SIGMOID_WEIGHTS 0
 #endif
+#ifndef PYLON_SOFTMAX_OPTIONS
+#define PYLON_SOFTMAX_OPTIONS 0
+#endif
 
 namespace pylon {
 
-constexpr bool SIGMOID = PYLON_SIGMOID_WEIGHTS != 0;
+constexpr bool SIGMOID = PYLON_SIGMOID_WEIGHTS != 0, OPTIONS = PYLON_SOFTMAX_OPTIONS != 0;
+static_assert(!(SIGMOID && OPTIONS), "sigmoid weights or a softmax's options");
+constexpr bool SPLIT = SIGMOID || OPTIONS;   // a weight is two bfloat16 numbers
 
-// What goes with sigmoid weights (all unused with a softmax).
+// What goes with sigmoid weights and with a softmax's options (all unused with a plain softmax).
 struct HeadOptions {
-  const float* score_bias;       // [nq] or null: added to the scaled scores
+  const float* score_bias;       // sigmoid weights: [nq] or null, added to the scaled scores
   const __nv_bfloat16* gate;     // [tokens, >= nq], rows gate_stride apart, or null
   long long gate_stride;
   float factor;                  // on every output
+  int gate_elements;             // gate is [tokens, >= nq * D]: a number for every element of the output
+  const float* slopes;           // a softmax with options: [nq] or null
+  const float* sinks;            // likewise
 };
 
 constexpr int D = PYLON_HEAD_DIM;
@@ -137,9 +150,17 @@ __device__ __forceinline__ unsigned pack_dropped(float lo, float hi, unsigned pa
 __device__ __forceinline__ float head_score_bias(const HeadOptions& o, int head) { return SIGMOID && o.score_bias ? o.score_bias[head] * 1.4426950408889634f : 0.f; }
 // What an output of this head is multiplied by.
 __device__ __forceinline__ float head_factor(const HeadOptions& o, size_t token, int head) {
-  if (!SIGMOID) return 1.f;
-  return o.gate ? o.factor * sigmoid_exp2(1.4426950408889634f * __bfloat162float(o.gate[token * o.gate_stride + head])) : o.factor;
+  if (!SPLIT) return 1.f;
+  return o.gate && !o.gate_elements ? o.factor * sigmoid_exp2(1.4426950408889634f * __bfloat162float(o.gate[token * o.gate_stride + head])) : o.factor;
 }
+
+// What element `col` of it is multiplied by besides.
+__device__ __forceinline__ float element_factor(const HeadOptions& o, size_t token, int head, int col) {
+  if (!SPLIT || !o.gate || !o.gate_elements) return 1.f;
+  return sigmoid_exp2(1.4426950408889634f * __bfloat162float(o.gate[token * o.gate_stride + (size_t)head * D + col]));
+}
+__device__ __forceinline__ float head_slope(const HeadOptions& o, int head) { return OPTIONS && o.slopes ? o.slopes[head] * 1.4426950408889634f : 0.f; }
+__device__ __forceinline__ float head_sink(const HeadOptions& o, int head) { return o.sinks[head] * 1.4426950408889634f; }   // log2 units
 
 // Gathers keys [tile * 64, tile * 64 + 64) of one KV head into a padded shared tile.  Keys
 // at or beyond kv_len, or without a page, are zero-filled.
@@ -219,7 +240,10 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
   int row_pos[MT][2], row_token[MT][2], row_head[MT][2], row_lo[MT][2];
   const bool bounded = p.window > 0 || p.chunk > 0;
   bool row_valid[MT][2];
-  float row_bias[MT][2];
+  float row_bias[MT][2], row_slope[MT][2];
+  // With slopes the scores are brought to log2 units before the softmax, whose own factor is then one.
+  const bool sloped = OPTIONS && p.heads.slopes != nullptr;
+  const float unit = sloped ? 1.f : p.scale_log2;
   int warp_min_pos = 0x7fffffff;
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
@@ -232,6 +256,7 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
       row_pos[mt][h] = pos0 + row_token[mt][h];
       row_lo[mt][h] = first_visible(p, row_pos[mt][h]);
       row_bias[mt][h] = head_score_bias(p.heads, row_head[mt][h]);
+      row_slope[mt][h] = head_slope(p.heads, row_head[mt][h]);
     }
   }
   // Smallest position among the warp's rows (rows past the end count as the first row): tiles
@@ -251,6 +276,12 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
   float row_max[MT][2], row_sum[MT][2];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) { row_max[mt][0] = row_max[mt][1] = -INFINITY; row_sum[mt][0] = row_sum[mt][1] = 0.f; }
+  if (OPTIONS && p.heads.sinks && split == 0) {   // a row's four lanes add their sums up: one of them has the sink
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) { row_max[mt][h] = head_sink(p.heads, row_head[mt][h]) / unit; row_sum[mt][h] = tq == 0 ? 1.f : 0.f; }
+  }
 
   auto load_tile = [&](int stage, int tile) {
     if (contiguous) {
@@ -324,6 +355,15 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
 #pragma unroll
               for (int i = 0; i < 4; ++i) s[mt][n][i] = soft_tanh(s[mt][n][i] * p.cap_pre);
         }
+        if (sloped) {
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+            for (int n = 0; n < BLOCK_N / 8; ++n)
+#pragma unroll
+              for (int i = 0; i < 4; ++i)
+                s[mt][n][i] = fmaf(s[mt][n][i], p.scale_log2, -row_slope[mt][i >> 1] * (float)(row_pos[mt][i >> 1] - (tile * BLOCK_N + 2 * tq + n * 8 + (i & 1))));
+        }
         if (!no_mask) {
           const int key_base = tile * BLOCK_N + 2 * tq;
 #pragma unroll
@@ -361,13 +401,13 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
             const float new_max = fmaxf(row_max[mt][h], mx);
             const float use_max = new_max == -INFINITY ? 0.f : new_max;
-            const float alpha = fast_exp2((row_max[mt][h] - use_max) * p.scale_log2);   // 2^-inf = 0 on the first tile
-            const float shift = use_max * p.scale_log2;
+            const float alpha = fast_exp2((row_max[mt][h] - use_max) * unit);   // 2^-inf = 0 on the first tile
+            const float shift = use_max * unit;
             float sum = 0.f;
 #pragma unroll
             for (int n = 0; n < BLOCK_N / 8; ++n) {
-              const float p0 = fast_exp2(s[mt][n][2 * h] * p.scale_log2 - shift);
-              const float p1 = fast_exp2(s[mt][n][2 * h + 1] * p.scale_log2 - shift);
+              const float p0 = fast_exp2(s[mt][n][2 * h] * unit - shift);
+              const float p1 = fast_exp2(s[mt][n][2 * h + 1] * unit - shift);
               s[mt][n][2 * h] = p0;
               s[mt][n][2 * h + 1] = p1;
               sum += p0 + p1;
@@ -393,7 +433,7 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
             for (int f = 0; f < 4; ++f) {
               const float low = s[mt][2 * kk + (f >> 1)][2 * (f & 1)], high = s[mt][2 * kk + (f >> 1)][2 * (f & 1) + 1];
               a[mt][f] = pack_bf16(low, high);
-              if (SIGMOID) dropped[mt][f] = pack_dropped(low, high, a[mt][f]);
+              if (SPLIT) dropped[mt][f] = pack_dropped(low, high, a[mt][f]);
             }
           }
 #pragma unroll
@@ -404,7 +444,7 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
             for (int mt = 0; mt < MT; ++mt) {
               mma_bf16(o[mt][2 * d2], a[mt], b[0], b[1]);
               mma_bf16(o[mt][2 * d2 + 1], a[mt], b[2], b[3]);
-              if (SIGMOID) {
+              if (SPLIT) {
                 mma_bf16(o[mt][2 * d2], dropped[mt], b[0], b[1]);
                 mma_bf16(o[mt][2 * d2 + 1], dropped[mt], b[2], b[3]);
               }
@@ -426,19 +466,22 @@ __global__ void __launch_bounds__(ATT_THREADS) paged_attention_mma_kernel(const 
       sum += __shfl_xor_sync(0xffffffffu, sum, 2);
       if (!row_valid[mt][h]) continue;
       const size_t token = (size_t)q0 + row_token[mt][h];
-      const float inv = SIGMOID ? (p.num_splits == 1 ? head_factor(p.heads, token, row_head[mt][h]) : 1.f) : (sum > 0.f ? 1.f / sum : 0.f);
+      float inv = SIGMOID ? 1.f : (sum > 0.f ? 1.f / sum : 0.f);
+      if (p.num_splits == 1) inv *= head_factor(p.heads, token, row_head[mt][h]);
       if (p.num_splits == 1) {
         __nv_bfloat16* dst = p.out + token * p.out_stride + (size_t)row_head[mt][h] * D;
 #pragma unroll
         for (int i = 0; i < D / 8; ++i)
-          *reinterpret_cast<__nv_bfloat162*>(dst + i * 8 + 2 * tq) = __floats2bfloat162_rn(o[mt][i][2 * h] * inv, o[mt][i][2 * h + 1] * inv);
+          *reinterpret_cast<__nv_bfloat162*>(dst + i * 8 + 2 * tq) =
+              __floats2bfloat162_rn(o[mt][i][2 * h] * inv * element_factor(p.heads, token, row_head[mt][h], i * 8 + 2 * tq),
+                                    o[mt][i][2 * h + 1] * inv * element_factor(p.heads, token, row_head[mt][h], i * 8 + 2 * tq + 1));
       } else {
         const size_t slot = ((size_t)split * p.total_tokens + token) * p.nq + row_head[mt][h];
         float* dst = p.partial_out + slot * D;
 #pragma unroll
         for (int i = 0; i < D / 8; ++i)
           *reinterpret_cast<float2*>(dst + i * 8 + 2 * tq) = make_float2(o[mt][i][2 * h] * inv, o[mt][i][2 * h + 1] * inv);
-        if (tq == 0 && !SIGMOID) p.partial_lse[slot] = sum > 0.f ? row_max[mt][h] * p.scale_log2 + log2f(sum) : -INFINITY;
+        if (tq == 0 && !SIGMOID) p.partial_lse[slot] = sum > 0.f ? row_max[mt][h] * unit + log2f(sum) : -INFINITY;
       }
     }
   }
@@ -767,6 +810,8 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
   // Segments of pairs that other blocks share leave partial results; the block publishes them
   // together (one fence and one round of counter updates for all of them, at the end of its run
   // or when the list is full), and combines those pairs for which it turns out to be last.
+  const bool sloped = OPTIONS && p.heads.slopes != nullptr;   // the scores are brought to log2 units before the softmax
+  const float unit = sloped ? 1.f : p.scale_log2;
   int pending_count = 0;
   auto publish_and_combine = [&]() {
     if (pending_count == 0) return;
@@ -818,7 +863,11 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
         const size_t token = (size_t)q0 + r / G;
         const int head = kv_head * G + r % G;
         // with sigmoid weights every segment's log-sum-exp is written as 0: the parts have been added up with weights of one
-        const float inv = SIGMOID ? head_factor(p.heads, token, head) : (run_total > 0.f ? 1.f / run_total : 0.f);
+        const float inv = (SIGMOID ? 1.f : (run_total > 0.f ? 1.f / run_total : 0.f)) * head_factor(p.heads, token, head);
+        if (SPLIT && p.heads.gate_elements) {
+          sum.x *= element_factor(p.heads, token, head, col); sum.y *= element_factor(p.heads, token, head, col + 1);
+          sum.z *= element_factor(p.heads, token, head, col + 2); sum.w *= element_factor(p.heads, token, head, col + 3);
+        }
         __nv_bfloat16* dst = p.out + token * p.out_stride + (size_t)head * D + col;
         *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(sum.x * inv, sum.y * inv), pack_bf16(sum.z * inv, sum.w * inv));
       }
@@ -841,12 +890,15 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
 
     int row_pos[2], row_lo[2];
     bool row_valid[2];
-    float row_bias[2];
+    float row_bias[2], row_slope[2];
+    // The sink is met by one segment of a pair: the first block's; in a cluster the last one's, whose share of the tiles is never empty.
+    const bool takes_sink = OPTIONS && p.heads.sinks && (CLUSTER ? cluster_rank == CLUSTER - 1 : (int)blockIdx.x == first_block);
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int m = g + 8 * h;
       row_valid[h] = m < packed_rows;
       row_bias[h] = head_score_bias(p.heads, kv_head * G + (row_valid[h] ? m % G : 0));
+      row_slope[h] = head_slope(p.heads, kv_head * G + (row_valid[h] ? m % G : 0));
       row_pos[h] = pos0 + (row_valid[h] ? m / G : 0);
       row_lo[h] = first_visible(p, row_pos[h]);
     }
@@ -962,6 +1014,13 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
 #pragma unroll
           for (int i = 0; i < 4; ++i) s[n][i] = soft_tanh(s[n][i] * p.cap_pre);
       }
+      if (sloped) {
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int i = 0; i < 4; ++i)
+            s[n][i] = fmaf(s[n][i], p.scale_log2, -row_slope[i >> 1] * (float)(row_pos[i >> 1] - (tile * BLOCK_N + warp * 16 + 2 * tq + n * 8 + (i & 1))));
+      }
       if (p.window > 0 || p.chunk > 0 || tile * BLOCK_N + BLOCK_N - 1 > pos0) {
         const int key_base = tile * BLOCK_N + warp * 16 + 2 * tq;
 #pragma unroll
@@ -993,13 +1052,13 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
         const float new_max = fmaxf(row_max[h], mx);
         const float use_max = new_max == -INFINITY ? 0.f : new_max;
-        const float alpha = fast_exp2((row_max[h] - use_max) * p.scale_log2);
-        const float shift = use_max * p.scale_log2;
+        const float alpha = fast_exp2((row_max[h] - use_max) * unit);
+        const float shift = use_max * unit;
         float sum = 0.f;
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
-          const float p0 = fast_exp2(s[n][2 * h] * p.scale_log2 - shift);
-          const float p1 = fast_exp2(s[n][2 * h + 1] * p.scale_log2 - shift);
+          const float p0 = fast_exp2(s[n][2 * h] * unit - shift);
+          const float p1 = fast_exp2(s[n][2 * h + 1] * unit - shift);
           s[n][2 * h] = p0;
           s[n][2 * h + 1] = p1;
           sum += p0 + p1;
@@ -1015,7 +1074,7 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
       a[2] = pack_bf16(s[1][0], s[1][1]);
       a[3] = pack_bf16(s[1][2], s[1][3]);
       unsigned dropped[4];
-      if (SIGMOID) {
+      if (SPLIT) {
 #pragma unroll
         for (int f = 0; f < 4; ++f) dropped[f] = pack_dropped(s[f >> 1][2 * (f & 1)], s[f >> 1][2 * (f & 1) + 1], a[f]);
       }
@@ -1025,7 +1084,7 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
         ldmatrix_x4_trans(b, vs + Tiles::offset(key_row + 8 * ((lane >> 3) & 1), d2 * 2 + (lane >> 4)));
         mma_bf16(o[2 * d2], a, b[0], b[1]);
         mma_bf16(o[2 * d2 + 1], a, b[2], b[3]);
-        if (SIGMOID) {
+        if (SPLIT) {
           mma_bf16(o[2 * d2], dropped, b[0], b[1]);
           mma_bf16(o[2 * d2 + 1], dropped, b[2], b[3]);
         }
@@ -1078,16 +1137,21 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
 #pragma unroll
       for (int w = 0; w < 4; ++w) mx = fmaxf(mx, merge_max[w * SMALL_ROWS + r]);
       float weight[4], total = 0.f;
+      if (takes_sink) {
+        const float sink = head_sink(p.heads, kv_head * G + r % G) / unit;
+        mx = fmaxf(mx, sink);
+        total = fast_exp2((sink - mx) * unit);
+      }
 #pragma unroll
       for (int w = 0; w < 4; ++w) {
         const float m = merge_max[w * SMALL_ROWS + r];
-        weight[w] = m == -INFINITY ? 0.f : fast_exp2((m - mx) * p.scale_log2);
+        weight[w] = m == -INFINITY ? 0.f : fast_exp2((m - mx) * unit);
         total += weight[w] * merge_sum[w * SMALL_ROWS + r];
       }
       const float inv = total > 0.f ? 1.f / total : 0.f;
 #pragma unroll
       for (int w = 0; w < 4; ++w) merge_max[w * SMALL_ROWS + r] = weight[w] * inv;   // from here on: the warp's share
-      row_lse[r] = total > 0.f ? mx * p.scale_log2 + log2f(total) : -INFINITY;     // the segment's log-sum-exp (log2)
+      row_lse[r] = total > 0.f ? mx * unit + log2f(total) : -INFINITY;     // the segment's log-sum-exp (log2)
     }
     __syncthreads();
     const size_t slot = (size_t)pair + blockIdx.x;
@@ -1126,7 +1190,7 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
       if (segments == 1) {
         const size_t token = (size_t)q0 + r / G;
         const int head = kv_head * G + r % G;
-        if (SIGMOID) value *= head_factor(p.heads, token, head);
+        if (SPLIT) value *= head_factor(p.heads, token, head) * element_factor(p.heads, token, head, col);
         p.out[token * p.out_stride + (size_t)head * D + col] = __float2bfloat16_rn(value);
       } else {
         p.decode_out[(slot * SMALL_ROWS + r) * D + col] = value;
@@ -1194,7 +1258,8 @@ __global__ void __launch_bounds__(ATT_THREADS, D <= 128 && CLUSTER_STAGES <= 2 ?
       }
       const size_t token = (size_t)q0 + r / G;
       const int head = kv_head * G + r % G;
-      p.out[token * p.out_stride + (size_t)head * D + col] = __float2bfloat16_rn(SIGMOID ? sum * head_factor(p.heads, token, head) : (total > 0.f ? sum / total : 0.f));
+      p.out[token * p.out_stride + (size_t)head * D + col] = __float2bfloat16_rn((SIGMOID ? sum : (total > 0.f ? sum / total : 0.f)) * head_factor(p.heads, token, head) *
+                                                                                  element_factor(p.heads, token, head, col));
     }
   }
 }
@@ -1238,11 +1303,11 @@ __global__ void combine_splits_kernel(const float* __restrict__ partial_out, con
       if (e < D) acc[i] += w * src[e];
     }
   }
-  const float inv = SIGMOID ? head_factor(heads, (size_t)(item / nq), (int)(item % nq)) : (total > 0.f ? 1.f / total : 0.f);
+  const float inv = (SIGMOID ? 1.f : (total > 0.f ? 1.f / total : 0.f)) * head_factor(heads, (size_t)(item / nq), (int)(item % nq));
 #pragma unroll
   for (int i = 0; i < (D + 31) / 32; ++i) {
     const int e = lane + 32 * i;
-    if (e < D) out[(size_t)(item / nq) * out_stride + (size_t)(item % nq) * D + e] = __float2bfloat16_rn(acc[i] * inv);
+    if (e < D) out[(size_t)(item / nq) * out_stride + (size_t)(item % nq) * D + e] = __float2bfloat16_rn(acc[i] * inv * element_factor(heads, (size_t)(item / nq), (int)(item % nq), e));
   }
 }
 
@@ -1529,25 +1594,39 @@ extern "C" int pylon_paged_attention_mma_masked(const void* q, long long q_strid
                                                 int nq, int nkv, int window, int chunk, float softcap, float scale, int num_rows,
                                                 int total_tokens, int max_q, int num_splits, int decode_blocks, int skip_large,
                                                 int rows_alike, int* error, cudaStream_t stream) {
-  if (SIGMOID) PYLON_REFUSE("paged_attention_mma: this library is built for sigmoid weights");
+  if (SPLIT) PYLON_REFUSE("paged_attention_mma: this library is built for sigmoid weights or a softmax with options");
   return attention_mma_entry(q, q_stride, k_pages, v_pages, out, scratch, counters, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv,
                              window, chunk, softcap, scale, num_rows, total_tokens, max_q, num_splits, decode_blocks, skip_large, rows_alike, error, stream,
-                             (long long)nq * D, HeadOptions{nullptr, nullptr, 0, 1.f});
+                             (long long)nq * D, HeadOptions{nullptr, nullptr, 0, 1.f, 0, nullptr, nullptr});
 }
 
 // Sigmoid weights (a library built for them): score_bias float32 [nq] or null; gate bfloat16 [tokens, >= nq] with rows gate_stride elements
-// apart, or null; factor on every output; out's rows out_stride elements apart.
+// apart (gate_elements != 0: [tokens, >= nq * D], a number for every element of the output), or null; factor on every output; out's rows out_stride elements apart.
 extern "C" int pylon_paged_attention_mma_sigmoid(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
                                                  void* out, float* scratch, unsigned* counters, const int* q_start, const int* kv_len,
                                                  const int* block_table, int table_width, int page_size, int num_pages,
                                                  int nq, int nkv, int window, int chunk, float softcap, float scale, int num_rows,
                                                  int total_tokens, int max_q, int num_splits, int decode_blocks, int skip_large,
-                                                 int rows_alike, int* error, const float* score_bias, const void* gate, long long gate_stride, float factor,
-                                                 long long out_stride, cudaStream_t stream) {
+                                                 int rows_alike, int* error, const float* score_bias, const void* gate, long long gate_stride, int gate_elements,
+                                                 float factor, long long out_stride, cudaStream_t stream) {
   if (!SIGMOID) PYLON_REFUSE("paged_attention_mma: this library is built for a softmax");
   return attention_mma_entry(q, q_stride, k_pages, v_pages, out, scratch, counters, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv,
                              window, chunk, softcap, scale, num_rows, total_tokens, max_q, num_splits, decode_blocks, skip_large, rows_alike, error, stream,
-                             out_stride, HeadOptions{score_bias, (const __nv_bfloat16*)gate, gate_stride, factor});
+                             out_stride, HeadOptions{score_bias, (const __nv_bfloat16*)gate, gate_stride, factor, gate_elements, nullptr, nullptr});
+}
+
+// A softmax with options (a library built for them): slopes and sinks float32 [nq] or null; the rest as with sigmoid weights.
+extern "C" int pylon_paged_attention_mma_options(const void* q, long long q_stride, const void* k_pages, const void* v_pages,
+                                                 void* out, float* scratch, unsigned* counters, const int* q_start, const int* kv_len,
+                                                 const int* block_table, int table_width, int page_size, int num_pages,
+                                                 int nq, int nkv, int window, int chunk, float softcap, float scale, int num_rows,
+                                                 int total_tokens, int max_q, int num_splits, int decode_blocks, int skip_large,
+                                                 int rows_alike, int* error, const float* slopes, const float* sinks, const void* gate, long long gate_stride,
+                                                 int gate_elements, float factor, long long out_stride, cudaStream_t stream) {
+  if (!OPTIONS) PYLON_REFUSE("paged_attention_mma: this library is not built for a softmax with options");
+  return attention_mma_entry(q, q_stride, k_pages, v_pages, out, scratch, counters, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv,
+                             window, chunk, softcap, scale, num_rows, total_tokens, max_q, num_splits, decode_blocks, skip_large, rows_alike, error, stream,
+                             out_stride, HeadOptions{nullptr, (const __nv_bfloat16*)gate, gate_stride, factor, gate_elements, slopes, sinks});
 }
 
 // The softmax without chunks and soft cap.

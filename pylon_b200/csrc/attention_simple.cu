@@ -18,9 +18,12 @@
 // With `bias` (float32 [bias_rows, nq]) the scaled (and capped) score of the key d = p - j positions back gets
 // bias[min(d, bias_rows - 1), h] added: a learnt function of the distance that is constant from bias_rows - 1 on.
 //
+// With `slopes` (float32 [nq]) that score loses slopes[h] for every position of distance.
+//
 // With `sigmoid` weights nothing is normalised: a visible key's weight is sigmoid(score + score_bias[h]) (score_bias float32 [nq] or
-// null).  `gate` ([tokens, >= nq] in the compute dtype, or null): head h's output is multiplied by sigmoid(gate[t, h]); `factor`
-// multiplies every output; the output's rows may lie out_stride elements apart.
+// null).  `gate` ([tokens, >= nq] in the compute dtype, or null): head h's output is multiplied by sigmoid(gate[t, h]), or with gate_elements
+// ([tokens, >= nq * dv]) element e of it by sigmoid(gate[t, h * dv + e]); `factor` multiplies every output; the output's rows may lie
+// out_stride elements apart.
 //
 // The keys of a token are walked in chunks of 128 positions aligned at position 0, so a
 // token's result depends on its position only, not on how the step was cut or batched.
@@ -39,7 +42,7 @@ __global__ void __launch_bounds__(SIMPLE_THREADS) paged_attention_simple_kernel(
     int num_pages, int nq, int nkv, int d, int dv, int window, int chunk, float softcap, float scale,
     const float* __restrict__ sinks, long long k_row_stride, long long v_row_stride, int keep_first, const float* __restrict__ bias,
     int bias_rows, int sigmoid, const float* __restrict__ score_bias, const T* __restrict__ gate, long long gate_stride, float factor,
-    long long out_stride) {
+    long long out_stride, const float* __restrict__ slopes, int gate_elements) {
   extern __shared__ long long shared[];
   long long* offsets = shared;                                      // [128] cache rows of the keys (page, head, slot), -1: none
   float* probs = reinterpret_cast<float*>(offsets + SIMPLE_THREADS);  // [128]
@@ -79,6 +82,7 @@ __global__ void __launch_bounds__(SIMPLE_THREADS) paged_attention_simple_kernel(
         for (int e = 0; e < d; ++e) dot = fmaf(qs[e], to_float<T>(krow[e]), dot);
         score = softcap > 0.f ? softcap * tanhf(dot / softcap) : dot;
         if (bias) score += bias[(size_t)(pos - j < bias_rows ? pos - j : bias_rows - 1) * nq + h];
+        if (slopes) score -= slopes[h] * (float)(pos - j);
       }
     }
     offsets[tid] = offset;
@@ -115,11 +119,13 @@ __global__ void __launch_bounds__(SIMPLE_THREADS) paged_attention_simple_kernel(
   T* orow = out + (size_t)t * out_stride + (size_t)h * dv;
   float inv = sigmoid ? 1.f : (running_sum > 0.f ? 1.f / running_sum : 0.f);
   inv *= factor;
-  if (gate) inv *= 1.f / (1.f + expf(-to_float<T>(gate[(size_t)t * gate_stride + h])));
+  if (gate && !gate_elements) inv *= 1.f / (1.f + expf(-to_float<T>(gate[(size_t)t * gate_stride + h])));
 #pragma unroll
   for (int k = 0; k < SIMPLE_MAX_DIMS_PER_THREAD; ++k) {
     const int e = tid + k * SIMPLE_THREADS;
-    if (e < dv) orow[e] = from_float<T>(acc[k] * inv);
+    if (e >= dv) continue;
+    const float open = gate && gate_elements ? 1.f / (1.f + expf(-to_float<T>(gate[(size_t)t * gate_stride + (size_t)h * dv + e]))) : 1.f;
+    orow[e] = from_float<T>(acc[k] * inv * open);
   }
 }
 
@@ -134,7 +140,8 @@ extern "C" int pylon_paged_attention_simple(const void* q, long long q_token_str
                                             int chunk, float softcap, float scale, const float* sinks,
                                             long long k_row_stride, long long v_row_stride, int num_tokens, int dtype,
                                             int keep_first, const float* bias, int bias_rows, int sigmoid, const float* score_bias,
-                                            const void* gate, long long gate_stride, float factor, long long out_stride, cudaStream_t stream) {
+                                            const void* gate, long long gate_stride, float factor, long long out_stride, const float* slopes, int gate_elements,
+                                            cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (d < 1 || d > 2048) PYLON_REFUSE("paged_attention_simple: head size %d is outside 1..2048", d);
   if (k_row_stride == 0) k_row_stride = d;
@@ -146,7 +153,7 @@ extern "C" int pylon_paged_attention_simple(const void* q, long long q_token_str
   if (keep_first < 0 || (keep_first > 0 && chunk > 0)) PYLON_REFUSE("paged_attention_simple: %d kept first keys (not with chunks)", keep_first);
   if (bias && bias_rows < 1) PYLON_REFUSE("paged_attention_simple: a bias table of %d rows", bias_rows);
   if (out_stride == 0) out_stride = (long long)nq * dv;
-  if (out_stride < (long long)nq * dv || (score_bias && !sigmoid) || (sigmoid && sinks)) PYLON_REFUSE("paged_attention_simple: output rows %lld apart, a number per head on the scores without sigmoid weights, or a sink with them", out_stride);
+  if (out_stride < (long long)nq * dv || (score_bias && !sigmoid) || (sigmoid && (sinks || slopes))) PYLON_REFUSE("paged_attention_simple: output rows %lld apart, a number per head on the scores without sigmoid weights, or a sink with them", out_stride);
   if (nkv < 1 || nq < 1 || nq % nkv) PYLON_REFUSE("paged_attention_simple: %d query heads over %d KV heads", nq, nkv);
   if (nq > 65535) PYLON_REFUSE("paged_attention_simple: %d query heads", nq);
   if (page_size < 1 || table_width < 1 || window < 0)
@@ -157,13 +164,13 @@ extern "C" int pylon_paged_attention_simple(const void* q, long long q_token_str
     paged_attention_simple_kernel<float><<<grid, SIMPLE_THREADS, smem, stream>>>(
         (const float*)q, q_token_stride, (const float*)k_pages, (const float*)v_pages, (float*)out, positions,
         token_row, block_table, table_width, page_size, num_pages, nq, nkv, d, dv, window, chunk, softcap, scale, sinks, k_row_stride, v_row_stride,
-        keep_first, bias, bias_rows, sigmoid, score_bias, (const float*)gate, gate_stride, factor, out_stride);
+        keep_first, bias, bias_rows, sigmoid, score_bias, (const float*)gate, gate_stride, factor, out_stride, slopes, gate_elements);
   else if (dtype == PYLON_DTYPE_BF16)
     paged_attention_simple_kernel<__nv_bfloat16><<<grid, SIMPLE_THREADS, smem, stream>>>(
         (const __nv_bfloat16*)q, q_token_stride, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages,
         (__nv_bfloat16*)out, positions, token_row, block_table, table_width, page_size, num_pages, nq, nkv, d, dv,
         window, chunk, softcap, scale, sinks, k_row_stride, v_row_stride, keep_first, bias, bias_rows, sigmoid, score_bias,
-        (const __nv_bfloat16*)gate, gate_stride, factor, out_stride);
+        (const __nv_bfloat16*)gate, gate_stride, factor, out_stride, slopes, gate_elements);
   else
     PYLON_REFUSE("paged_attention_simple: unknown dtype %d", dtype);
   PYLON_CHECK_LAUNCH("paged_attention_simple");

@@ -39,6 +39,11 @@
 // rescaled.  A weight is two bfloat16 numbers, the rounded weight and what the rounding dropped (it counts with 16 of its 24 bits):
 // the two halves fill exactly the columns of the scores they replace, and the weighted sum is two products over one tile of values.
 // Two sigmoids share a reciprocal: with a = 1 + 2^-x and b = 1 + 2^-y, 1 / (a b) times b and times a.
+//
+// Built with -DPYLON_SOFTMAX_OPTIONS=1 the softmax has what few designs ask for: a slope per head on the distance (the score of the key d
+// positions back loses slopes[h] d), a sink per head (the denominator also holds exp(sinks[h]), met before all keys), outputs times a
+// factor and the sigmoid of a gate per head or per element, rows of the output in a wider row; and its weights enter the weighted sum as two
+// bfloat16 numbers, as the sigmoid ones do.
 #include "common.cuh"
 
 #include <cuda.h>
@@ -51,11 +56,16 @@
 #ifndef PYLON_SIGMOID_WEIGHTS
 #define PYLON_SIGMOID_WEIGHTS 0
 #endif
+#ifndef PYLON_SOFTMAX_OPTIONS
+#define PYLON_SOFTMAX_OPTIONS 0
+#endif
 
 namespace pylon {
 
 constexpr int D = PYLON_HEAD_DIM;
-constexpr bool SIGMOID = PYLON_SIGMOID_WEIGHTS != 0;
+constexpr bool SIGMOID = PYLON_SIGMOID_WEIGHTS != 0, OPTIONS = PYLON_SOFTMAX_OPTIONS != 0;
+static_assert(!(SIGMOID && OPTIONS), "sigmoid weights or a softmax's options");
+constexpr bool SPLIT = SIGMOID || OPTIONS;     // a weight is two bfloat16 numbers
 static_assert(D == 64 || D == 128, "the tcgen05 attention is built for head sizes 64 and 128");
 constexpr int FA_BM = 128, FA_BN = 64, FA_STAGES = 2, FA_THREADS = 192;
 constexpr int FA_SMALL_ROWS = 16;                  // rows with at most this many packed query rows belong to the decode kernel
@@ -85,10 +95,13 @@ struct FaParams {
   float scale_log2;
   int* error;
   long long out_stride;            // elements between the output rows of two tokens
-  // with sigmoid weights
-  const float* score_bias;         // [nq] or null
+  const float* score_bias;         // sigmoid weights: [nq] or null
+  const float* slopes;             // a softmax with options: [nq] or null
+  const float* sinks;              // likewise
+  // with either
   const __nv_bfloat16* gate;       // [tokens, >= nq] with rows gate_stride elements apart, or null: head h of token t is multiplied by its sigmoid
   long long gate_stride;
+  int gate_elements;               // gate is [tokens, >= nq * D]: a number for every element
   float factor;                    // on every output
 };
 
@@ -342,7 +355,7 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
         for (int kk = 0; kk < FA_BN / 16; ++kk) {   // 16 keys: 32 bytes along a row of P, two 8-key groups (2048 bytes) down V
           const uint64_t b = fa_desc(v_tile + kk * 2048, FA_BN * 128, 1024);
           fa_mma_a_tmem(tmem_base + FA_O_COLUMN, tmem_base + (t & 1) * FA_S_COLUMNS + kk * 8, b, idesc_o, (t | kk) != 0 ? 1u : 0u);
-          if (SIGMOID) fa_mma_a_tmem(tmem_base + FA_O_COLUMN, tmem_base + (t & 1) * FA_S_COLUMNS + FA_BN / 2 + kk * 8, b, idesc_o, 1u);   // what the rounding dropped
+          if (SPLIT) fa_mma_a_tmem(tmem_base + FA_O_COLUMN, tmem_base + (t & 1) * FA_S_COLUMNS + FA_BN / 2 + kk * 8, b, idesc_o, 1u);   // what the rounding dropped
         }
         fa_commit(&v_empty[t & 1]);
         fa_commit(&pv_done[t & 1]);
@@ -384,8 +397,11 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
       fa_mbar_arrive(q_full);
     }
     const unsigned lane_base = tmem_base + ((unsigned)(warp * 32) << 16);
-    float reference = -INFINITY;   // the maximum the weights refer to (log2 units, scaled)
-    float sum = 0.f;
+    const bool sloped = OPTIONS && p.slopes != nullptr, sunk = OPTIONS && p.sinks != nullptr;
+    const float slope_log2 = sloped ? p.slopes[head] * 1.4426950408889634f : 0.f;
+    const float unit = sloped ? 1.f : p.scale_log2;   // with slopes the scores are brought to log2 units first
+    float reference = sunk ? p.sinks[head] * 1.4426950408889634f : -INFINITY;   // the maximum the weights refer to (log2 units, scaled); a sink is met first
+    float sum = sunk ? 1.f : 0.f;
     const float bias_log2 = SIGMOID && p.score_bias ? p.score_bias[head] * 1.4426950408889634f : 0.f;
     bool alive = true;
     for (int t = 0; t < num_tiles; ++t) {
@@ -407,6 +423,11 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
         // tanh to float32 accuracy from one exponential and one division: 1 - 2 / (e^(2x) + 1)
 #pragma unroll
         for (int j = 0; j < FA_BN; ++j) s[j] = 1.f - __fdividef(2.f, fa_exp2(s[j] * (p.cap_pre * 2.8853900817779268f)) + 1.f);
+      }
+      if (sloped) {
+        const float here = -slope_log2 * (float)(pos - key0);   // what the tile's first key loses; every key after it loses one slope less
+#pragma unroll
+        for (int j = 0; j < FA_BN; ++j) s[j] = fmaf(s[j], p.scale_log2, fmaf(slope_log2, (float)j, here));
       }
       const bool masked = p.window > 0 || p.chunk > 0 || key0 + FA_BN - 1 > pos0 + token_lo || !valid;
       if (masked) {
@@ -445,7 +466,7 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
         for (int j = 8; j < FA_BN; ++j) lane_max[j & 7] = fmaxf(lane_max[j & 7], s[j]);
         float tile_max = fmaxf(fmaxf(fmaxf(lane_max[0], lane_max[1]), fmaxf(lane_max[2], lane_max[3])),
                                fmaxf(fmaxf(lane_max[4], lane_max[5]), fmaxf(lane_max[6], lane_max[7])));
-        tile_max *= p.scale_log2;   // the scale is positive: the largest score stays the largest
+        tile_max *= unit;   // the scale is positive: the largest score stays the largest
         // The reference moves only when the maximum has grown by more than the step (or was not set yet).
         const bool move = tile_max > reference + FA_RESCALE_STEP || (reference == -INFINITY && tile_max > -INFINITY);
         const float alpha = move ? (reference == -INFINITY ? 0.f : fa_exp2(reference - tile_max)) : 1.f;
@@ -456,9 +477,18 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
         float part_sum[4] = {0.f, 0.f, 0.f, 0.f};   // four chains, for the same reason
 #pragma unroll
         for (int j = 0; j < FA_BN; j += 2) {
-          const float w0 = fa_exp2(fmaf(s[j], p.scale_log2, -use)), w1 = fa_exp2(fmaf(s[j + 1], p.scale_log2, -use));   // 0 for masked keys
+          const float w0 = fa_exp2(fmaf(s[j], unit, -use)), w1 = fa_exp2(fmaf(s[j + 1], unit, -use));   // 0 for masked keys
           part_sum[(j >> 1) & 3] += w0 + w1;
           packed[j / 2] = fa_pack(w0, w1);
+          if (SPLIT) { s[j] = w0; s[j + 1] = w1; }
+        }
+        if (SPLIT) {
+          unsigned dropped[FA_BN / 2];
+#pragma unroll
+          for (int j = 0; j < FA_BN; j += 2)
+            dropped[j / 2] = fa_pack(s[j] - __uint_as_float(packed[j / 2] << 16), s[j + 1] - __uint_as_float(packed[j / 2] & 0xffff0000u));
+          fa_tmem_store_16(lane_base + (t & 1) * FA_S_COLUMNS + FA_BN / 2, dropped);
+          fa_tmem_store_16(lane_base + (t & 1) * FA_S_COLUMNS + FA_BN / 2 + 16, dropped + 16);
         }
         sum += (part_sum[0] + part_sum[1]) + (part_sum[2] + part_sum[3]);
         // The weights go into tensor memory over this tile's scores, two to a column (this lane's scores are in registers
@@ -500,16 +530,29 @@ __global__ void __launch_bounds__(FA_THREADS, 2) attention_tcgen05_kernel(const 
     if (alive) {
       fa_fence_after();
       float inv = sum > 0.f ? 1.f / sum : 0.f;
-      if (SIGMOID) {
-        inv = p.factor;
-        if (p.gate && valid) inv *= __fdividef(1.f, 1.f + fa_exp2(-1.4426950408889634f * __bfloat162float(p.gate[(size_t)(q0 + token) * p.gate_stride + head])));
+      if (SPLIT) {
+        inv = SIGMOID ? p.factor : inv * p.factor;
+        if (p.gate && !p.gate_elements && valid) inv *= __fdividef(1.f, 1.f + fa_exp2(-1.4426950408889634f * __bfloat162float(p.gate[(size_t)(q0 + token) * p.gate_stride + head])));
       }
       __nv_bfloat16* dst = p.out + (size_t)(q0 + token) * p.out_stride + (size_t)head * D;
+      const __nv_bfloat16* gates = SPLIT && p.gate && p.gate_elements ? p.gate + (size_t)(q0 + token) * p.gate_stride + (size_t)head * D : nullptr;
 #pragma unroll 1
       for (int c = 0; c < D / 32; ++c) {
         unsigned raw[32];
         fa_tmem_load_32(lane_base + FA_O_COLUMN + c * 32, raw);   // warp-wide: rows that are not stored load all the same
         if (valid) {
+          if (SPLIT && gates) {
+#pragma unroll
+            for (int j = 0; j < 32; j += 8) {
+              const uint4 eight = *reinterpret_cast<const uint4*>(gates + c * 32 + j);
+              const unsigned words[4] = {eight.x, eight.y, eight.z, eight.w};
+#pragma unroll
+              for (int i = 0; i < 8; ++i) {
+                const float z = __uint_as_float((i & 1) ? words[i / 2] & 0xffff0000u : words[i / 2] << 16);
+                raw[j + i] = __float_as_uint(__uint_as_float(raw[j + i]) * __fdividef(1.f, 1.f + fa_exp2(-1.4426950408889634f * z)));
+              }
+            }
+          }
 #pragma unroll
           for (int j = 0; j < 32; j += 8)
             *reinterpret_cast<uint4*>(dst + c * 32 + j) = make_uint4(
@@ -590,7 +633,7 @@ static int attention_tcgen05_entry(const void* q, long long q_stride, const void
                                                     int page_size, int num_pages, int nq, int nkv, int window, int chunk, float softcap,
                                                     float scale, int first_row, int num_rows, int max_q, int skip_small, int* error,
                                                     cudaStream_t stream, long long out_stride, const float* score_bias, const void* gate,
-                                                    long long gate_stride, float factor) {
+                                                    long long gate_stride, float factor, const float* slopes, const float* sinks, int gate_elements) {
   if (num_rows <= 0) return 0;
   if (out_stride < (long long)nq * D || out_stride % 8) PYLON_REFUSE("paged_attention_tcgen05: output rows of %d elements %lld apart (a multiple of 8)", nq * D, out_stride);
   if (chunk < 0 || softcap < 0.f) PYLON_REFUSE("paged_attention_tcgen05: chunk %d, soft cap %f", chunk, softcap);
@@ -623,6 +666,8 @@ static int attention_tcgen05_entry(const void* q, long long q_stride, const void
   p.chunk = chunk;
   p.cap_pre = softcap > 0.f ? scale / softcap : 0.f;
   p.error = error;
+  if (gate_elements && gate && (gate_stride % 8 || (uintptr_t)gate % 16)) PYLON_REFUSE("paged_attention_tcgen05: a gate for every element must be 16-byte aligned, its rows a multiple of 8 apart");
+  p.slopes = slopes; p.sinks = sinks; p.gate_elements = gate_elements;
   p.out_stride = out_stride; p.score_bias = score_bias; p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride; p.factor = factor;
   const long long q_tiles = ((long long)max_q * p.group + FA_BM - 1) / FA_BM;
   if (q_tiles > 65535) PYLON_REFUSE("paged_attention_tcgen05: too many query tiles");
@@ -635,22 +680,34 @@ extern "C" int pylon_paged_attention_tcgen05_masked(const void* q, long long q_s
                                                     int page_size, int num_pages, int nq, int nkv, int window, int chunk, float softcap,
                                                     float scale, int first_row, int num_rows, int max_q, int skip_small, int* error,
                                                     cudaStream_t stream) {
-  if (SIGMOID) PYLON_REFUSE("paged_attention_tcgen05: this library is built for sigmoid weights");
+  if (SPLIT) PYLON_REFUSE("paged_attention_tcgen05: this library is built for sigmoid weights or a softmax with options");
   return attention_tcgen05_entry(q, q_stride, k_pages, v_pages, out, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv, window, chunk,
-                                 softcap, scale, first_row, num_rows, max_q, skip_small, error, stream, (long long)nq * D, nullptr, nullptr, 0, 1.f);
+                                 softcap, scale, first_row, num_rows, max_q, skip_small, error, stream, (long long)nq * D, nullptr, nullptr, 0, 1.f, nullptr, nullptr, 0);
 }
 
 // Sigmoid weights (a library built for them): score_bias float32 [nq] or null; gate bfloat16 [tokens, >= nq] with rows gate_stride elements
-// apart, or null; factor on every output; out's rows out_stride elements apart.
+// apart (gate_elements != 0: [tokens, >= nq * D], a number for every element of the output), or null; factor on every output; out's rows out_stride elements apart.
 extern "C" int pylon_paged_attention_tcgen05_sigmoid(const void* q, long long q_stride, const void* k_pages, const void* v_pages, void* out,
                                                      const int* q_start, const int* kv_len, const int* block_table, int table_width,
                                                      int page_size, int num_pages, int nq, int nkv, int window, int chunk, float softcap,
                                                      float scale, int first_row, int num_rows, int max_q, int skip_small, int* error,
-                                                     const float* score_bias, const void* gate, long long gate_stride, float factor, long long out_stride,
-                                                     cudaStream_t stream) {
+                                                     const float* score_bias, const void* gate, long long gate_stride, int gate_elements, float factor,
+                                                     long long out_stride, cudaStream_t stream) {
   if (!SIGMOID) PYLON_REFUSE("paged_attention_tcgen05: this library is built for a softmax");
   return attention_tcgen05_entry(q, q_stride, k_pages, v_pages, out, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv, window, chunk,
-                                 softcap, scale, first_row, num_rows, max_q, skip_small, error, stream, out_stride, score_bias, gate, gate_stride, factor);
+                                 softcap, scale, first_row, num_rows, max_q, skip_small, error, stream, out_stride, score_bias, gate, gate_stride, factor, nullptr, nullptr, gate_elements);
+}
+
+// A softmax with options (a library built for them): slopes and sinks float32 [nq] or null; the rest as with sigmoid weights.
+extern "C" int pylon_paged_attention_tcgen05_options(const void* q, long long q_stride, const void* k_pages, const void* v_pages, void* out,
+                                                     const int* q_start, const int* kv_len, const int* block_table, int table_width,
+                                                     int page_size, int num_pages, int nq, int nkv, int window, int chunk, float softcap,
+                                                     float scale, int first_row, int num_rows, int max_q, int skip_small, int* error,
+                                                     const float* slopes, const float* sinks, const void* gate, long long gate_stride, int gate_elements,
+                                                     float factor, long long out_stride, cudaStream_t stream) {
+  if (!OPTIONS) PYLON_REFUSE("paged_attention_tcgen05: this library is not built for a softmax with options");
+  return attention_tcgen05_entry(q, q_stride, k_pages, v_pages, out, q_start, kv_len, block_table, table_width, page_size, num_pages, nq, nkv, window, chunk,
+                                 softcap, scale, first_row, num_rows, max_q, skip_small, error, stream, out_stride, nullptr, gate, gate_stride, factor, slopes, sinks, gate_elements);
 }
 
 // The softmax without chunks and soft cap.

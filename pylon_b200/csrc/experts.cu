@@ -15,6 +15,12 @@
 // unit (slot_share, written by the plan), and the rows are then added up as they are.  Activation 4 is the clamped gated unit:
 // g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + 1).
 //
+// A third way (RouteScored.on 2): the scores are the softmax over all of the router's outputs; a group may be worth its largest choice
+// score; the shares may be times a factor.  The router's last outputs may be experts that hand their input back: whoever chooses one gets
+// chosen -1 and no slot, and same_share [T] receives the shares of those a token chose, for whoever adds share * h.  And behind the `top`
+// choices every token may have `always` more, the pieces of an expert that every token goes through, with a share of one; their matrices
+// lie behind the experts'.  A token's choices and shares then lie top + always apart.
+//
 // Nothing here needs the host to know how many tokens an expert got, so the step stays one sequence of launches (and
 // can be captured): the (token, choice) pairs are sorted by expert into row tiles of ROWS slots, every expert's span
 // padded to whole tiles, and the grouped products run over the most tiles there can be; a tile beyond the last one, and
@@ -61,7 +67,7 @@ __device__ __forceinline__ long long glu_row(int n, int half, int n_out, int int
 
 // The `top` largest of a token's logits (the lower index wins a tie) and the softmax over just those; one warp.  logits is spoilt.
 __device__ __forceinline__ void route_choose(float* logits, int* __restrict__ chosen, float* __restrict__ share, long long t, int experts, int top,
-                                             int lane) {
+                                             int per, int lane) {
   float first = 0.f, total = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
@@ -80,34 +86,47 @@ __device__ __forceinline__ void route_choose(float* logits, int* __restrict__ ch
     const float weight = expf(best - first);
     total += weight;
     if (lane == 0) {
-      chosen[t * top + k] = where;
-      share[t * top + k] = weight;
+      chosen[t * per + k] = where;
+      share[t * per + k] = weight;
       logits[where] = -INFINITY;
     }
     __syncwarp();
   }
   const float inv = 1.f / total;
-  if (lane < top) share[t * top + lane] *= inv;
-  for (int k = 32 + lane; k < top; k += 32) share[t * top + k] *= inv;
+  if (lane < top) share[t * per + lane] *= inv;
+  for (int k = 32 + lane; k < top; k += 32) share[t * per + k] *= inv;
 }
 
 // How the scores are made and the choice is restricted; correction null: none; groups 0: no groups.
 struct RouteScored {
-  int on;                    // 0: the softmax form above; the rest is unused then
+  int on;                    // 0: the softmax form above, the rest is unused then; 1: sigmoids; 2: the softmax over all of the router's outputs
   const float* correction;   // [experts] or null
   int groups, keep;
   float share_eps;
   int normalize;             // 0: the shares are the scores as they are
   int extra;                 // rows of the router behind the experts'
   float* extra_out;          // [T, extra]
+  int group_best;            // a group is worth its largest choice score instead of the sum of its two largest
+  float share_scale;         // on the shares
+  int real;                  // outputs from here on are experts that hand their input back: chosen is -1, the share joins same_share
+  float* same_share;         // [T] or null
 };
 
 // One warp.  logits [experts + extra] holds z; choice [experts] and worth [groups] are scratch.
 __device__ __forceinline__ void route_choose_scored(float* logits, float* choice, float* worth, int* __restrict__ chosen, float* __restrict__ share,
-                                                    long long t, int experts, int top, int lane, const RouteScored& mode) {
+                                                    long long t, int experts, int top, int per, int lane, const RouteScored& mode) {
   for (int x = lane; x < mode.extra; x += 32) mode.extra_out[t * mode.extra + x] = 1.f / (1.f + expf(-logits[experts + x]));
+  float largest = 0.f, over = 1.f;   // of the softmax over all
+  if (mode.on == 2) {
+    largest = -INFINITY;
+    for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, logits[e]);
+    largest = warp_max(largest);
+    over = 0.f;
+    for (int e = lane; e < experts; e += 32) over += expf(logits[e] - largest);
+    over = warp_sum(over);
+  }
   for (int e = lane; e < experts; e += 32) {
-    const float s = 1.f / (1.f + expf(-logits[e]));
+    const float s = mode.on == 2 ? expf(logits[e] - largest) / over : 1.f / (1.f + expf(-logits[e]));
     logits[e] = s;
     choice[e] = s + (mode.correction != nullptr ? mode.correction[e] : 0.f);
   }
@@ -121,7 +140,7 @@ __device__ __forceinline__ void route_choose_scored(float* logits, float* choice
         if (c > first) { second = first; first = c; }
         else if (c > second) second = c;
       }
-      worth[g] = size > 1 ? first + second : first;
+      worth[g] = size > 1 && !mode.group_best ? first + second : first;
     }
     __syncwarp();
     for (int k = 0; k < mode.keep; ++k) {   // the best group not yet kept, the lower index on a tie; a kept group's worth becomes +inf
@@ -143,7 +162,7 @@ __device__ __forceinline__ void route_choose_scored(float* logits, float* choice
       if (worth[e / size] != INFINITY) choice[e] = -INFINITY;
     __syncwarp();
   }
-  float total = 0.f;
+  float total = 0.f, handed_back = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int where = 0x7fffffff;
@@ -158,18 +177,21 @@ __device__ __forceinline__ void route_choose_scored(float* logits, float* choice
     }
     if (where == 0x7fffffff) where = 0;
     const float s = logits[where];
+    const bool same = where >= mode.real;
     total += s;
+    if (same) handed_back += s;
     if (lane == 0) {
-      chosen[t * top + k] = where;
-      share[t * top + k] = s;
+      chosen[t * per + k] = same ? -1 : where;
+      share[t * per + k] = mode.normalize ? s : s * mode.share_scale;
       choice[where] = -INFINITY;
     }
     __syncwarp();
   }
+  const float inv = mode.normalize ? mode.share_scale / (total + mode.share_eps) : mode.share_scale;
+  if (mode.same_share != nullptr && lane == 0) mode.same_share[t] = handed_back * inv;
   if (!mode.normalize) return;
-  const float inv = 1.f / (total + mode.share_eps);
-  if (lane < top) share[t * top + lane] *= inv;
-  for (int k = 32 + lane; k < top; k += 32) share[t * top + k] *= inv;
+  if (lane < top) share[t * per + lane] *= inv;
+  for (int k = 32 + lane; k < top; k += 32) share[t * per + k] *= inv;
 }
 
 // h [T, width] in T; router float32 [experts, width]; bias float32 [experts] or null.  chosen int32 [T, top], share float32 [T, top].
@@ -194,7 +216,7 @@ __device__ __forceinline__ void route_load(float (&x)[V], const T* from) {
 template <typename T, int TOKENS, int V>
 __global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict__ h, long long ld, const float* __restrict__ router, const float* __restrict__ bias,
                                                             int* __restrict__ chosen, float* __restrict__ share, int width, int experts, int top, int num_tokens,
-                                                            RouteScored mode) {
+                                                            int always, RouteScored mode) {
   extern __shared__ float route_shared[];
   constexpr int SIDE = 8;   // experts side by side: the tokens' rows are read once per eight experts
   const int rows = experts + mode.extra;                                        // rows of the router
@@ -243,16 +265,21 @@ __global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict_
   }
   for (int i = warp; i < TOKENS && t0 + i < num_tokens; i += 4) {
     float* mine = logits + i * per_token;
-    if (mode.on) route_choose_scored(mine, mine + rows, mine + rows + experts, chosen, share, t0 + i, experts, top, lane, mode);
-    else route_choose(mine, chosen, share, t0 + i, experts, top, lane);
+    const int per = top + always;
+    if (mode.on) route_choose_scored(mine, mine + rows, mine + rows + experts, chosen, share, t0 + i, experts, top, per, lane, mode);
+    else route_choose(mine, chosen, share, t0 + i, experts, top, per, lane);
+    for (int k = lane; k < always; k += 32) {   // the pieces every token goes through lie behind the experts
+      chosen[(long long)(t0 + i) * per + top + k] = mode.real + k;
+      share[(long long)(t0 + i) * per + top + k] = 1.f;
+    }
   }
 }
 
-// One block.  chosen [pairs]; slot_of [pairs] out; source [max_slots] out: the pair in a slot, or -1; tile_expert [max_tiles] out:
+// One block.  chosen [pairs], `per` to a token, -1: none; the last `always` experts are every token's.  slot_of [pairs] out; source [max_slots] out: the pair in a slot, or -1; tile_expert [max_tiles] out:
 // the expert of a row tile of tile_rows slots, or -1; slot_share [max_slots] out, or null: the share of the pair in a slot.  Shared memory: 2 * experts + 1 ints.
 __global__ void experts_plan_kernel(const int* __restrict__ chosen, int* __restrict__ slot_of, int* __restrict__ source,
                                     int* __restrict__ tile_expert, int pairs, int experts, int max_slots, int max_tiles, int tile_rows,
-                                    const float* __restrict__ share, float* __restrict__ slot_share) {
+                                    const float* __restrict__ share, float* __restrict__ slot_share, int per, int always) {
   extern __shared__ int plan[];
   grid_dependency_wait();
   allow_dependents();
@@ -265,7 +292,12 @@ __global__ void experts_plan_kernel(const int* __restrict__ chosen, int* __restr
   }
   for (int tile = threadIdx.x; tile < max_tiles; tile += blockDim.x) tile_expert[tile] = -1;
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&count[chosen[i]], 1);
+  const int real = experts - always;   // the pieces every token goes through: their tokens in order, nothing to count
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const int e = chosen[i];
+    if (e >= 0 && e < real) atomicAdd(&count[e], 1);
+  }
+  for (int k = threadIdx.x; k < always; k += blockDim.x) count[real + k] = pairs / per;
   __syncthreads();
   if (threadIdx.x == 0) {
     int at = 0;
@@ -282,7 +314,12 @@ __global__ void experts_plan_kernel(const int* __restrict__ chosen, int* __restr
   }
   __syncthreads();
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int slot = atomicAdd(&count[chosen[i]], 1);   // the order inside an expert's span does not matter: rows do not see each other
+    const int e = chosen[i];
+    if (e < 0) {   // handed back: no slot
+      slot_of[i] = -1;
+      continue;
+    }
+    const int slot = e >= real ? first[e] + i / per : atomicAdd(&count[e], 1);   // the order inside an expert's span does not matter: rows do not see each other
     slot_of[i] = slot;
     source[slot] = i;
     if (slot_share) slot_share[slot] = share[i];
@@ -504,11 +541,13 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
 
 // share null: the rows are added up as they are.
 // out[t, c] = sum_k share[t, k] * y[slot_of[t * top + k], c], the choices in their order; y in float32 or in the compute dtype.
+// With `same` (rows in C, same_ld apart) and same_share (float32 [T]): + same_share[t] * same[t, c].  A slot of -1 is none.
 // With `common` ([T, width] in C, an expert that every token goes through) and `gate` (float32 [T]): + gate[t] * common[t, c].
 template <typename Y, typename C>
 __global__ void experts_gather_kernel(const Y* __restrict__ y, const int* __restrict__ slot_of, const float* __restrict__ share,
                                       float* __restrict__ out, int width, int top, long long total, const C* __restrict__ common,
-                                      const float* __restrict__ gate, int parts, long long part_stride) {
+                                      const float* __restrict__ gate, int parts, long long part_stride, const C* __restrict__ same, long long same_ld,
+                                      const float* __restrict__ same_share) {
   grid_dependency_wait();
   allow_dependents();
   const long long item = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -517,12 +556,15 @@ __global__ void experts_gather_kernel(const Y* __restrict__ y, const int* __rest
   const int c = (int)(item % width);
   float acc = 0.f;
   for (int k = 0; k < top; ++k) {
-    const Y* row = y + (long long)slot_of[t * top + k] * width + c;
+    const int slot = slot_of[t * top + k];
+    if (slot < 0) continue;
+    const Y* row = y + (long long)slot * width + c;
     float value = to_float<Y>(row[0]);
     for (int part = 1; part < parts; ++part) value += to_float<Y>(row[part * part_stride]);
     acc = fmaf(share ? share[t * top + k] : 1.f, value, acc);
   }
   if (common != nullptr) acc = fmaf(gate[t], to_float<C>(common[item]), acc);
+  if (same != nullptr) acc = fmaf(same_share[t], to_float<C>(same[t * same_ld + c]), acc);
   out[item] = acc;
 }
 
@@ -546,24 +588,28 @@ using namespace pylon;
 
 extern "C" int pylon_experts_row_tile() { return EXPERT_ROWS; }
 
-// scored != 0: the sigmoid form (see RouteScored); router is then float32 [experts + extra, width].
+// scored 1: the sigmoid form, 2: the softmax over all (see RouteScored); router is then float32 [experts + extra, width].  `experts` counts the last
+// `identity` outputs, experts that hand their input back; chosen and share are [T, top + always].
 extern "C" int pylon_experts_route(const void* h, long long ld, const float* router, const float* bias, int* chosen, float* share, int width,
                                    int experts, int top, int num_tokens, int dtype, int scored, const float* correction, int groups, int keep,
-                                   float share_eps, int normalize, int extra, float* extra_out, cudaStream_t stream) {
+                                   float share_eps, int normalize, int extra, float* extra_out, int group_best, float share_scale, int identity,
+                                   float* same_share, int always, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (experts < 1 || top < 1 || top > experts || experts > 2048) PYLON_REFUSE("experts_route: %d of %d experts (at most 2048)", top, experts);
+  if (scored < 0 || scored > 2 || identity < 0 || identity >= experts || (identity > 0 && (!scored || !same_share)) || always < 0)
+    PYLON_REFUSE("experts_route: form %d, %d experts that hand their input back of %d, %d pieces for every token", scored, identity, experts, always);
   if (!scored && (correction || groups || extra)) PYLON_REFUSE("experts_route: a correction, groups and extra rows go with the sigmoid form");
   if (scored && (groups < 0 || (groups > 0 && (experts % groups || keep < 1 || keep > groups || top > keep * (experts / groups))) || extra < 0 || extra > 64 ||
                  (extra > 0 && !extra_out)))
     PYLON_REFUSE("experts_route: %d groups of which %d are kept for %d of %d experts, %d extra rows", groups, keep, top, experts, extra);
-  const RouteScored mode{scored ? 1 : 0, correction, groups, keep, share_eps, normalize, extra, extra_out};
+  const RouteScored mode{scored, correction, groups, keep, share_eps, normalize, extra, extra_out, group_best, share_scale, experts - identity, same_share};
   const int per_token = experts + extra + (scored ? experts + groups : 0);
   const bool few = num_tokens < 512;   // a step of few tokens: a block each
   const size_t element = dtype == PYLON_DTYPE_F32 ? 4 : 2;
   const bool pieces = width % 4 == 0 && ld % 4 == 0 && (uintptr_t)h % (4 * element) == 0 && (uintptr_t)router % 16 == 0;
 #define PYLON_ROUTE(T, TOKENS, V)                                                                                                            \
   launch_dependent(experts_route_kernel<T, TOKENS, V>, dim3((unsigned)((num_tokens + TOKENS - 1) / TOKENS)), dim3(128),                      \
-                   (size_t)TOKENS * (4 * 8 + per_token) * sizeof(float), stream, (const T*)h, ld, router, bias, chosen, share, width, experts, top, num_tokens, mode)
+                   (size_t)TOKENS * (4 * 8 + per_token) * sizeof(float), stream, (const T*)h, ld, router, bias, chosen, share, width, experts, top, num_tokens, always, mode)
 #define PYLON_ROUTE_SIZES(T)                                                                                                                 \
   if (few) { if (pieces) PYLON_ROUTE(T, 1, 4); else PYLON_ROUTE(T, 1, 1); }                                                                  \
   else { if (pieces) PYLON_ROUTE(T, 4, 4); else PYLON_ROUTE(T, 4, 1); }
@@ -577,13 +623,14 @@ extern "C" int pylon_experts_route(const void* h, long long ld, const float* rou
 
 // tile_rows: the slots of a row tile (pylon_experts_row_tile() for the products of this file, 128 for the grouped tcgen05 product).
 extern "C" int pylon_experts_plan(const int* chosen, int* slot_of, int* source, int* tile_expert, int pairs, int experts, int max_slots,
-                                  int max_tiles, int tile_rows, const float* share, float* slot_share, cudaStream_t stream) {
+                                  int max_tiles, int tile_rows, const float* share, float* slot_share, int per, int always, cudaStream_t stream) {
   if (pairs <= 0) return 0;
+  if (per < 1 || pairs % per || always < 0 || always >= experts || always >= per) PYLON_REFUSE("experts_plan: %d pairs, %d to a token, %d of %d experts every token's", pairs, per, always, experts);
   if (slot_share && !share) PYLON_REFUSE("experts_plan: shares per slot need the shares per choice");
   if (tile_rows < 1 || max_slots < pairs || (long long)max_tiles * tile_rows < max_slots)
     PYLON_REFUSE("experts_plan: %d slots in %d tiles of %d for %d pairs", max_slots, max_tiles, tile_rows, pairs);
   launch_dependent(experts_plan_kernel, dim3(1), dim3(1024), (size_t)(2 * experts + 1) * sizeof(int), stream, chosen, slot_of, source, tile_expert,
-                   pairs, experts, max_slots, max_tiles, tile_rows, share, slot_share);
+                   pairs, experts, max_slots, max_tiles, tile_rows, share, slot_share, per, always);
   PYLON_CHECK_LAUNCH("experts_plan");
 }
 
@@ -653,16 +700,19 @@ extern "C" int pylon_experts_sort_rows(const void* h, long long ld, const int* s
 
 // parts > 1: y is float32 [parts, slots, width], the rows' partial sums.
 // y: [slots, width] in float32 (y_dtype PYLON_DTYPE_F32) or bfloat16; out float32 [num_tokens, width].
+// same (rows same_ld apart, in common_dtype) and same_share (float32 [num_tokens]): out += same_share[t] * same[t].
 // common ([num_tokens, width] in common_dtype) and gate (float32 [num_tokens]), both or neither: out += gate[t] * common[t].
 extern "C" int pylon_experts_gather(const void* y, const int* slot_of, const float* share, float* out, int num_tokens, int width, int top, int y_dtype,
-                                    const void* common, const float* gate, int common_dtype, int parts, long long slots, cudaStream_t stream) {
+                                    const void* common, const float* gate, int common_dtype, int parts, long long slots, const void* same, long long same_ld,
+                                    const float* same_share, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (parts < 1 || (parts > 1 && (y_dtype != PYLON_DTYPE_F32 || slots < 1))) PYLON_REFUSE("experts_gather: %d parts", parts);
   if ((common == nullptr) != (gate == nullptr)) PYLON_REFUSE("experts_gather: a common expert's output and its gate go together");
   const long long total = (long long)num_tokens * width;
   const dim3 grid((unsigned)((total + 255) / 256));
-  const bool common_f32 = common == nullptr || common_dtype == PYLON_DTYPE_F32;
-#define PYLON_GATHER(Y, C) launch_dependent(experts_gather_kernel<Y, C>, grid, dim3(256), 0, stream, (const Y*)y, slot_of, share, out, width, top, total, (const C*)common, gate, parts, slots * width)
+  if (common && same) PYLON_REFUSE("experts_gather: a common expert or experts that hand their input back, not both");
+  const bool common_f32 = (common == nullptr && same == nullptr) || common_dtype == PYLON_DTYPE_F32;
+#define PYLON_GATHER(Y, C) launch_dependent(experts_gather_kernel<Y, C>, grid, dim3(256), 0, stream, (const Y*)y, slot_of, share, out, width, top, total, (const C*)common, gate, parts, slots * width, (const C*)same, same_ld, same_share)
   if (y_dtype == PYLON_DTYPE_F32) { if (common_f32) PYLON_GATHER(float, float); else PYLON_GATHER(float, __nv_bfloat16); }
   else if (y_dtype == PYLON_DTYPE_BF16) { if (common_f32) PYLON_GATHER(__nv_bfloat16, float); else PYLON_GATHER(__nv_bfloat16, __nv_bfloat16); }
   else PYLON_REFUSE("experts_gather: unknown dtype %d", y_dtype);

@@ -7,9 +7,21 @@
 // a = p * f_i comes as float32 tables cos/sin [positions, rot / 2] (any scaling of the frequencies, and
 // any factor on cos and sin, is in the tables).  Layout 0 pairs element i with i + rot / 2, layout 1
 // element 2 i with 2 i + 1, i < rot / 2; elements from `rot` on pass unchanged.  All arithmetic is float32.
+//
+// Further: the norm may run over a token's whole q row and whole k row, all heads at once (weights as long as those rows); a query may be
+// multiplied by a factor by position (q_factors [positions]); and the values may be the projected keys, biases included, as they are before
+// norm and rotation (values_from_keys: there are no value columns then).
 #include "common.cuh"
 
 namespace pylon {
+
+// norm_mode 0: no norm of q and k, 1: per head before the rotation, 2: per head after it, 3: over the whole row, before it.
+struct RotaryOptions {
+  int norm_mode;
+  int values_from_keys;
+  const float* q_factors;   // float32 [factor_positions] or null
+  int factor_positions;
+};
 
 constexpr int ROTARY_THREADS = 128;
 constexpr int ROTARY_WARPS = ROTARY_THREADS / 32;
@@ -33,29 +45,42 @@ __device__ __forceinline__ void unit_rms(float* buf, int n, int size, const floa
   for (int e = lane; e < n; e += 32) buf[e] *= weight ? inv * weight[e] : inv;
 }
 
-// One warp per (token, head of q, k or v).  qkv [T, ld] holds [q: nq x d | k: nkv x d | v: nkv x dv] per token; q is
-// written back in place, k and v go into the token's slot of its pages.  norm_mode 0: no norm of q and k; 1: before the
-// rotation; 2: after it.
-template <typename T>
+// One warp per (token, head of q, k or v); WHOLE: a block per token, whose warps take the heads in turn behind the two sums.  qkv [T, ld] holds [q: nq x d | k: nkv x d | v: nkv x dv] per token; q is
+// written back in place, k and v go into the token's slot of its pages.
+template <typename T, bool WHOLE>
 __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
     T* __restrict__ qkv, long long ld, const float* __restrict__ bias, const float* __restrict__ cos_table, const float* __restrict__ sin_table,
-    int rot, int layout, int table_positions, int norm_mode, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
+    int rot, int layout, int table_positions, RotaryOptions options, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps,
     const int* __restrict__ positions, const int* __restrict__ token_row, const int* __restrict__ block_table, int table_width, int page_size,
     T* __restrict__ k_pages, T* __restrict__ v_pages, int num_pages, int nq, int nkv, int d, int dv, int norm_size, int num_tokens, int* __restrict__ error_word) {
   extern __shared__ float rotary_shared[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int widest = d > dv ? d : dv;
   float* buf = rotary_shared + (size_t)warp * widest;
-  const int per_token = nq + 2 * nkv;
-  const long long item = (long long)blockIdx.x * ROTARY_WARPS + warp;
-  if (item >= (long long)num_tokens * per_token) return;
-  const int t = (int)(item / per_token), hh = (int)(item % per_token);
+  const int per_token = nq + 2 * nkv, norm_mode = options.norm_mode;
+  const long long item = WHOLE ? 0 : (long long)blockIdx.x * ROTARY_WARPS + warp;
+  if (!WHOLE && item >= (long long)num_tokens * per_token) return;
+  const int t = WHOLE ? (int)blockIdx.x : (int)(item / per_token);
   const int row = token_row[t];
   if (row < 0) return;   // a padding token: nothing of it is kept
   const int pos = positions[t];
+  float q_inv = 1.f, k_inv = 1.f;
+  if (WHOLE) {
+    float* scratch = rotary_shared + (size_t)ROTARY_WARPS * widest;   // [34]
+    float q_squares = 0.f, k_squares = 0.f;
+    for (int e = threadIdx.x; e < (nq + nkv) * d; e += ROTARY_THREADS) {
+      const float x = to_float<T>(qkv[(size_t)t * ld + e]) + (bias ? bias[e] : 0.f);
+      if (e < nq * d) q_squares = fmaf(x, x, q_squares);
+      else k_squares = fmaf(x, x, k_squares);
+    }
+    q_inv = rsqrtf(block_sum(q_squares, scratch) / (nq * norm_size) + eps);
+    k_inv = rsqrtf(block_sum(k_squares, scratch) / (nkv * norm_size) + eps);
+  }
+  for (int hh = WHOLE ? warp : (int)(item % per_token); hh < per_token; hh += WHOLE ? ROTARY_WARPS : per_token) {
+  __syncwarp();
   const bool is_q = hh < nq, is_v = hh >= nq + nkv;
   const int width = is_v ? dv : d;
-  const int column = is_q ? hh * d : (is_v ? (nq + nkv) * d + (hh - nq - nkv) * dv : hh * d);
+  const int column = is_q ? hh * d : (is_v ? (options.values_from_keys ? (hh - nkv) * d : (nq + nkv) * d + (hh - nq - nkv) * dv) : hh * d);
   T* src = qkv + (size_t)t * ld + column;
   for (int e = lane; e < width; e += 32) buf[e] = to_float<T>(src[e]) + (bias ? bias[column + e] : 0.f);
   __syncwarp();
@@ -63,6 +88,10 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
     const float* weight = is_q ? q_weight : k_weight;
     if (norm_mode == 1) {
       unit_rms(buf, d, norm_size, weight, eps, lane);
+      __syncwarp();
+    }
+    if (WHOLE) {
+      for (int e = lane; e < d; e += 32) buf[e] *= is_q ? q_inv * weight[column + e] : k_inv * weight[column - nq * d + e];
       __syncwarp();
     }
     if (rot > 0 && pos < table_positions) {
@@ -73,6 +102,10 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
       unit_rms(buf, d, norm_size, weight, eps, lane);
       __syncwarp();
     }
+    if (is_q && options.q_factors && pos < options.factor_positions) {
+      for (int e = lane; e < d; e += 32) buf[e] *= options.q_factors[pos];
+      __syncwarp();
+    }
   }
   T* dst = src;
   if (!is_q) {
@@ -80,15 +113,16 @@ __global__ void __launch_bounds__(ROTARY_THREADS) qkv_rotate_write_kernel(
     const int page = logical < table_width ? block_table[(size_t)row * table_width + logical] : -1;
     if (page < 0 || page >= num_pages) {
       if (lane == 0 && error_word) atomicMax(error_word, PYLON_ERROR_BAD_PAGE);
-      return;
+      continue;
     }
     const int head = is_v ? hh - nq - nkv : hh - nq;
     dst = (is_v ? v_pages : k_pages) + (((size_t)page * nkv + head) * page_size + pos % page_size) * width;
   }
   for (int e = lane; e < width; e += 32) dst[e] = from_float<T>(buf[e]);
+  }
 }
 
-// The same for bfloat16 rows without biases whose pairs lie rot / 2 apart, rot a multiple of 16.  A block takes one token; `lanes` (a power
+// The same for bfloat16 rows whose pairs lie rot / 2 apart, rot a multiple of 16.  A block takes one token; `lanes` (a power
 // of two) lanes share a head, each with 8 neighbouring elements as one 16-byte piece; the rotation partners of a lane's elements are all in
 // one other lane.  A lane meets the same elements of several heads, so it reads its angles once, and four heads' pieces are on their
 // way at once.
@@ -108,11 +142,13 @@ __device__ __forceinline__ void load_8(float (&x)[8], const float* from) {
 constexpr int ROTARY_VEC_MOST = 512;   // threads of a block at most: a step of few tokens gives every head lanes of its own
 
 __global__ void __launch_bounds__(ROTARY_VEC_MOST, 2) qkv_rotate_write_vec_kernel(
-    __nv_bfloat16* __restrict__ qkv, long long ld, const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot, int table_positions,
-    int norm_mode, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps, const int* __restrict__ positions,
+    __nv_bfloat16* __restrict__ qkv, long long ld, const float* __restrict__ bias, const float* __restrict__ cos_table, const float* __restrict__ sin_table, int rot,
+    int table_positions, RotaryOptions options, const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps, const int* __restrict__ positions,
     const int* __restrict__ token_row, const int* __restrict__ block_table, int table_width, int page_size, __nv_bfloat16* __restrict__ k_pages,
     __nv_bfloat16* __restrict__ v_pages, int num_pages, int nq, int nkv, int d, int dv, int norm_size, int lanes, int* __restrict__ error_word) {
   constexpr int SIDE = 4;                              // heads of a lane on their way at once
+  __shared__ float scratch[34];
+  const int norm_mode = options.norm_mode;
   const int t = blockIdx.x, row = token_row[t];        // position, page and angles do not depend on the kernel ahead
   if (row < 0) {                                       // a padding token: nothing of it is kept
     grid_dependency_wait();                            // a grid must not end before the grid ahead of it has
@@ -133,8 +169,34 @@ __global__ void __launch_bounds__(ROTARY_VEC_MOST, 2) qkv_rotate_write_vec_kerne
   const bool page_there = page >= 0 && page < num_pages;
   const size_t slot = (size_t)(page_there ? page : 0) * nkv * page_size + pos % page_size;
   const int lane = threadIdx.x & 31, apart = half >> 3, partner = (mine < half ? lane + apart : lane - apart) & 31;
+  const float q_factor = options.q_factors && pos < options.factor_positions ? options.q_factors[pos] : 1.f;
   grid_dependency_wait();
   allow_dependents();
+  auto column_of = [&](int hh) { return hh < nq + nkv ? hh * d : (options.values_from_keys ? (hh - nkv) * d : (nq + nkv) * d + (hh - nq - nkv) * dv); };
+  auto add_bias = [&](float (&x)[8], int hh) {
+    if (!bias) return;
+    float b[8];
+    load_8(b, bias + column_of(hh) + mine);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] += b[i];
+  };
+  float q_inv = 1.f, k_inv = 1.f;
+  if (norm_mode == 3) {                                // over the whole rows: their sums first, the pieces come from the cache the second time
+    float q_squares = 0.f, k_squares = 0.f;
+    for (int hh = group; hh < nq + nkv; hh += groups) {
+      if (mine >= d) continue;
+      float x[8];
+      unpack_8(x, *reinterpret_cast<const uint4*>(qkv + (size_t)t * ld + hh * d + mine));
+      add_bias(x, hh);
+      float squares = 0.f;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) squares = fmaf(x[i], x[i], squares);
+      if (hh < nq) q_squares += squares;
+      else k_squares += squares;
+    }
+    q_inv = rsqrtf(block_sum(q_squares, scratch) / (nq * norm_size) + eps);
+    k_inv = rsqrtf(block_sum(k_squares, scratch) / (nkv * norm_size) + eps);
+  }
   for (int h0 = 0; h0 < heads; h0 += SIDE * groups) {  // the same turns for every lane: all of a warp meet the shuffles
     uint4 raw[SIDE];
 #pragma unroll
@@ -142,7 +204,7 @@ __global__ void __launch_bounds__(ROTARY_VEC_MOST, 2) qkv_rotate_write_vec_kerne
       const int hh = h0 + k * groups + group;
       const bool is_v = hh >= nq + nkv;
       const bool live = hh < heads && mine < (is_v ? dv : d);
-      raw[k] = live ? *reinterpret_cast<const uint4*>(qkv + (size_t)t * ld + (is_v ? (nq + nkv) * d + (hh - nq - nkv) * dv : hh * d) + mine) : make_uint4(0u, 0u, 0u, 0u);
+      raw[k] = live ? *reinterpret_cast<const uint4*>(qkv + (size_t)t * ld + column_of(hh) + mine) : make_uint4(0u, 0u, 0u, 0u);
     }
 #pragma unroll
     for (int k = 0; k < SIDE; ++k) {
@@ -151,6 +213,7 @@ __global__ void __launch_bounds__(ROTARY_VEC_MOST, 2) qkv_rotate_write_vec_kerne
       const bool is_q = hh < nq, is_v = hh >= nq + nkv;
       float x[8];
       unpack_8(x, raw[k]);
+      if (hh < heads && mine < (is_v ? dv : d)) add_bias(x, hh);
       auto unit = [&]() {
         float squares = 0.f;
 #pragma unroll
@@ -168,6 +231,12 @@ __global__ void __launch_bounds__(ROTARY_VEC_MOST, 2) qkv_rotate_write_vec_kerne
         }
       };
       if (norm_mode == 1) unit();
+      if (norm_mode == 3 && !is_v && mine < d) {
+        float w[8];
+        load_8(w, is_q ? q_weight + hh * d + mine : k_weight + (hh - nq) * d + mine);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] *= (is_q ? q_inv : k_inv) * w[i];
+      }
       if (rot > 0) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
@@ -176,9 +245,17 @@ __global__ void __launch_bounds__(ROTARY_VEC_MOST, 2) qkv_rotate_write_vec_kerne
         }
       }
       if (norm_mode == 2) unit();
+      if (is_q) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] *= q_factor;
+      }
       if (hh >= heads || mine >= (is_v ? dv : d)) continue;
-      uint4 result = raw[k];                             // a value stays what it is
-      if (!is_v) {
+      uint4 result = raw[k];                             // a value without a bias stays what it is
+      if (is_v && bias) {                                // neither normed nor rotated: its own numbers again
+        unpack_8(x, raw[k]);
+        add_bias(x, hh);
+      }
+      if (!is_v || bias) {
         unsigned words[4];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
@@ -266,32 +343,39 @@ using namespace pylon;
 extern "C" int pylon_qkv_rotate_write(void* qkv, long long ld, const float* bias, const float* cos_table, const float* sin_table, int rot, int layout,
                                       int table_positions, int norm_mode, const float* q_weight, const float* k_weight, float eps, const int* positions,
                                       const int* token_row, const int* block_table, int table_width, int page_size, void* k_pages, void* v_pages,
-                                      int num_pages, int nq, int nkv, int d, int dv, int norm_size, int num_tokens, int dtype, int* error_word, cudaStream_t stream) {
+                                      int num_pages, int nq, int nkv, int d, int dv, int norm_size, int num_tokens, int dtype, int* error_word, int values_from_keys,
+                                      const float* q_factors, int factor_positions, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
+  if (values_from_keys && dv != d) PYLON_REFUSE("qkv_rotate_write: values of %d that are keys of %d", dv, d);
+  if (norm_mode == 3 && (!q_weight || !k_weight)) PYLON_REFUSE("qkv_rotate_write: a norm over whole rows needs its weights");
+  const RotaryOptions options{norm_mode, values_from_keys, q_factors, factor_positions};
   if (norm_size < 1 || norm_size > d) PYLON_REFUSE("qkv_rotate_write: a norm over %d of %d elements", norm_size, d);
   if (nq < 1 || nkv < 1 || d < 1 || dv < 1 || d > 2048 || dv > 2048) PYLON_REFUSE("qkv_rotate_write: %d / %d heads of %d and %d", nq, nkv, d, dv);
   if (rot < 0 || rot > d || rot % 2 || (rot > 0 && (!cos_table || !sin_table))) PYLON_REFUSE("qkv_rotate_write: %d rotated elements of %d", rot, d);
-  if (norm_mode < 0 || norm_mode > 2 || page_size < 1 || table_width < 1) PYLON_REFUSE("qkv_rotate_write: norm mode %d, page size %d, table width %d", norm_mode, page_size, table_width);
+  if (norm_mode < 0 || norm_mode > 3 || page_size < 1 || table_width < 1) PYLON_REFUSE("qkv_rotate_write: norm mode %d, page size %d, table width %d", norm_mode, page_size, table_width);
   const long long items = (long long)num_tokens * (nq + 2 * nkv);
-  const unsigned blocks = (unsigned)((items + ROTARY_WARPS - 1) / ROTARY_WARPS);
-  const size_t smem = (size_t)ROTARY_WARPS * (d > dv ? d : dv) * sizeof(float);
-  if (dtype == PYLON_DTYPE_F32)
-    qkv_rotate_write_kernel<float><<<blocks, ROTARY_THREADS, smem, stream>>>(
-        (float*)qkv, ld, bias, cos_table, sin_table, rot, layout, table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row, block_table,
-        table_width, page_size, (float*)k_pages, (float*)v_pages, num_pages, nq, nkv, d, dv, norm_size, num_tokens, error_word);
-  else if (dtype == PYLON_DTYPE_BF16 && !bias && layout == 0 && rot % 16 == 0 && d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && ld % 8 == 0 &&
+  const bool whole = norm_mode == 3;
+  const unsigned blocks = whole ? (unsigned)num_tokens : (unsigned)((items + ROTARY_WARPS - 1) / ROTARY_WARPS);
+  const size_t smem = ((size_t)ROTARY_WARPS * (d > dv ? d : dv) + 34) * sizeof(float);
+#define PYLON_ROTATE_WRITE(T, WHOLE)                                                                                                                     \
+  qkv_rotate_write_kernel<T, WHOLE><<<blocks, ROTARY_THREADS, smem, stream>>>(                                                                           \
+      (T*)qkv, ld, bias, cos_table, sin_table, rot, layout, table_positions, options, q_weight, k_weight, eps, positions, token_row, block_table,        \
+      table_width, page_size, (T*)k_pages, (T*)v_pages, num_pages, nq, nkv, d, dv, norm_size, num_tokens, error_word)
+  if (dtype == PYLON_DTYPE_F32) {
+    if (whole) PYLON_ROTATE_WRITE(float, true); else PYLON_ROTATE_WRITE(float, false);
+  } else if (dtype == PYLON_DTYPE_BF16 && layout == 0 && (uintptr_t)bias % 16 == 0 && rot % 16 == 0 && d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && ld % 8 == 0 &&
            (uintptr_t)qkv % 16 == 0 && (uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0 && (uintptr_t)cos_table % 16 == 0 && (uintptr_t)sin_table % 16 == 0 &&
            (uintptr_t)q_weight % 16 == 0 && (uintptr_t)k_weight % 16 == 0) {
     int lanes = 1;
     while (lanes * 8 < (d > dv ? d : dv)) lanes *= 2;
     const int threads = num_tokens <= 148 ? ROTARY_VEC_MOST : ROTARY_THREADS;
-    launch_dependent(qkv_rotate_write_vec_kernel, dim3((unsigned)num_tokens), dim3(threads), 0, stream, (__nv_bfloat16*)qkv, ld, cos_table, sin_table, rot,
-                     table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row, block_table, table_width, page_size, (__nv_bfloat16*)k_pages,
+    launch_dependent(qkv_rotate_write_vec_kernel, dim3((unsigned)num_tokens), dim3(threads), 0, stream, (__nv_bfloat16*)qkv, ld, bias, cos_table, sin_table, rot,
+                     table_positions, options, q_weight, k_weight, eps, positions, token_row, block_table, table_width, page_size, (__nv_bfloat16*)k_pages,
                      (__nv_bfloat16*)v_pages, num_pages, nq, nkv, d, dv, norm_size, lanes, error_word);
-  } else if (dtype == PYLON_DTYPE_BF16)
-    qkv_rotate_write_kernel<__nv_bfloat16><<<blocks, ROTARY_THREADS, smem, stream>>>(
-        (__nv_bfloat16*)qkv, ld, bias, cos_table, sin_table, rot, layout, table_positions, norm_mode, q_weight, k_weight, eps, positions, token_row,
-        block_table, table_width, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages, nq, nkv, d, dv, norm_size, num_tokens, error_word);
+  } else if (dtype == PYLON_DTYPE_BF16) {
+    if (whole) PYLON_ROTATE_WRITE(__nv_bfloat16, true); else PYLON_ROTATE_WRITE(__nv_bfloat16, false);
+  }
+#undef PYLON_ROTATE_WRITE
   else
     PYLON_REFUSE("qkv_rotate_write: unknown dtype %d", dtype);
   PYLON_CHECK_LAUNCH("qkv_rotate_write");

@@ -208,6 +208,10 @@ _SIGNATURES = {
     "min_gru.cu": {
         "pylon_min_gru": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_int, c_int, c_int, c_void_p],
     },
+    "join_norm.cu": {
+        "pylon_join_norm": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p,
+                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
+    },
     "output_norm.cu": {
         "pylon_output_norm": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
     },
@@ -227,12 +231,13 @@ _SIGNATURES = {
     "experts.cu": {
         "pylon_experts_row_tile": [],
         "pylon_experts_route": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
-                                c_float, c_int, c_int, c_void_p, c_void_p],
-        "pylon_experts_plan": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
+                                c_float, c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_int, c_void_p],
+        "pylon_experts_plan": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "pylon_experts_product": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                   c_int, c_void_p, c_float, c_float, c_int, c_void_p],
         "pylon_experts_sort_rows": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
-        "pylon_experts_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p],
+        "pylon_experts_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p,
+                                 c_longlong, c_void_p, c_void_p],
     },
     "gemm_f32.cu": {
         "pylon_gemm_f32_nt": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_void_p],
@@ -251,7 +256,8 @@ _SIGNATURES = {
     },
     "rotary.cu": {
         "pylon_qkv_rotate_write": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
-                                   c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+                                   c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int,
+                                   c_void_p],
         "pylon_latent_norm_rotate_write": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int,
                                            c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "pylon_rotate_heads": [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
@@ -282,7 +288,7 @@ _SIGNATURES = {
         "pylon_paged_attention_simple": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
                                          c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_longlong, c_float,
-                                         c_longlong, c_void_p],
+                                         c_longlong, c_void_p, c_int, c_void_p],
     },
     "attention_window.cu": {
         "pylon_window_attention": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
@@ -299,7 +305,10 @@ _SIGNATURES = {
                                              c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "pylon_paged_attention_mma_sigmoid": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                               c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int,
-                                              c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_float, c_longlong, c_void_p],
+                                              c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_longlong, c_void_p],
+        "pylon_paged_attention_mma_options": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                              c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int,
+                                              c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_longlong, c_void_p],
         "pylon_attention_scratch_floats": [c_int, c_int, c_int, c_int, c_int, c_int],
         "pylon_attention_decode_blocks": [],
     },
@@ -310,7 +319,10 @@ _SIGNATURES = {
                                                  c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "pylon_paged_attention_tcgen05_sigmoid": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                                   c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-                                                  c_void_p, c_longlong, c_float, c_longlong, c_void_p],
+                                                  c_void_p, c_longlong, c_int, c_float, c_longlong, c_void_p],
+        "pylon_paged_attention_tcgen05_options": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                                  c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p,
+                                                  c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_float, c_longlong, c_void_p],
     },
     "sampling.cu": {
         "pylon_sample": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
@@ -436,13 +448,67 @@ def add_rmsnorm(
 
 @dataclass(frozen=True)
 class ScatteredRows:
-    """A block ``[T, width]`` that is not put together yet: token t's row is the sum over k < ``top`` of the rows ``slot_of[t * top + k]``, each
-    times ``share[t, k]`` (None: as they are).  ``rows``: ``[slots, width]`` in the compute dtype, or float32 ``[parts, slots, width]`` partial sums."""
+    """A block ``[T, width]`` that is not put together yet: token t's row is the sum over k < ``top`` of the rows ``slot_of[t * top + k]`` (-1:
+    none), each times ``share[t, k]`` (None: as they are), plus ``same_share[t]`` times row t of ``same`` where given.  ``rows``: ``[slots, width]`` in
+    the compute dtype, or float32 ``[parts, slots, width]`` partial sums; ``same [T, width]`` in the compute dtype."""
 
     rows: torch.Tensor
     slot_of: torch.Tensor
     top: int
     share: Optional[torch.Tensor]
+    same: Optional[torch.Tensor] = None
+    same_share: Optional[torch.Tensor] = None
+
+
+@dataclass(frozen=True)
+class SideBySide:
+    """What two sublayers leave for the stream: ``output`` (``[T, width]`` in the compute dtype or float32 partial sums ``[parts, T, width]``), a
+    float32 vector ``bias [width]`` on every row of it, and ``rows``, a second output in either form or as :class:`ScatteredRows`.  The last two may
+    be missing."""
+
+    output: torch.Tensor
+    bias: Optional[torch.Tensor] = None
+    rows: Union[torch.Tensor, ScatteredRows, None] = None
+
+
+def join_norm(residual: torch.Tensor, joined: SideBySide, weight: Optional[torch.Tensor] = None, eps: float = 0.0, dtype: Optional[torch.dtype] = None,
+              rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """``residual += output + bias + rows`` in float32, in place, then RMSNorm of the sum times the float32 ``weight [width]`` in ``dtype``
+    (without a weight: nothing is normed or returned).  With ``rows`` (int32) only those tokens are normed, and ``residual`` stays as it is."""
+    output, bias, second = joined.output, joined.bias, joined.rows
+    slot_of = share = same = same_share = None
+    top, second_rows = 1, residual.shape[0]
+    if isinstance(second, ScatteredRows):
+        slot_of, share, top, same, same_share, second = second.slot_of, second.share, second.top, second.same, second.same_share, second.rows
+        second_rows = second.shape[-2]
+        _need(slot_of.dtype == torch.int32 and slot_of.is_contiguous() and slot_of.numel() == residual.shape[0] * top, "join_norm: slot_of must be int32 [T, top]")
+        _need(share is None or (share.dtype == torch.float32 and share.is_contiguous() and share.numel() == slot_of.numel()), "join_norm: share must be float32 [T, top]")
+    _need_cuda(residual, output, bias, second, slot_of, share, same, same_share, weight, rows)
+    _need(residual.dtype == torch.float32 and residual.dim() == 2 and residual.is_contiguous(), "join_norm: residual must be contiguous float32 [T, width]")
+    tokens, width = residual.shape
+    dtypes = {block.dtype for block in (output, second) if block is not None and block.dim() == 2} | ({same.dtype} if same is not None else set()) | ({dtype} if weight is not None else set())
+    _need(len(dtypes) <= 1, "join_norm: the blocks and the result are of one dtype")
+    dtype = dtypes.pop() if dtypes else torch.float32
+    for block, count in ((output, tokens), (second, second_rows)):
+        _need(block is None or (block.dim() in (2, 3) and block.is_contiguous() and block.shape[-2:] == (count, width) and (block.dim() == 2 or block.dtype == torch.float32)),
+              "join_norm: an output must be contiguous [T, width] in the compute dtype or float32 [parts, T, width]")
+    for vector in (bias, weight):
+        _need(vector is None or (vector.dtype == torch.float32 and vector.shape == (width,) and vector.is_contiguous()), "join_norm: bias and weight must be float32 [width]")
+    _need((same is None) == (same_share is None) and (same is None or (same.shape == (tokens, width) and same.stride(1) == 1 and same_share.dtype == torch.float32
+                                                                       and same_share.shape == (tokens,) and same_share.is_contiguous())),
+          "join_norm: rows handed back must be [T, width] with float32 [T] shares")
+    n_rows, out = tokens, None
+    if rows is not None:
+        _need(weight is not None and rows.dtype == torch.int32 and rows.dim() == 1 and rows.is_contiguous(), "join_norm: rows must be contiguous int32, and need a norm")
+        n_rows = rows.shape[0]
+    if weight is not None:
+        out = torch.empty((n_rows, width), dtype=dtype, device=residual.device)
+    library = _library("join_norm.cu")
+    _check(library, library.pylon_join_norm(
+        _ptr(residual), _ptr(output), output.shape[0] if output.dim() == 3 else 0, _ptr(bias), _ptr(second), second.shape[0] if second is not None and second.dim() == 3 else 0,
+        second_rows, _ptr(slot_of), _ptr(share), top, _ptr(same), 0 if same is None else same.stride(0), _ptr(same_share), _ptr(weight), _ptr(rows), _ptr(out),
+        n_rows, tokens, width, float(eps), _dtype_code(dtype), _stream()))
+    return out
 
 
 def output_norm(residual: torch.Tensor, output: Union[torch.Tensor, ScatteredRows], weight: torch.Tensor, eps: float, dtype: torch.dtype) -> torch.Tensor:
@@ -451,6 +517,7 @@ def output_norm(residual: torch.Tensor, output: Union[torch.Tensor, ScatteredRow
     slot_of = share = None
     top, slots = 1, 0
     if isinstance(output, ScatteredRows):
+        _need(output.same is None, "output_norm: no rows handed back")
         slot_of, share, top, slots, output = output.slot_of, output.share, output.top, output.rows.shape[-2], output.rows
         _need(slot_of.dtype == torch.int32 and slot_of.is_contiguous() and slot_of.numel() == residual.shape[0] * top, "output_norm: slot_of must be int32 [T, top]")
         _need(share is None or (share.dtype == torch.float32 and share.is_contiguous() and share.numel() == slot_of.numel()), "output_norm: share must be float32 [T, top]")
@@ -950,15 +1017,22 @@ def paged_attention(
     score_bias: Optional[torch.Tensor] = None,
     head_gate: Optional[torch.Tensor] = None,
     out_factor: float = 1.0,
+    distance_slopes: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """Causal attention of every token of a step over its request's pages.
 
-    ``split_weights`` (latent rows on the tensor cores): a softmax weight enters the weighted sum as two bfloat16 numbers, the rounded
+    ``split_weights`` (softmax weights on the tensor cores): a weight enters the weighted sum as two bfloat16 numbers, the rounded
     weight and what the rounding dropped, so that it counts with 16 bits instead of 8, at twice the products over the values.
 
+    ``distance_slopes`` (float32 ``[nq]``, softmax weights): the scaled (and capped) score of the key ``p - j`` positions back loses
+    ``distance_slopes[h] * (p - j)``.  Slopes, gated outputs, a factor and an ``out`` that is a slice of wider rows, and sinks with any of these or
+    with ``split_weights``, run in bfloat16 on the tensor-core kernels built for a softmax with options (weights split as above), for values as wide
+    as the keys, a multiple of 16 up to 256; else on the plain kernel.
+
     ``weighting="sigmoid"``: the weight of a visible key is ``sigmoid(score + score_bias[h])`` (float32 ``[nq]``, or None) and nothing is
-    divided by a sum over the keys.  Then ``head_gate`` (``[T, nq]`` in the cache dtype, any row stride) multiplies head h of token t by
-    ``sigmoid(head_gate[t, h])``, ``out_factor`` multiplies everything, and ``out`` may be a slice of wider rows.  On the tensor cores
+    divided by a sum over the keys.  ``head_gate`` (with either weighting; ``[T, nq]`` in the cache dtype, any row stride) multiplies head h of token t by
+    ``sigmoid(head_gate[t, h])``, or as ``[T, nq * value width]`` (and more than one value to a head) element by element; ``out_factor`` multiplies
+    everything, and ``out`` may be a slice of wider rows.  On the tensor cores
     (values as wide as the keys, a multiple of 16 up to 256) the same kernels run as for the softmax, built for sigmoid weights; a
     weight enters the weighted sum as two bfloat16 numbers, the rounded weight and what the rounding dropped.
 
@@ -999,7 +1073,7 @@ def paged_attention(
     else on ``mma.sync``; decoded tokens on their own kernel.  float32, and other head sizes up
     to 512, take the plain kernel.
     """
-    _need_cuda(q, k_pages, v_pages, positions, token_row, q_start, kv_len, block_table, out, sinks, distance_bias)
+    _need_cuda(q, k_pages, v_pages, positions, token_row, q_start, kv_len, block_table, out, sinks, distance_bias, distance_slopes)
     _need(sinks is None or (sinks.dtype == torch.float32 and sinks.shape == (nq,) and sinks.is_contiguous()), "paged_attention: sinks must be float32 [nq]")
     _need(distance_bias is None or (distance_bias.dtype == torch.float32 and distance_bias.dim() == 2 and distance_bias.shape[0] >= 1 and distance_bias.shape[1] == nq
                                     and distance_bias.is_contiguous()), "paged_attention: distance_bias must be contiguous float32 [rows, nq]")
@@ -1030,19 +1104,30 @@ def paged_attention(
     if out is None:
         out = torch.empty((tokens, nq * dv), dtype=q.dtype, device=q.device)
     sigmoid = weighting == "sigmoid"
+    plain_out = head_gate is None and out_factor == 1.0 and out.is_contiguous()
+    options = not sigmoid and (distance_slopes is not None or not plain_out or split_weights)
+    gate_elements = head_gate is not None and head_gate.shape[-1] == nq * dv and dv > 1
     _need(weighting in ("softmax", "sigmoid"), f"paged_attention: unknown weighting {weighting!r}")
-    _need(out.shape == (tokens, nq * dv) and out.dtype == q.dtype and out.stride(1) == 1 and (sigmoid or out.is_contiguous()), "paged_attention: out has the wrong shape or dtype")
-    _need(sigmoid or (score_bias is None and head_gate is None and out_factor == 1.0), "paged_attention: a number per head on the scores, gated heads and a factor go with sigmoid weights")
-    _need(not sigmoid or (sinks is None and not plain_only), "paged_attention: no sink, kept first keys and bias by distance with sigmoid weights")
+    _need(out.shape == (tokens, nq * dv) and out.dtype == q.dtype and out.stride(1) == 1, "paged_attention: out has the wrong shape or dtype")
+    _need(sigmoid or score_bias is None, "paged_attention: a number per head on the scores goes with sigmoid weights")
+    _need(not sigmoid or (sinks is None and distance_slopes is None and not plain_only), "paged_attention: no sink, kept first keys, bias by distance and slopes with sigmoid weights")
+    _need(not options or not plain_only, "paged_attention: no slopes, gated outputs, factor or split weights beside kept first keys and a bias by distance")
+    _need(distance_slopes is None or (distance_slopes.dtype == torch.float32 and distance_slopes.shape == (nq,) and distance_slopes.is_contiguous()), "paged_attention: distance_slopes must be float32 [nq]")
     _need_cuda(score_bias, head_gate)
     _need(score_bias is None or (score_bias.dtype == torch.float32 and score_bias.shape == (nq,) and score_bias.is_contiguous()), "paged_attention: score_bias must be float32 [nq]")
-    _need(head_gate is None or (head_gate.dtype == q.dtype and head_gate.shape == (tokens, nq) and head_gate.stride(1) == 1), "paged_attention: head_gate must be [T, nq] in the cache dtype")
+    _need(head_gate is None or (head_gate.dtype == q.dtype and head_gate.shape in ((tokens, nq), (tokens, nq * dv)) and head_gate.stride(1) == 1),
+          "paged_attention: head_gate must be [T, nq] or [T, nq * value width] in the cache dtype")
     scale = 1.0 / math.sqrt(d) if scale is None else float(scale)
     _need(scale > 0 or sigmoid, "paged_attention: the softmax scale must be positive")
-    if q.dtype == torch.bfloat16 and d % 16 == 0 and d <= 256 and not force_simple and same_width and sinks is None and not plain_only \
-            and (not sigmoid or (scale > 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0)):
-        defines = {"PYLON_HEAD_DIM": d, **({"PYLON_SIGMOID_WEIGHTS": 1} if sigmoid else {})}
-        extra = (_ptr(score_bias), _ptr(head_gate), 0 if head_gate is None else head_gate.stride(0), float(out_factor), out.stride(0)) if sigmoid else ()
+    if q.dtype == torch.bfloat16 and d % 16 == 0 and d <= 256 and not force_simple and same_width and (sinks is None or options) and not plain_only \
+            and (not (sigmoid or options) or (scale > 0 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0
+                                              and (not gate_elements or (head_gate.stride(0) % 8 == 0 and head_gate.data_ptr() % 16 == 0)))):
+        defines = {"PYLON_HEAD_DIM": d, **({"PYLON_SIGMOID_WEIGHTS": 1} if sigmoid else {"PYLON_SOFTMAX_OPTIONS": 1} if options else {})}
+        extra, form = (), "masked"
+        if sigmoid or options:
+            form = "sigmoid" if sigmoid else "options"
+            extra = (*((_ptr(score_bias),) if sigmoid else (_ptr(distance_slopes), _ptr(sinks))), _ptr(head_gate), 0 if head_gate is None else head_gate.stride(0),
+                     int(gate_elements), float(out_factor), out.stride(0))
         library = _library("attention_mma.cu", defines)
         group = nq // nkv
         any_large = max_q * group > 16
@@ -1063,7 +1148,7 @@ def paged_attention(
                 large = [index for index, count in enumerate(row_tokens) if count * group > 16]
                 if large and large[-1] - large[0] + 1 == len(large):   # one run of rows: the scheduler puts decoded rows first
                     first_row, row_count = large[0], len(large)
-            entry = fast.pylon_paged_attention_tcgen05_sigmoid if sigmoid else fast.pylon_paged_attention_tcgen05_masked
+            entry = getattr(fast, f"pylon_paged_attention_tcgen05_{form}")
             _check(fast, entry(
                 _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(q_start), _ptr(kv_len), _ptr(block_table),
                 block_table.shape[1], page_size, num_pages, nq, nkv, int(window or 0), int(chunk or 0), float(softcap or 0.0), scale,
@@ -1082,14 +1167,14 @@ def paged_attention(
             scratch = torch.empty((floats,), dtype=torch.float32, device=q.device)
         if blocks:
             counters = _zeroed_counters(q.device, "attention", rows * nkv)
-        entry = library.pylon_paged_attention_mma_sigmoid if sigmoid else library.pylon_paged_attention_mma_masked
+        entry = getattr(library, f"pylon_paged_attention_mma_{form}")
         _check(library, entry(
             _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(scratch), _ptr(counters), _ptr(q_start), _ptr(kv_len),
             _ptr(block_table), block_table.shape[1], page_size, num_pages, nq, nkv, int(window or 0), int(chunk or 0), float(softcap or 0.0),
             scale, rows, tokens,
             int(max_q), splits, blocks, int(use_tcgen05), int(bool(rows_alike)), _ptr(attention_error_word(q.device)), *extra, _stream()))
         return out
-    if ((plain_only or sinks is not None) and q.dtype == torch.bfloat16 and not force_simple and chunk is None and softcap is None and d % 16 == 0 and d <= 256 and dv % 8 == 0 and dv <= 256
+    if ((plain_only or sinks is not None) and not options and q.dtype == torch.bfloat16 and not force_simple and chunk is None and softcap is None and d % 16 == 0 and d <= 256 and dv % 8 == 0 and dv <= 256
             and nq // nkv <= 8 and q.stride(0) % 2 == 0 and q.data_ptr() % 4 == 0):
         library = _library("attention_window.cu", {"PYLON_HEAD_DIM": d, "PYLON_VALUE_DIM": dv})
         splits = window_attention_splits(rows, nkv, max_q, max_kv, window, keep_first, _multiprocessors(q.device)) if num_splits is None else int(num_splits)
@@ -1109,7 +1194,8 @@ def paged_attention(
         _ptr(q), q.stride(0), _ptr(k_pages), _ptr(v_pages), _ptr(out), _ptr(positions), _ptr(token_row), _ptr(block_table),
         block_table.shape[1], page_size, num_pages, nq, nkv, d, dv, int(window or 0), int(chunk or 0), float(softcap or 0.0), scale,
         _ptr(sinks), 0, 0, tokens, _dtype_code(q.dtype), int(keep_first), _ptr(distance_bias), 0 if distance_bias is None else distance_bias.shape[0],
-        int(sigmoid), _ptr(score_bias), _ptr(head_gate), 0 if head_gate is None else head_gate.stride(0), float(out_factor), out.stride(0), _stream()))
+        int(sigmoid), _ptr(score_bias), _ptr(head_gate), 0 if head_gate is None else head_gate.stride(0), float(out_factor), out.stride(0),
+        _ptr(distance_slopes), int(gate_elements), _stream()))
     return out
 
 
@@ -1172,7 +1258,7 @@ def _latent_attention(q, pages, dv, positions, token_row, q_start, kv_len, block
     _check(library, library.pylon_paged_attention_simple(
         _ptr(q), q.stride(0), _ptr(pages), _ptr(pages), _ptr(out), _ptr(positions), _ptr(token_row), _ptr(block_table),
         block_table.shape[1], page_size, num_pages, nq, 1, d, dv, int(window or 0), 0, 0.0, float(scale),
-        _ptr(sinks), d, d, tokens, _dtype_code(q.dtype), 0, None, 0, 0, None, None, 0, 1.0, 0, _stream()))
+        _ptr(sinks), d, d, tokens, _dtype_code(q.dtype), 0, None, 0, 0, None, None, 0, 1.0, 0, None, 0, _stream()))
     return out
 
 
@@ -1657,7 +1743,8 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
                    top: int, activation: str = "silu", interleaved: bool = False, gated: bool = True, routing: str = "softmax",
                    correction: Optional[torch.Tensor] = None, groups: int = 0, groups_keep: int = 0, share_eps: float = 0.0,
                    common_up: Optional[torch.Tensor] = None, common_down: Optional[torch.Tensor] = None, share_normalized: bool = True,
-                   weigh: str = "output", limit: Optional[float] = None, alpha: float = 1.702, scattered: bool = False) -> Union[torch.Tensor, "ScatteredRows"]:
+                   weigh: str = "output", limit: Optional[float] = None, alpha: float = 1.702, scattered: bool = False, group_score: str = "two",
+                   share_scale: float = 1.0, identity: int = 0, always: int = 0) -> Union[torch.Tensor, "ScatteredRows"]:
     """``sum over a token's top experts e of share_e * W_down,e (act(W_gate,e h) * (W_up,e h))`` (``csrc/experts.cu``).
 
     ``h [T, width]``; ``router`` float32 ``[experts, width]`` and ``router_bias`` float32 ``[experts]`` (or None): the logits are
@@ -1677,6 +1764,11 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     ``activation="clamped"`` with a ``limit``: the clamped gated unit of :func:`swiglu`.  ``scattered=True`` (no common expert): the experts'
     rows are handed on where they lie, as :class:`ScatteredRows`, for a reader that adds them up itself.
 
+    ``routing="softmax_all"``: the scores are the softmax over all of the router's outputs, the rest as with sigmoids.  ``group_score="best"``: a group
+    is worth its largest choice score.  ``share_scale`` on the shares.  ``identity`` n: the router has n outputs behind the experts', each handing
+    ``h`` itself back times its share; groups, correction and top count them.  ``always`` m: the last m of the stacked experts have no router output,
+    and every token goes through them with a share of one.
+
     The tokens are sorted by expert on the device.  A step of few tokens runs the experts' products from row tiles of 32 slots that
     gather their rows themselves (``mma.sync``, bound by the matrices coming from memory); a bfloat16 step with about half a
     128-row tile or more per expert (gated: interleaved weights and ``silu``) copies the rows into their sorted order and runs both
@@ -1687,34 +1779,39 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     _need(activation in ACTIVATIONS or clamped, f"expert_mixture: activation {activation!r}")
     _need(clamped == (limit is not None) and (not clamped or (gated and limit > 0)), "expert_mixture: a clamped unit is gated and has a positive limit")
     _need(weigh in ("output", "input") and (weigh == "output" or gated), "expert_mixture: shares weigh a gated expert's output or its input")
-    _need(routing in ("softmax", "sigmoid"), f"expert_mixture: routing {routing!r}")
+    _need(routing in ("softmax", "sigmoid", "softmax_all") and group_score in ("two", "best"), f"expert_mixture: routing {routing!r}, groups worth their {group_score!r}")
     _need(h.dim() == 2 and h.stride(1) == 1, "expert_mixture: h must be [T, width]")
     tokens, width = h.shape
     halves = 2 if gated else 1
     experts, inner = w_gate_up.shape[0], w_gate_up.shape[1] // halves
     _need(w_gate_up.shape == (experts, halves * inner, width) and w_down.shape == (experts, width, inner) and w_gate_up.is_contiguous() and w_down.is_contiguous()
           and w_gate_up.dtype == h.dtype and w_down.dtype == h.dtype, "expert_mixture: w_gate_up [experts, 2 F, width] (ungated: [experts, F, width]) and w_down [experts, width, F] in h's dtype")
-    scored = routing == "sigmoid"
+    scored = {"softmax": 0, "sigmoid": 1, "softmax_all": 2}[routing]
+    _need(0 <= always < experts and identity >= 0, f"expert_mixture: {always} of {experts} experts every token's, {identity} that hand their input back")
+    choices, per = experts - always + identity, top + always   # the router's outputs; what a token goes through
     extra = 1 if common_up is not None else 0
-    _need(scored or share_normalized, "expert_mixture: shares that do not add up to one go with sigmoid routing")
-    _need(scored or (correction is None and not groups and not extra), "expert_mixture: a correction, groups and a common expert go with sigmoid routing")
-    _need(router.dtype == torch.float32 and router.shape == (experts + extra, width) and router.is_contiguous(), "expert_mixture: router must be float32 [experts (+ 1), width]")
-    _need(router_bias is None or (router_bias.dtype == torch.float32 and router_bias.shape == (experts,)), "expert_mixture: router_bias must be float32 [experts]")
-    _need(correction is None or (correction.dtype == torch.float32 and correction.shape == (experts,) and correction.is_contiguous()), "expert_mixture: correction must be float32 [experts]")
-    _need(1 <= top <= experts, f"expert_mixture: top {top} of {experts} experts")
+    _need(scored or share_normalized, "expert_mixture: shares that do not add up to one go with scores over all experts")
+    _need(scored or (correction is None and not groups and not extra and not identity and share_scale == 1.0),
+          "expert_mixture: a correction, groups, a common expert, a factor and experts that hand their input back go with scores over all experts")
+    _need(not (identity or always) or (weigh == "output" and not extra), "expert_mixture: experts that hand their input back or are every token's: weighed on their output, without a common expert")
+    _need(router.dtype == torch.float32 and router.shape == (choices + extra, width) and router.is_contiguous(), "expert_mixture: router must be float32 [choices (+ 1), width]")
+    _need(router_bias is None or (router_bias.dtype == torch.float32 and router_bias.shape == (choices,)), "expert_mixture: router_bias must be float32 [choices]")
+    _need(correction is None or (correction.dtype == torch.float32 and correction.shape == (choices,) and correction.is_contiguous()), "expert_mixture: correction must be float32 [choices]")
+    _need(1 <= top <= choices, f"expert_mixture: top {top} of {choices} experts")
     _need(not interleaved or (gated and inner % 8 == 0), "expert_mixture: interleaved rows need a gated unit of an inner width that is a multiple of 8")
     _need((common_up is None) == (common_down is None), "expert_mixture: a common expert has both its matrices")
     _need(not scattered or common_up is None, "expert_mixture: rows cannot stay scattered beside a common expert")
     library = _library("experts.cu")
-    pairs = tokens * top
+    pairs = tokens * per
     grouped = ((not gated or (interleaved and activation in ("silu", "clamped"))) and h.dtype == torch.bfloat16 and pairs * 2 >= EXPERT_TILE_ROWS * experts and width % 8 == 0
                and inner % 8 == 0 and h.stride(0) % 8 == 0 and h.data_ptr() % 16 == 0)
     tile = EXPERT_TILE_ROWS if grouped else library.pylon_experts_row_tile()
     max_tiles = min(pairs, experts) + pairs // tile    # every expert with tokens ends in at most one partly filled tile
     max_slots = max_tiles * tile
     device = h.device
-    chosen = torch.empty((tokens, top), dtype=torch.int32, device=device)
-    share = torch.empty((tokens, top), dtype=torch.float32, device=device)
+    chosen = torch.empty((tokens, per), dtype=torch.int32, device=device)
+    share = torch.empty((tokens, per), dtype=torch.float32, device=device)
+    same, same_share = (h, torch.empty((tokens,), dtype=torch.float32, device=device)) if identity else (None, None)
     slot_of = torch.empty((pairs,), dtype=torch.int32, device=device)
     source = torch.empty((max_slots,), dtype=torch.int32, device=device)
     tile_expert = torch.empty((max_tiles,), dtype=torch.int32, device=device)
@@ -1722,12 +1819,12 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
     code, kind = _dtype_code(h.dtype), 4 if clamped else ACTIVATIONS[activation]
     slot_share = torch.empty((max_slots,), dtype=torch.float32, device=device) if weigh == "input" else None
     limit, out_share = float(limit or 0.0), share if slot_share is None else None
-    _check(library, library.pylon_experts_route(_ptr(h), h.stride(0), _ptr(router), _ptr(router_bias), _ptr(chosen), _ptr(share), width, experts, top,
-                                                tokens, code, int(scored), _ptr(correction), int(groups or 0), int(groups_keep or 0), float(share_eps), int(bool(share_normalized)), extra,
-                                                _ptr(common_gate), _stream()))
+    _check(library, library.pylon_experts_route(_ptr(h), h.stride(0), _ptr(router), _ptr(router_bias), _ptr(chosen), _ptr(share), width, choices, top,
+                                                tokens, code, scored, _ptr(correction), int(groups or 0), int(groups_keep or 0), float(share_eps), int(bool(share_normalized)), extra,
+                                                _ptr(common_gate), int(group_score == "best"), float(share_scale), identity, _ptr(same_share), always, _stream()))
     _check(library, library.pylon_experts_plan(_ptr(chosen), _ptr(slot_of), _ptr(source), _ptr(tile_expert), pairs, experts, max_slots, max_tiles, tile,
-                                               _ptr(share), _ptr(slot_share), _stream()))
-    common, common_code = None, F32
+                                               _ptr(share), _ptr(slot_share), per, always, _stream()))
+    common, common_code = None, code if identity else F32
     if extra:   # the expert of every token: two plain products around the activation
         common = linear(activation_in_place(linear(h, common_up), activation), common_down)
         common_code = _dtype_code(common.dtype)
@@ -1735,7 +1832,7 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
         product = _library("gemm_tcgen05.cu")
         error, sms = _ptr(tcgen05_error_word(device)), _multiprocessors(device)
         rows = torch.empty((max_slots, width), dtype=h.dtype, device=device)
-        _check(library, library.pylon_experts_sort_rows(_ptr(h), h.stride(0), _ptr(source), _ptr(rows), width, top, max_slots, code, _stream()))
+        _check(library, library.pylon_experts_sort_rows(_ptr(h), h.stride(0), _ptr(source), _ptr(rows), width, per, max_slots, code, _stream()))
         act = torch.empty((max_slots, inner), dtype=h.dtype, device=device)
         _check(product, product.pylon_gemm_tcgen05_grouped(_ptr(rows), _ptr(w_gate_up), _ptr(act), max_slots, halves * inner, width, width, width, inner,
                                                            1 if gated else 0, limit, float(alpha), _ptr(slot_share), _ptr(tile_expert), experts, error, sms, _stream()))
@@ -1745,23 +1842,23 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
         _check(product, product.pylon_gemm_tcgen05_grouped(_ptr(act), _ptr(w_down), _ptr(y), max_slots, width, inner, inner, inner, width, 0, 0.0, 1.0, None,
                                                            _ptr(tile_expert), experts, error, sms, _stream()))
         if scattered:
-            return ScatteredRows(y, slot_of, top, out_share)
+            return ScatteredRows(y, slot_of, per, out_share, same, same_share)
         out = torch.empty((1, tokens, width), dtype=torch.float32, device=device)
-        _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, top, code, _ptr(common), _ptr(common_gate),
-                                                     common_code, 1, 0, _stream()))
+        _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, per, code, _ptr(common), _ptr(common_gate),
+                                                     common_code, 1, 0, _ptr(same), 0 if same is None else same.stride(0), _ptr(same_share), _stream()))
         return out
     act = torch.empty((max_slots, inner), dtype=h.dtype, device=device)
-    _check(library, library.pylon_experts_product(_ptr(h), h.stride(0), _ptr(w_gate_up), _ptr(source), _ptr(tile_expert), 1, top, _ptr(act), inner, width,
+    _check(library, library.pylon_experts_product(_ptr(h), h.stride(0), _ptr(w_gate_up), _ptr(source), _ptr(tile_expert), 1, per, _ptr(act), inner, width,
                                                   max_tiles, 1 if gated else 2, kind, int(interleaved), code, _ptr(slot_share), limit, float(alpha), 1, _stream()))
     parts = _expert_parts(experts, width, inner, _multiprocessors(device)) if h.dtype == torch.bfloat16 else 1
     y = torch.empty((parts, max_slots, width), dtype=torch.float32, device=device)
     _check(library, library.pylon_experts_product(_ptr(act), inner, _ptr(w_down), _ptr(source), _ptr(tile_expert), 0, 1, _ptr(y), width, inner,
                                                   max_tiles, 0, kind, 0, code, None, 0.0, 1.0, parts, _stream()))
     if scattered:
-        return ScatteredRows(y, slot_of, top, out_share)
+        return ScatteredRows(y, slot_of, per, out_share, same, same_share)
     out = torch.empty((1, tokens, width), dtype=torch.float32, device=device)
-    _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, top, _dtype_code(torch.float32), _ptr(common),
-                                                 _ptr(common_gate), common_code, parts, max_slots, _stream()))
+    _check(library, library.pylon_experts_gather(_ptr(y), _ptr(slot_of), _ptr(out_share), _ptr(out), tokens, width, per, _dtype_code(torch.float32), _ptr(common),
+                                                 _ptr(common_gate), common_code, parts, max_slots, _ptr(same), 0 if same is None else same.stride(0), _ptr(same_share), _stream()))
     return out
 
 
@@ -1828,22 +1925,29 @@ def qkv_rotate_write(
     qkv: torch.Tensor, bias: Optional[torch.Tensor], cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], rotary_dim: int, layout: str,
     norm: Optional[str], q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
     token_row: torch.Tensor, block_table: torch.Tensor, page_size: int, k_pages: torch.Tensor, v_pages: torch.Tensor, nq: int, nkv: int,
-    head_dim: int, value_dim: int, norm_size: Optional[int] = None,
+    head_dim: int, value_dim: int, norm_size: Optional[int] = None, values_from_keys: bool = False, q_factors: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """``norm_size``: how many elements of a q or k head are its own (default: all ``d``; the rest are zeros, and the mean of the norm's
     squares is over its own).  On ``qkv [T, nq * d + nkv * d + nkv * dv]``: add ``bias`` (float32, one number per column), rotate the first
     ``rotary_dim`` elements of every q and k head by the tables (``layout``: ``"halves"`` pairs element i with i + rotary_dim / 2,
     ``"neighbours"`` element 2 i with 2 i + 1), divide every q and k head by its root mean square (``norm``: ``"before"`` or
     ``"after"`` the rotation, ``None``: not at all; times ``q_weight`` / ``k_weight [d]`` where given), write q back in place and
-    k, v into the token's slot of its pages ``[pages, nkv, page_size, d]`` and ``[pages, nkv, page_size, dv]``.  Returns ``qkv``."""
-    _need_cuda(qkv, bias, cos, sin, q_weight, k_weight, positions, token_row, block_table, k_pages, v_pages)
-    tokens, columns = qkv.shape[0], nq * head_dim + nkv * head_dim + nkv * value_dim
+    k, v into the token's slot of its pages ``[pages, nkv, page_size, d]`` and ``[pages, nkv, page_size, dv]``.  Returns ``qkv``.
+
+    ``norm="whole"``: the norm runs over the whole q row and the whole k row, before the rotation, with weights ``[nq * d]`` and ``[nkv * d]``.
+    ``values_from_keys``: the values are the keys with their bias, as they are before norm and rotation, and ``qkv`` has no value columns.
+    ``q_factors`` (float32 ``[positions]``): what a query is multiplied by, by its position."""
+    _need_cuda(qkv, bias, cos, sin, q_weight, k_weight, positions, token_row, block_table, k_pages, v_pages, q_factors)
+    tokens, columns = qkv.shape[0], nq * head_dim + nkv * head_dim + (0 if values_from_keys else nkv * value_dim)
+    _need(not values_from_keys or value_dim == head_dim, "qkv_rotate_write: values that are the keys are as wide as they are")
+    _need(q_factors is None or (q_factors.dtype == torch.float32 and q_factors.dim() == 1 and q_factors.is_contiguous()), "qkv_rotate_write: q_factors must be float32 [positions]")
     _need(qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] == columns, "qkv_rotate_write: qkv must be [T, nq * d + nkv * d + nkv * dv]")
     _need(bias is None or (bias.dtype == torch.float32 and bias.shape == (columns,) and bias.is_contiguous()), "qkv_rotate_write: bias must be float32, one per column")
-    _need(layout in ROTARY_LAYOUTS and norm in (None, "before", "after"), f"qkv_rotate_write: layout {layout!r}, norm {norm!r}")
+    _need(layout in ROTARY_LAYOUTS and norm in (None, "before", "after", "whole"), f"qkv_rotate_write: layout {layout!r}, norm {norm!r}")
     table_positions = _rotary_tables(cos, sin, rotary_dim, "qkv_rotate_write")
-    for weight in (q_weight, k_weight):
-        _need(weight is None or (weight.dtype == torch.float32 and weight.shape == (head_dim,) and weight.is_contiguous()), "qkv_rotate_write: norm weights must be float32 [d]")
+    for weight, heads in ((q_weight, nq), (k_weight, nkv)):
+        size = heads * head_dim if norm == "whole" else head_dim
+        _need(weight is None or (weight.dtype == torch.float32 and weight.shape == (size,) and weight.is_contiguous()), f"qkv_rotate_write: norm weights must be float32 [{size}]")
     for meta in (positions, token_row):
         _need(meta.dtype == torch.int32 and meta.is_contiguous() and meta.shape[0] >= tokens, "qkv_rotate_write: positions/token_row must be int32 [T]")
     _need(block_table.dtype == torch.int32 and block_table.dim() == 2 and block_table.is_contiguous(), "qkv_rotate_write: block_table must be contiguous int32 [rows, width]")
@@ -1853,9 +1957,10 @@ def qkv_rotate_write(
     library = _library("rotary.cu")
     _check(library, library.pylon_qkv_rotate_write(
         _ptr(qkv), qkv.stride(0), _ptr(bias), _ptr(cos), _ptr(sin), rotary_dim if cos is not None else 0, ROTARY_LAYOUTS[layout], table_positions,
-        {None: 0, "before": 1, "after": 2}[norm], _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(positions), _ptr(token_row), _ptr(block_table),
+        {None: 0, "before": 1, "after": 2, "whole": 3}[norm], _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(positions), _ptr(token_row), _ptr(block_table),
         block_table.shape[1], page_size, _ptr(k_pages), _ptr(v_pages), k_pages.shape[0], nq, nkv, head_dim, value_dim,
-        head_dim if norm_size is None else int(norm_size), tokens, _dtype_code(qkv.dtype), _ptr(cache_write_error_word(k_pages.device)), _stream()))
+        head_dim if norm_size is None else int(norm_size), tokens, _dtype_code(qkv.dtype), _ptr(cache_write_error_word(k_pages.device)),
+        int(values_from_keys), _ptr(q_factors), 0 if q_factors is None else q_factors.shape[0], _stream()))
     return qkv
 
 

@@ -26,11 +26,19 @@ the per-head norm of q and k behind the rotation instead of before it (``qk_norm
 together with values of their own width, chunks or a soft cap: one kernel for bias, rotation, norm and cache write
 (``ops.qkv_rotate_write``) then stands between the product and the attention.
 
-``weighting="sigmoid"``: a visible key's weight is ``sigmoid(score + b_h)``, not a softmax: nothing is divided by a sum over the keys
+Mixers with one of the following are **stacked**: what reads the input - the projections and the gates - is one product, then one kernel for
+biases, norms, rotation, the queries' factor and the cache write, the attention, which gates as it writes, and the output product.
+``values_from_keys``: the values are the projected keys as they are before norm and rotation (biases included), and there is no value
+projection.  ``distance_slopes``: a number per head that a score loses per position of distance.  ``fixed_sink``: the softmax's denominator holds
+``exp(fixed_sink)``, the score of a key without a value.  ``query_factor``: an encoding with ``query_factors``, a factor on the queries by
+position.  ``head_gate``: head h's output is multiplied by ``sigmoid((W_g x)_h)``, ``W_g [heads, width]``; ``output_gate``: every element
+of it is, ``W_g [heads * value_dim, width]``; both read the mixer's input.  ``out_bias``: a bias on the output product.  These go with biases, norms
+per head or over whole rows (``qk_norm``), rotations, windows, chunks and a soft cap.  In bfloat16 a softmax weight of such a mixer enters the
+sum over the values as two bfloat16 numbers, the rounded weight and what the rounding dropped.
+
+``weighting="sigmoid"`` (stacked as well): a visible key's weight is ``sigmoid(score + b_h)``, not a softmax: nothing is divided by a sum over the keys
 (``score_bias``: b, a learnt number per head; without it zero).  It goes with every option of the paragraph above and with windows, chunks
-and a soft cap.  ``head_gate``: head h's output is multiplied by ``sigmoid((W_g x)_h)``, ``W_g [heads, width]`` reading the mixer's input; its
-rows ride in the projections' product and the attention kernels multiply as they write.  In bfloat16 such a mixer keeps keys and
-values at one width, the larger of the two rounded up to a multiple of 16 (zero rows and columns of the weights fill it), so that
+and a soft cap.  In bfloat16 a stacked mixer keeps keys and values at one width, the larger of the two rounded up to a multiple of 16 (zero rows and columns of the weights fill it), so that
 every size up to 256 has the tensor-core kernels.
 """
 from __future__ import annotations
@@ -88,6 +96,12 @@ class GroupedQueryAttention(Mixer):
         weighting: str = "softmax",
         score_bias: bool = False,
         head_gate: bool = False,
+        output_gate: bool = False,
+        values_from_keys: bool = False,
+        distance_slopes: Optional[Sequence[float]] = None,
+        fixed_sink: Optional[float] = None,
+        query_factor: Optional[PartSpec] = None,
+        out_bias: bool = False,
     ) -> None:
         if n_heads % n_kv_heads:
             raise ValueError(f"{n_heads} query heads cannot be grouped over {n_kv_heads} KV heads")
@@ -109,7 +123,24 @@ class GroupedQueryAttention(Mixer):
             raise ValueError("kept first positions go with a window, and not with chunks")
         if self.bias_rows is not None and (self.bias_rows < 2 or not self.bias_far > self.bias_rows // 2):
             raise ValueError(f"a bias table of {self.bias_rows} rows that ends at distance {self.bias_far}")
-        plain_scores = self.plain_scores = self.keep_first > 0 or self.bias_rows is not None or self.has_sink or qk_norm == "whole"
+        self.has_output_gate, self.values_from_keys, self.has_out_bias = bool(output_gate), bool(values_from_keys), bool(out_bias)
+        self.distance_slopes = None if distance_slopes is None else tuple(float(value) for value in distance_slopes)
+        self.fixed_sink = None if fixed_sink is None else float(fixed_sink)
+        self.query_factor = None if query_factor is None else POSITION_ENCODINGS.build(query_factor)
+        self.stacked = weighting == "sigmoid" or bool(head_gate) or self.has_output_gate or self.values_from_keys or self.distance_slopes is not None \
+            or self.fixed_sink is not None or self.query_factor is not None or self.has_out_bias
+        if self.stacked and (self.keep_first or distance_bias is not None or sink or value_mix is not None):
+            raise NotImplementedError("stacked mixers: without kept first positions, a learnt bias by distance, learnt sinks and value mixing")
+        if head_gate and output_gate:
+            raise ValueError("heads are gated as a whole or element by element, not both")
+        if self.values_from_keys and self.value_dim != self.head_dim:
+            raise ValueError(f"values that are the keys are as wide as they are, {self.head_dim} and not {self.value_dim}")
+        if self.distance_slopes is not None and len(self.distance_slopes) != self.n_heads:
+            raise ValueError(f"a slope for each of {self.n_heads} heads, not {len(self.distance_slopes)}")
+        if weighting == "sigmoid" and (self.has_output_gate or self.values_from_keys or self.distance_slopes is not None or self.fixed_sink is not None
+                                       or self.query_factor is not None or self.has_out_bias):
+            raise NotImplementedError("sigmoid weights: of the stacked mixers' options with gated heads only")
+        plain_scores = self.plain_scores = not self.stacked and (self.keep_first > 0 or self.bias_rows is not None or self.has_sink or qk_norm == "whole")
         self.general = self.value_dim != self.head_dim or self.chunk is not None or self.softcap is not None or value_mix is not None or plain_scores
         self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
         if qk_norm not in ("before", "after", "whole"):
@@ -119,11 +150,11 @@ class GroupedQueryAttention(Mixer):
         if weighting not in ("softmax", "sigmoid"):
             raise ValueError(f"the weights of the keys are a 'softmax' or each a 'sigmoid', not {weighting!r}")
         self.weighting, self.has_score_bias, self.has_head_gate = weighting, bool(score_bias), bool(head_gate)
-        self.splits_products = weighting == "sigmoid"
-        if weighting == "sigmoid" and (plain_scores or value_mix is not None or bias):
-            raise NotImplementedError("sigmoid weights: without whole-row norms, kept first positions, a bias by distance, a sink, value mixing and projection biases")
-        if weighting != "sigmoid" and (score_bias or head_gate):
-            raise NotImplementedError("a number per head added to the scores and a gate per head go with sigmoid weights")
+        self.splits_products = self.stacked and not self.has_out_bias
+        if weighting == "sigmoid" and (qk_norm == "whole" or bias):
+            raise NotImplementedError("sigmoid weights: without whole-row norms and projection biases")
+        if weighting != "sigmoid" and score_bias:
+            raise NotImplementedError("a number per head added to the scores goes with sigmoid weights")
         self.bias, self.bias_suffix, self.qk_norm_place, self.qk_norm_weight = bool(bias), bias_suffix, qk_norm, bool(qk_norm_weight)
         self.window = None if window is None else int(window)
         self.scale = 1.0 / math.sqrt(self.head_dim) if scale is None else float(scale)
@@ -131,17 +162,17 @@ class GroupedQueryAttention(Mixer):
         self.names = {
             "q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "value_mix": "vmix", "distance_bias": "distance_bias", "sink": "sink",
-            "score_bias": "score_bias", "head_gate": "g_proj.weight",
+            "score_bias": "score_bias", "head_gate": "g_proj.weight", "output_gate": "g_proj.weight",
             **(names or {}),
         }
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.mix_weight = self.b_qkv = self.bias_table = self.sink = None
-        self.score_bias = None
+        self.score_bias = self.b_in = self.b_out = self.slopes = self.sinks = None
         self.kept_head_dim = self.head_dim     # the width keys have in the cache, and queries in the product: wider than head_dim when they are kept padded
         self.kept_value_dim = self.value_dim   # the width values have in the cache: wider than value_dim when they are kept padded
         # what the kernels that fuse norm, rotation and cache write do not take goes through the kernel that takes everything
         self.rotary_general = self.bias or self.qk_norm_place == "after" or (self.qk_norm_eps is not None and not self.qk_norm_weight) \
             or (self.position is not None and (self.general or getattr(self.position, "layout", "halves") != "halves"))
-        self.rotary_general = self.rotary_general or weighting == "sigmoid"
+        self.rotary_general = self.rotary_general or self.stacked
         if self.rotary_general and (value_mix is not None or (self.position is not None and not hasattr(self.position, "tables"))):
             raise NotImplementedError("biases, a norm behind the rotation or a rotation beside values of their own width: not with value mixing, and "
                                       "only with an encoding that rotates by tables of cos and sin")
@@ -152,9 +183,10 @@ class GroupedQueryAttention(Mixer):
         decls = [
             TensorDecl(n["q"], (self.q_size, self.width)),
             TensorDecl(n["k"], (self.kv_size, self.width)),
-            TensorDecl(n["v"], (self.v_size, self.width)),
             TensorDecl(n["o"], (self.width, self.out_size)),
         ]
+        if not self.values_from_keys:
+            decls.append(TensorDecl(n["v"], (self.v_size, self.width)))
         if self.value_mix is not None:   # the source layer's weight is in the checkpoint too, and is not used
             decls.append(TensorDecl(n["value_mix"], (), "vector", (0.5, 0.1)))
         if self.qk_norm_eps is not None and self.qk_norm_weight:
@@ -168,15 +200,19 @@ class GroupedQueryAttention(Mixer):
             decls.append(TensorDecl(n["score_bias"], (self.n_heads,), "vector", (-7.0, 0.5)))   # about minus the logarithm of a context's length
         if self.has_head_gate:
             decls.append(TensorDecl(n["head_gate"], (self.n_heads, self.width)))
+        if self.has_output_gate:
+            decls.append(TensorDecl(n["output_gate"], (self.out_size, self.width)))
         if self.bias:
             decls += [TensorDecl(n[key] + self.bias_suffix, (size,), "vector", (0.0, 0.02))
-                      for key, size in (("q", self.q_size), ("k", self.kv_size), ("v", self.v_size))]
+                      for key, size in (("q", self.q_size), ("k", self.kv_size), ("v", self.v_size)) if not (key == "v" and self.values_from_keys)]
+        if self.has_out_bias:
+            decls.append(TensorDecl(n["o"] + self.bias_suffix, (self.width,), "vector", (0.0, 0.02)))
         return decls
 
     def load(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> None:
         n = self.names
-        if self.weighting == "sigmoid":
-            self._load_sigmoid(tensors, dtype)
+        if self.stacked:
+            self._load_stacked(tensors, dtype, device)
             return
         w_v, w_o = tensors[n["v"]], tensors[n["o"]]
         b_v = tensors[n["v"] + self.bias_suffix] if self.bias else None
@@ -211,8 +247,9 @@ class GroupedQueryAttention(Mixer):
         if self.has_sink:
             self.sink = tensors[n["sink"]].contiguous()
 
-    def _load_sigmoid(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype) -> None:
+    def _load_stacked(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> None:
         n = self.names
+        self.kept_head_dim, self.kept_value_dim = self.head_dim, self.value_dim
         if dtype == torch.bfloat16 and max(self.head_dim, self.value_dim) <= 256:
             self.kept_head_dim = self.kept_value_dim = -(-max(self.head_dim, self.value_dim) // 16) * 16
 
@@ -220,25 +257,36 @@ class GroupedQueryAttention(Mixer):
             if kept == width:
                 return weight
             padded = weight.new_zeros((heads, kept, weight.shape[1]))
-            padded[:, :width] = weight.view(heads, width, -1)
+            padded[:, :width] = weight.reshape(heads, width, -1)
             return padded.view(heads * kept, -1)
 
-        rows = [wider(tensors[n["q"]], self.n_heads, self.head_dim, self.kept_head_dim), wider(tensors[n["k"]], self.n_kv_heads, self.head_dim, self.kept_head_dim),
-                wider(tensors[n["v"]], self.n_kv_heads, self.value_dim, self.kept_value_dim)]
+        parts = [("q", self.n_heads, self.head_dim, self.kept_head_dim), ("k", self.n_kv_heads, self.head_dim, self.kept_head_dim),
+                 ("v", self.n_kv_heads, self.value_dim, self.kept_value_dim)][: 2 if self.values_from_keys else 3]
+        rows = [wider(tensors[n[key]], heads, size, kept) for key, heads, size, kept in parts]
         if self.has_head_gate:
             rows.append(tensors[n["head_gate"]])
+        if self.has_output_gate:   # as wide as the heads are kept: an element that is filled up is zero, whatever its gate
+            rows.append(wider(tensors[n["output_gate"]], self.n_heads, self.value_dim, self.kept_value_dim))
         filled = sum(part.shape[0] for part in rows)
         if filled % 8:   # the gate's rows fill up whole 16-byte pieces of the product's rows
             rows.append(rows[0].new_zeros((-filled % 8, self.width)))
         self.input_rows = torch.cat(rows, dim=0).contiguous()
         self.output_columns = wider(tensors[n["o"]].t(), self.n_heads, self.value_dim, self.kept_value_dim).t().contiguous()
         if self.qk_norm_eps is not None and self.qk_norm_weight:
-            fill = self.kept_head_dim - self.head_dim
-            self.q_norm, self.k_norm = (torch.nn.functional.pad(tensors[n[key]], (0, fill)).contiguous() for key in ("q_norm", "k_norm"))
+            sizes = {"q_norm": self.n_heads, "k_norm": self.n_kv_heads} if self.qk_norm_place == "whole" else {"q_norm": 1, "k_norm": 1}
+            self.q_norm, self.k_norm = (wider(tensors[n[key]].unsqueeze(1), heads, self.head_dim, self.kept_head_dim).reshape(-1).contiguous() for key, heads in sizes.items())
+        if self.bias:
+            self.b_in = torch.cat([wider(tensors[n[key] + self.bias_suffix].unsqueeze(1), heads, size, kept).reshape(-1) for key, heads, size, kept in parts]).contiguous()
+        if self.has_out_bias:
+            self.b_out = tensors[n["o"] + self.bias_suffix].contiguous()
+        if self.distance_slopes is not None:
+            self.slopes = torch.tensor(self.distance_slopes, dtype=torch.float32, device=device)
+        if self.fixed_sink is not None:
+            self.sinks = torch.full((self.n_heads,), self.fixed_sink, dtype=torch.float32, device=device)
         self.score_bias = tensors[n["score_bias"]].contiguous() if self.has_score_bias else None
 
     def weight_bytes(self) -> int:
-        if self.weighting == "sigmoid":
+        if self.stacked:
             return (self.input_rows.numel() + self.output_columns.numel()) * self.input_rows.element_size() + (0 if self.q_norm is None else 8 * self.head_dim)
         return (self.w_qkv.numel() + self.w_o.numel()) * self.w_qkv.element_size() + (0 if self.q_norm is None else 8 * self.head_dim)
 
@@ -249,10 +297,11 @@ class GroupedQueryAttention(Mixer):
 
     # -- run -----------------------------------------------------------------------------
     def forward(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> torch.Tensor:
-        if self.weighting == "sigmoid":
-            context = torch.empty((h.shape[0], self.output_columns.shape[1]), dtype=h.dtype, device=h.device)
-            self.middle(ops.linear_stacked(h, self.input_rows), step, cache, context, 1.0)
-            return ops.linear_for_residual(context, self.output_columns)
+        if self.stacked:
+            output, bias = self.forward_unjoined(h, step, cache)
+            if bias is None:
+                return output
+            return ops.add_bias((output.sum(dim=0) if output.dim() == 3 else output.float()).contiguous(), bias).unsqueeze(0)   # float32: one partial sum
         if self.rotary_general:
             return self._forward_rotary_general(h, step, cache)
         if self.general:
@@ -331,20 +380,30 @@ class GroupedQueryAttention(Mixer):
         )
         return ops.linear_for_residual(context, self.w_o)
 
+    def forward_unjoined(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> tuple[torch.Tensor, Optional[torch.Tensor]]:
+        if not self.stacked:
+            return self.forward(h, step, cache), None
+        context = torch.empty((h.shape[0], self.output_columns.shape[1]), dtype=h.dtype, device=h.device)
+        self.middle(ops.linear_stacked(h, self.input_rows), step, cache, context, 1.0)
+        return ops.linear_for_residual(context, self.output_columns), self.b_out
+
     def middle(self, proj: torch.Tensor, step: StepView, cache: LayerCache, out: torch.Tensor, factor: float) -> None:
-        """Sigmoid weights: one kernel for norms, rotation and cache write on the projections, then the attention, which gates its heads
-        and multiplies them by ``factor`` as it writes them."""
+        """Stacked mixers: one kernel for biases, norms, rotation, factor and cache write on the projections, then the attention, which gates
+        its heads and multiplies them by ``factor`` as it writes them."""
         cos, sin, rotary_dim, layout = self.position.tables(proj.device) if self.position is not None else (None, None, 0, "halves")
-        columns = (self.n_heads + self.n_kv_heads) * self.kept_head_dim + self.n_kv_heads * self.kept_value_dim
+        columns = (self.n_heads + self.n_kv_heads) * self.kept_head_dim + (0 if self.values_from_keys else self.n_kv_heads * self.kept_value_dim)
+        gates = self.n_heads * self.kept_value_dim if self.has_output_gate else self.n_heads
         qkv = proj[:, :columns]
         ops.qkv_rotate_write(
-            qkv, None, cos, sin, rotary_dim, layout, None if self.qk_norm_eps is None else self.qk_norm_place, self.q_norm, self.k_norm,
+            qkv, self.b_in, cos, sin, rotary_dim, layout, None if self.qk_norm_eps is None else self.qk_norm_place, self.q_norm, self.k_norm,
             self.qk_norm_eps or 0.0, step.positions, step.token_row, cache.block_table, cache.page_size, cache.k_pages, cache.v_pages,
-            self.n_heads, self.n_kv_heads, self.kept_head_dim, self.kept_value_dim, norm_size=self.head_dim,
+            self.n_heads, self.n_kv_heads, self.kept_head_dim, self.kept_value_dim, norm_size=self.head_dim, values_from_keys=self.values_from_keys,
+            q_factors=None if self.query_factor is None else self.query_factor.query_factors(proj.device),
         )
         ops.paged_attention(
             qkv, cache.k_pages, cache.v_pages, step.positions, step.token_row, step.q_start, step.kv_len, cache.block_table,
             self.n_heads, step.max_q, step.max_kv, window=self.window, scale=self.scale, out=out, row_tokens=step.row_tokens,
-            rows_alike=step.rows_alike, chunk=self.chunk, softcap=self.softcap, weighting="sigmoid", score_bias=self.score_bias,
-            head_gate=proj[:, columns: columns + self.n_heads] if self.has_head_gate else None, out_factor=factor,
+            rows_alike=step.rows_alike, chunk=self.chunk, softcap=self.softcap, weighting=self.weighting, score_bias=self.score_bias,
+            head_gate=proj[:, columns: columns + gates] if self.has_head_gate or self.has_output_gate else None, out_factor=factor,
+            sinks=self.sinks, distance_slopes=self.slopes, split_weights=True,
         )

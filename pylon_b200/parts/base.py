@@ -197,6 +197,8 @@ class Part:
 
 
 class Norm(Part):
+    joins = False   # True: ``apply`` takes outputs that were left side by side (:meth:`ResidualStream.add_together`) in its own kernel
+
     def apply(self, stream: "ResidualStream", rows: Optional[torch.Tensor] = None, read: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Fold what is pending into the stream and return the normalised activations of all tokens, or of ``rows``
         only.  ``read``: for a stream of several copies, the float32 weights ``[copies]`` of the combination that is
@@ -249,6 +251,11 @@ class Mixer(Part):
     def forward(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> torch.Tensor:
         """Returns the delta for the residual stream (see :class:`ResidualStream`)."""
         raise NotImplementedError
+
+    def forward_unjoined(self, h: torch.Tensor, step: StepView, cache: LayerCache) -> tuple[torch.Tensor, Optional[torch.Tensor]]:
+        """The same for a reader that adds up several things in one pass: (a delta, a float32 vector ``[width]`` to be added to every one
+        of its rows, or ``None``)."""
+        return self.forward(h, step, cache), None
 
 
 class FeedForward(Part):
@@ -303,18 +310,33 @@ class ResidualStream:
         self.pending: Optional[torch.Tensor] = None
         self.pending_scale = 1.0
         self.pending_route: Optional[StreamRoute] = None
+        self.joined = None                               # ops.SideBySide: outputs that one kernel adds together, with the next norm
         self.activation: Optional[torch.Tensor] = None   # the sum in the compute dtype, where the last kernel that wrote the sum left it
 
     @property
     def plain(self) -> bool:
         """One copy, and what is pending is added as it is: the case the fused add + RMSNorm kernels are written for."""
-        return self.residual.dim() == 2 and self.pending_scale == 1.0 and self.pending_route is None
+        return self.residual.dim() == 2 and self.joined is None and self.pending_scale == 1.0 and self.pending_route is None
 
     def add(self, delta: torch.Tensor, scale: float = 1.0, route: Optional[StreamRoute] = None) -> None:
-        if self.pending is not None:
+        if self.pending is not None or self.joined is not None:
             self.flush()
         self.pending, self.pending_scale, self.pending_route = delta, float(scale), route
         self.activation = None
+
+    def add_together(self, joined) -> None:
+        """Leaves the outputs of sublayers that stood side by side (:class:`ops.SideBySide`) for the next norm, whose kernel adds them all
+        to the sum as it reads it; for a residual stream of one copy."""
+        self.flush()
+        self.joined, self.activation = joined, None
+
+    def settle(self) -> None:
+        """Adds now what was left by :meth:`add_together`: for readers without a kernel that takes it."""
+        if self.joined is not None:
+            from pylon_b200.kernels import ops
+
+            joined, self.joined = self.joined, None
+            ops.join_norm(self.residual, joined)
 
     def read(self, dtype: torch.dtype) -> torch.Tensor:
         """The sum as it is (nothing pending, no norm) in ``dtype``: what a sublayer reads whose norm stands on its output."""
@@ -329,6 +351,7 @@ class ResidualStream:
         return pending
 
     def flush(self) -> None:
+        self.settle()
         if self.pending is None:
             return
         from pylon_b200.kernels import ops

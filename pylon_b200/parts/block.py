@@ -10,6 +10,7 @@ from typing import Mapping, Optional, Sequence
 
 import torch
 
+from pylon_b200.kernels import ops
 from pylon_b200.parts.base import (
     BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, LayerCache, ResidualStream, StepView, StreamRoute, TensorDecl,
 )
@@ -145,6 +146,8 @@ class HyperPreNormBlock(Block):
 class ParallelSublayers(Block):
     """One norm, two readers: with ``h = norm(x)`` the layer is ``x = x + (mixer(h) + feed_forward(h))``.  Both outputs join the
     32-bit residual sum (the mixer's first, the feed-forward's at the next norm); ``feed_forward=None`` leaves the second out.
+    Where the norms have a kernel for it (``Norm.joins``) the two outputs stay where they lie - the mixer's product, perhaps as partial
+    sums and without its bias, the experts' rows in their slots - and the next norm's kernel adds everything to the sum.
     The tensors: the mixer's under ``mixer_prefix``, the feed-forward's under ``ffn_prefix``, the norm's under ``norm_prefix``."""
 
     def __init__(self, mixer: PartSpec, feed_forward: Optional[PartSpec], norm: PartSpec, mixer_prefix: str = "mix.", ffn_prefix: str = "mlp.",
@@ -174,6 +177,11 @@ class ParallelSublayers(Block):
 
     def forward(self, stream: ResidualStream, step: StepView, cache: LayerCache) -> None:
         h = self.norm.apply(stream)
+        if self.norm.joins and stream.residual.dim() == 2:
+            output, bias = self.mixer.forward_unjoined(h, step, cache)
+            rows = None if self.feed_forward is None else self.feed_forward.forward_scattered(h, step)
+            stream.add_together(ops.SideBySide(output, bias, rows))
+            return
         stream.add(self.mixer.forward(h, step, cache))
         if self.feed_forward is not None:
             stream.add(self.feed_forward.forward(h, step))

@@ -17,22 +17,25 @@ from pylon_b200.parts.base import NORMS, Norm, ResidualStream, TensorDecl
 @NORMS.register("rmsnorm")
 class RMSNorm(Norm):
     """``offset``: the checkpoint stores the weight less this number (a checkpoint that holds the weight's difference from one has ``offset=1``:
-    ``y = x / rms(x) * (1 + w)``); the sum is formed once at load, in float32."""
+    ``y = x / rms(x) * (1 + w)``); the sum is formed once at load, in float32.  ``one_number``: the weight is a single number for all
+    coordinates (a tensor without dimensions)."""
 
-    def __init__(self, width: int, eps: float, weight_name: str = "weight", offset: float = 0.0) -> None:
+    joins = True   # the kernel that adds outputs side by side to the stream norms it in the same pass
+
+    def __init__(self, width: int, eps: float, weight_name: str = "weight", offset: float = 0.0, one_number: bool = False) -> None:
         self.width = int(width)
         self.eps = float(eps)
         self.weight_name = weight_name
-        self.offset = float(offset)
+        self.offset, self.one_number = float(offset), bool(one_number)
         self.weight: Optional[torch.Tensor] = None
         self.dtype: Optional[torch.dtype] = None
 
     def tensors(self) -> Sequence[TensorDecl]:
         init = None if self.offset == 0.0 else (1.0 - self.offset, 0.02)
-        return (TensorDecl(self.weight_name, (self.width,), "vector", init),)
+        return (TensorDecl(self.weight_name, () if self.one_number else (self.width,), "vector", init),)
 
     def load(self, tensors: Mapping[str, torch.Tensor], dtype: torch.dtype, device: torch.device) -> None:
-        weight = tensors[self.weight_name]
+        weight = tensors[self.weight_name].expand(self.width)   # one number is spread over the row: the kernels take a weight per coordinate
         self.weight = (weight if self.offset == 0.0 else weight + self.offset).contiguous()
         self.dtype = dtype
 
@@ -40,6 +43,11 @@ class RMSNorm(Norm):
         return self.width * 4
 
     def apply(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None, read: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if stream.joined is not None:
+            joined = stream.joined
+            if rows is None:   # with a row selection the stream stays as it is, and what is pending stays pending
+                stream.joined = None
+            return ops.join_norm(stream.residual, joined, self.weight, self.eps, self.dtype, rows=rows)
         if not stream.plain:
             return _apply_to_streams(self, "rmsnorm", stream, rows, read)
         delta, stream.pending = stream.pending, None
@@ -60,6 +68,7 @@ class RMSNorm(Norm):
 def _apply_to_streams(norm, kind: str, stream: ResidualStream, rows: Optional[torch.Tensor], read: Optional[torch.Tensor]) -> torch.Tensor:
     """The general form: one or several copies of the stream, a factor on the pending delta, a route by which it enters
     the copies, the combination of copies that is read, layer norm or RMS norm - one kernel."""
+    stream.settle()
     if rows is None:
         delta, scale, route = stream.take_pending()
     else:   # the stream stays as it is: what is pending stays pending
@@ -122,6 +131,7 @@ class DynamicTanh(Norm):
         return self.width * 8 + 4
 
     def apply(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None, read: Optional[torch.Tensor] = None) -> torch.Tensor:
+        stream.settle()
         if rows is None:
             delta, scale, route = stream.take_pending()
         else:   # the stream stays as it is: what is pending stays pending

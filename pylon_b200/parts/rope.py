@@ -18,7 +18,10 @@ changes the frequencies f_j = theta^(-2j / rotary_dim) for contexts longer than 
   ``hi = min(ceil(index(slow)), rotary_dim - 1)`` and ``ramp_j = clamp((j - lo) / max(hi - lo, 0.001), 0, 1)`` the frequency is
   ``f_j / factor * ramp_j + f_j (1 - ramp_j)``, and cos and sin are both multiplied by ``0.1 ln(factor) + 1``.
 
-Frequencies and angles of scaled tables are formed in float64 and rounded once to float32.
+Frequencies and angles of scaled tables, and of all tables with ``exact_angles``, are formed in float64, and cos and sin rounded once to float32.
+
+``log_steps`` is not a rotation: a query at position p is multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``, from a float32
+table by position formed in float64 (``query_factors``).
 """
 from __future__ import annotations
 
@@ -33,7 +36,7 @@ from pylon_b200.parts.base import POSITION_ENCODINGS, PositionEncoding
 @POSITION_ENCODINGS.register("rope")
 class RotaryEncoding(PositionEncoding):
     def __init__(self, head_dim: int, theta: float, max_positions: int, rotary_dim: Optional[int] = None,
-                 scaling: Optional[Mapping[str, float]] = None, layout: str = "halves") -> None:
+                 scaling: Optional[Mapping[str, float]] = None, layout: str = "halves", exact_angles: bool = False) -> None:
         self.head_dim = int(head_dim)
         self.rotary_dim = int(rotary_dim if rotary_dim is not None else head_dim)
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= self.head_dim:
@@ -45,7 +48,7 @@ class RotaryEncoding(PositionEncoding):
         self.theta = float(theta)
         self.max_positions = int(max_positions)
         self.scaling = None if scaling is None else dict(scaling)
-        self.layout = layout
+        self.layout, self.exact_angles = layout, bool(exact_angles)
         self._tables: Optional[tuple[torch.Tensor, torch.Tensor]] = None
 
     def set_max_positions(self, positions: int) -> None:
@@ -80,7 +83,7 @@ class RotaryEncoding(PositionEncoding):
     def tables(self, device: torch.device) -> tuple[torch.Tensor, torch.Tensor, int, str]:
         """(cos, sin, rotary_dim, layout): float32 ``[positions, rotary_dim // 2]`` tables, any scaling and factor included."""
         if self._tables is None or self._tables[0].device != device:
-            if self.scaling is None:
+            if self.scaling is None and not self.exact_angles:
                 exponent = torch.arange(0, self.rotary_dim, 2, dtype=torch.float32) / self.rotary_dim
                 inv_freq = 1.0 / (self.theta ** exponent)
                 angles = torch.arange(self.max_positions, dtype=torch.float32).unsqueeze(1) * inv_freq.unsqueeze(0)
@@ -97,3 +100,21 @@ class RotaryEncoding(PositionEncoding):
             return None   # the kernels that fuse the rotation pair element j with j + rotary_dim / 2
         cos, sin, rotary_dim, _ = self.tables(device)
         return cos, sin, rotary_dim
+
+
+@POSITION_ENCODINGS.register("log_steps")
+class LogSteps(PositionEncoding):
+    """A factor on the queries that grows with the logarithm of their position, in steps of ``every`` positions."""
+
+    def __init__(self, coef: float, every: float, max_positions: int) -> None:
+        self.coef, self.every, self.max_positions = float(coef), float(every), int(max_positions)
+        if not self.every > 0:
+            raise ValueError(f"the factor steps up every so many positions, not every {every!r}")
+        self._factors: Optional[torch.Tensor] = None
+
+    def query_factors(self, device: torch.device) -> torch.Tensor:
+        """float32 ``[positions]``."""
+        if self._factors is None or self._factors.device != device:
+            steps = torch.floor((torch.arange(self.max_positions, dtype=torch.float64) + 1.0) / self.every)
+            self._factors = (1.0 + self.coef * torch.log(steps + 1.0)).to(torch.float32).to(device).contiguous()
+        return self._factors
