@@ -25,17 +25,17 @@ SINK_SCORE = 0.0           # attention_2: the softmax's denominator holds exp(SI
 def _mixer(config: PinedraConfig, m: PinedraAttention, positions: int) -> PartSpec:
     params = {
         "width": config.width, "n_heads": m.heads, "n_kv_heads": m.kv_heads, "head_dim": m.dim, "value_dim": m.vdim, "scale": m.scale,
-        "names": {"q": "q", "k": "k", "v": "v", "o": "o", "q_norm": "q.norm", "k_norm": "k.norm", "head_gate": "g", "output_gate": "g"},
+        "names": {"q": "q", "k": "k", "v": "v", "o": "o", "q_norm": "q.norm", "k_norm": "k.norm", "output_gate": "g"},
     }
     if m.kind == "attention":
-        params.update(values_from_keys=True, qk_norm="whole", qk_norm_eps=config.norm_eps, bias=True, out_bias=True, output_gate=True)
+        params.update(values_from_keys=True, qk_norm="whole", qk_norm_eps=config.norm_eps, bias=True, out_bias=True, output_gate="elements")
     elif m.kind == "attention_2":
         params.update(qk_norm_eps=config.norm_eps, distance_slopes=tuple(2.0 ** (-SLOPE_SPAN * (h + 1) / m.heads) for h in range(m.heads)),
-                      fixed_sink=SINK_SCORE, output_gate=True)
+                      fixed_sink=SINK_SCORE, output_gate="elements")
         if m.temperature is not None:
             params["query_factor"] = PartSpec("log_steps", {"coef": m.temperature[0], "every": m.temperature[1], "max_positions": positions})
     else:
-        params.update(bias=True, head_gate=True, softcap=m.softcap, chunk=m.chunk)
+        params.update(bias=True, output_gate="heads", softcap=m.softcap, chunk=m.chunk)
         if m.rot is not None:
             params["position"] = PartSpec("rope", {"head_dim": m.dim, "theta": m.rot.base, "max_positions": positions, "rotary_dim": m.rot.dims,
                                                    "exact_angles": True})

@@ -31,7 +31,7 @@ biases, norms, rotation, the queries' factor and the cache write, the attention,
 ``values_from_keys``: the values are the projected keys as they are before norm and rotation (biases included), and there is no value
 projection.  ``distance_slopes``: a number per head that a score loses per position of distance.  ``fixed_sink``: the softmax's denominator holds
 ``exp(fixed_sink)``, the score of a key without a value.  ``query_factor``: an encoding with ``query_factors``, a factor on the queries by
-position.  ``head_gate``: head h's output is multiplied by ``sigmoid((W_g x)_h)``, ``W_g [heads, width]``; ``output_gate``: every element
+position.  ``output_gate="heads"``: head h's output is multiplied by ``sigmoid((W_g x)_h)``, ``W_g [heads, width]``; ``"elements"``: every element
 of it is, ``W_g [heads * value_dim, width]``; both read the mixer's input.  ``out_bias``: a bias on the output product.  These go with biases, norms
 per head or over whole rows (``qk_norm``), rotations, windows, chunks and a soft cap.  In bfloat16 a softmax weight of such a mixer enters the
 sum over the values as two bfloat16 numbers, the rounded weight and what the rounding dropped.
@@ -96,7 +96,7 @@ class GroupedQueryAttention(Mixer):
         weighting: str = "softmax",
         score_bias: bool = False,
         head_gate: bool = False,
-        output_gate: bool = False,
+        output_gate: Optional[str] = None,
         values_from_keys: bool = False,
         distance_slopes: Optional[Sequence[float]] = None,
         fixed_sink: Optional[float] = None,
@@ -123,23 +123,25 @@ class GroupedQueryAttention(Mixer):
             raise ValueError("kept first positions go with a window, and not with chunks")
         if self.bias_rows is not None and (self.bias_rows < 2 or not self.bias_far > self.bias_rows // 2):
             raise ValueError(f"a bias table of {self.bias_rows} rows that ends at distance {self.bias_far}")
-        self.has_output_gate, self.values_from_keys, self.has_out_bias = bool(output_gate), bool(values_from_keys), bool(out_bias)
+        if output_gate not in (None, "heads", "elements"):
+            raise ValueError(f"an output is gated by its 'heads' or its 'elements', not {output_gate!r}")
+        self.output_gate, self.values_from_keys, self.has_out_bias = output_gate, bool(values_from_keys), bool(out_bias)
         self.distance_slopes = None if distance_slopes is None else tuple(float(value) for value in distance_slopes)
         self.fixed_sink = None if fixed_sink is None else float(fixed_sink)
         self.query_factor = None if query_factor is None else POSITION_ENCODINGS.build(query_factor)
-        self.stacked = weighting == "sigmoid" or bool(head_gate) or self.has_output_gate or self.values_from_keys or self.distance_slopes is not None \
+        self.stacked = weighting == "sigmoid" or output_gate is not None or self.values_from_keys or self.distance_slopes is not None \
             or self.fixed_sink is not None or self.query_factor is not None or self.has_out_bias
         if self.stacked and (self.keep_first or distance_bias is not None or sink or value_mix is not None):
             raise NotImplementedError("stacked mixers: without kept first positions, a learnt bias by distance, learnt sinks and value mixing")
-        if head_gate and output_gate:
-            raise ValueError("heads are gated as a whole or element by element, not both")
         if self.values_from_keys and self.value_dim != self.head_dim:
             raise ValueError(f"values that are the keys are as wide as they are, {self.head_dim} and not {self.value_dim}")
         if self.distance_slopes is not None and len(self.distance_slopes) != self.n_heads:
             raise ValueError(f"a slope for each of {self.n_heads} heads, not {len(self.distance_slopes)}")
-        if weighting == "sigmoid" and (self.has_output_gate or self.values_from_keys or self.distance_slopes is not None or self.fixed_sink is not None
+        if head_gate and output_gate is not None:
+            raise ValueError("heads are gated once: head_gate is output_gate='heads' under its older name")
+        if weighting == "sigmoid" and (self.values_from_keys or self.distance_slopes is not None or self.fixed_sink is not None
                                        or self.query_factor is not None or self.has_out_bias):
-            raise NotImplementedError("sigmoid weights: of the stacked mixers' options with gated heads only")
+            raise NotImplementedError("sigmoid weights: of the stacked mixers' options with gated outputs only")
         plain_scores = self.plain_scores = not self.stacked and (self.keep_first > 0 or self.bias_rows is not None or self.has_sink or qk_norm == "whole")
         self.general = self.value_dim != self.head_dim or self.chunk is not None or self.softcap is not None or value_mix is not None or plain_scores
         self.qk_norm_eps = None if qk_norm_eps is None else float(qk_norm_eps)
@@ -149,12 +151,14 @@ class GroupedQueryAttention(Mixer):
             raise NotImplementedError("whole-row norms, kept first positions, a bias by distance and a sink: without rotation, value mixing and projection biases")
         if weighting not in ("softmax", "sigmoid"):
             raise ValueError(f"the weights of the keys are a 'softmax' or each a 'sigmoid', not {weighting!r}")
-        self.weighting, self.has_score_bias, self.has_head_gate = weighting, bool(score_bias), bool(head_gate)
+        self.weighting, self.has_score_bias = weighting, bool(score_bias)
         self.splits_products = self.stacked and not self.has_out_bias
         if weighting == "sigmoid" and (qk_norm == "whole" or bias):
             raise NotImplementedError("sigmoid weights: without whole-row norms and projection biases")
-        if weighting != "sigmoid" and score_bias:
-            raise NotImplementedError("a number per head added to the scores goes with sigmoid weights")
+        if weighting != "sigmoid" and (score_bias or head_gate):
+            raise NotImplementedError("a number per head added to the scores, and this name for a gate per head, go with sigmoid weights (output_gate with either)")
+        if head_gate:
+            self.output_gate = "heads"
         self.bias, self.bias_suffix, self.qk_norm_place, self.qk_norm_weight = bool(bias), bias_suffix, qk_norm, bool(qk_norm_weight)
         self.window = None if window is None else int(window)
         self.scale = 1.0 / math.sqrt(self.head_dim) if scale is None else float(scale)
@@ -162,9 +166,10 @@ class GroupedQueryAttention(Mixer):
         self.names = {
             "q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "value_mix": "vmix", "distance_bias": "distance_bias", "sink": "sink",
-            "score_bias": "score_bias", "head_gate": "g_proj.weight", "output_gate": "g_proj.weight",
+            "score_bias": "score_bias", "head_gate": "g_proj.weight",
             **(names or {}),
         }
+        self.names.setdefault("output_gate", self.names["head_gate"])
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.mix_weight = self.b_qkv = self.bias_table = self.sink = None
         self.score_bias = self.b_in = self.b_out = self.slopes = self.sinks = None
         self.kept_head_dim = self.head_dim     # the width keys have in the cache, and queries in the product: wider than head_dim when they are kept padded
@@ -198,10 +203,8 @@ class GroupedQueryAttention(Mixer):
             decls.append(TensorDecl(n["sink"], (self.n_heads,), "vector", (0.0, 1.0)))
         if self.has_score_bias:
             decls.append(TensorDecl(n["score_bias"], (self.n_heads,), "vector", (-7.0, 0.5)))   # about minus the logarithm of a context's length
-        if self.has_head_gate:
-            decls.append(TensorDecl(n["head_gate"], (self.n_heads, self.width)))
-        if self.has_output_gate:
-            decls.append(TensorDecl(n["output_gate"], (self.out_size, self.width)))
+        if self.output_gate is not None:
+            decls.append(TensorDecl(n["output_gate"], (self.n_heads if self.output_gate == "heads" else self.out_size, self.width)))
         if self.bias:
             decls += [TensorDecl(n[key] + self.bias_suffix, (size,), "vector", (0.0, 0.02))
                       for key, size in (("q", self.q_size), ("k", self.kv_size), ("v", self.v_size)) if not (key == "v" and self.values_from_keys)]
@@ -263,9 +266,9 @@ class GroupedQueryAttention(Mixer):
         parts = [("q", self.n_heads, self.head_dim, self.kept_head_dim), ("k", self.n_kv_heads, self.head_dim, self.kept_head_dim),
                  ("v", self.n_kv_heads, self.value_dim, self.kept_value_dim)][: 2 if self.values_from_keys else 3]
         rows = [wider(tensors[n[key]], heads, size, kept) for key, heads, size, kept in parts]
-        if self.has_head_gate:
-            rows.append(tensors[n["head_gate"]])
-        if self.has_output_gate:   # as wide as the heads are kept: an element that is filled up is zero, whatever its gate
+        if self.output_gate == "heads":
+            rows.append(tensors[n["output_gate"]])
+        if self.output_gate == "elements":   # as wide as the heads are kept: an element that is filled up is zero, whatever its gate
             rows.append(wider(tensors[n["output_gate"]], self.n_heads, self.value_dim, self.kept_value_dim))
         filled = sum(part.shape[0] for part in rows)
         if filled % 8:   # the gate's rows fill up whole 16-byte pieces of the product's rows
@@ -392,7 +395,7 @@ class GroupedQueryAttention(Mixer):
         its heads and multiplies them by ``factor`` as it writes them."""
         cos, sin, rotary_dim, layout = self.position.tables(proj.device) if self.position is not None else (None, None, 0, "halves")
         columns = (self.n_heads + self.n_kv_heads) * self.kept_head_dim + (0 if self.values_from_keys else self.n_kv_heads * self.kept_value_dim)
-        gates = self.n_heads * self.kept_value_dim if self.has_output_gate else self.n_heads
+        gates = self.n_heads * self.kept_value_dim if self.output_gate == "elements" else self.n_heads
         qkv = proj[:, :columns]
         ops.qkv_rotate_write(
             qkv, self.b_in, cos, sin, rotary_dim, layout, None if self.qk_norm_eps is None else self.qk_norm_place, self.q_norm, self.k_norm,
@@ -404,6 +407,6 @@ class GroupedQueryAttention(Mixer):
             qkv, cache.k_pages, cache.v_pages, step.positions, step.token_row, step.q_start, step.kv_len, cache.block_table,
             self.n_heads, step.max_q, step.max_kv, window=self.window, scale=self.scale, out=out, row_tokens=step.row_tokens,
             rows_alike=step.rows_alike, chunk=self.chunk, softcap=self.softcap, weighting=self.weighting, score_bias=self.score_bias,
-            head_gate=proj[:, columns: columns + gates] if self.has_head_gate or self.has_output_gate else None, out_factor=factor,
+            head_gate=proj[:, columns: columns + gates] if self.output_gate is not None else None, out_factor=factor,
             sinks=self.sinks, distance_slopes=self.slopes, split_weights=True,
         )
