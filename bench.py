@@ -18,8 +18,8 @@ decode steps) at B = 1, 8, 64 with its share of the HBM roofline; the output rat
 serving workloads at the 8B and 14B shapes; and a full-depth float32 run at the 14B shape with
 its largest logit error against the plain implementation.
 
-``--workload designs`` is another measurement with a line of its own: Vopepel, Fikerax, Zemavik, Rirusun and Zabusun beside Qwen3 dense at equal width, depth,
-heads, feed-forward and vocabulary (sizes ``2k`` and ``4k``; ``--designs`` picks among the six): prefill of a 2,048-token prompt, decode at batch 8 and a context of 2,048,
+``--workload designs`` is another measurement with a line of its own: Vopepel, Fikerax, Zemavik, Rirusun, Zabusun and Pinedra beside Qwen3 dense at equal width, depth,
+heads, feed-forward and vocabulary (sizes ``2k`` and ``4k``; ``--designs`` picks among the seven): prefill of a 2,048-token prompt, decode at batch 8 and a context of 2,048,
 and the time of every kernel entry point in one step of each kind.
 """
 from __future__ import annotations
@@ -475,7 +475,7 @@ def run_serving_workload(name: str, torch) -> dict:
 
 
 # ---------------------------------------------------------------------------------------
-# Vopepel, Fikerax, Zemavik, Rirusun and Zabusun beside Qwen3 at equal size (--workload designs)
+# Vopepel, Fikerax, Zemavik, Rirusun, Zabusun and Pinedra beside Qwen3 at equal size (--workload designs)
 # ---------------------------------------------------------------------------------------
 DESIGN_SIZES = {
     # width, layers, heads / kv heads / head size of the attention, inner width of the feed-forward, vocabulary
@@ -487,8 +487,8 @@ _TIMED_OPS = ("linear", "linear_stacked", "linear_for_residual", "linear_swiglu"
               "streams_update_norm", "add_rmsnorm", "swiglu", "qk_norm_mix_kv_write", "qk_norm_rope_kv_write", "embed_gather", "lightning_attention",
               "qkv_rotate_write", "latent_norm_rotate_write", "rotate_heads", "linear_heads", "state_space", "expert_mixture", "mean_of_normed",
               "gated_unit", "add_bias", "concat_cast", "linear_recurrence", "matrix_memory", "weighted_sum", "residual_add",
-              "min_gru", "output_norm", "embedding_norm")
-DESIGNS = ("vopepel", "qwen3", "fikerax", "zemavik", "rirusun", "zabusun")
+              "min_gru", "output_norm", "embedding_norm", "join_norm")
+DESIGNS = ("vopepel", "qwen3", "fikerax", "zemavik", "rirusun", "zabusun", "pinedra")
 
 
 def vopepel_fields(size: dict) -> dict:
@@ -584,6 +584,23 @@ def zabusun_fields(size: dict) -> dict:
                      "rot": {"dims": dim // 2, "base": 500_000.0, "scaling": {"factor": 8.0, "original": 4_096, "fast": 32.0, "slow": 1.0}}},
             "left_scale": 1.0, "right": {"width": size["width"]}, "right_scale": 1.0}}
     return {"architecture": "Zabusun", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5}, "logit_scale": 1.0,
+            "layers": [layer(index) for index in range(size["layers"])]}
+
+
+def pinedra_fields(size: dict) -> dict:
+    """A Pinedra model of the given size: of every three layers the first has slopes, a sink and the queries' factor, the second values that are
+    its keys, the third half of every head rotated, a soft cap and chunks of 1,024 positions; every layer's feed-forward is a mixture of 8 experts
+    of half the inner width and 2 that hand their input back, in 5 groups of which 2 are kept and a token uses 2 experts, and a shared expert of
+    the same width; no layer runs twice, so that the depth is the other designs'."""
+    def layer(index: int) -> dict:
+        dim = size["head_dim"]
+        sizes = {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": dim, "vdim": dim, "scale": dim ** -0.5}
+        kind, more = (("attention_2", {"q_temp": {"coef": 0.1, "every": 1_024}}), ("attention", {}),
+                      ("attention_3", {"rot": {"dims": dim // 2, "base": 500_000.0}, "softcap": 30.0, "mask": {"size": 1_024}}))[index % 3]
+        return {"type": kind, "mixer": {**sizes, **more}, "mlp": {
+            "kind": "moe", "expert": {"ff": size["ff"] // 2}, "router": {"experts": 8, "top": 2, "identity": 2, "scale": 2.0, "groups": {"count": 5, "keep": 2}},
+            "shared": {"ff": size["ff"] // 2}}}
+    return {"architecture": "Pinedra", "vocab": size["vocab"], "width": size["width"], "embedding": {"scale": size["width"] ** 0.5}, "norm": {"eps": 1e-5},
             "layers": [layer(index) for index in range(size["layers"])]}
 
 
@@ -703,21 +720,22 @@ def time_design(engine, torch, ops, rng, batch: int, steps: int) -> dict:
 
 
 def run_design_comparison(torch, sizes, batch: int, steps: int, designs=DESIGNS) -> dict:
-    """Vopepel, Fikerax, Zemavik, Rirusun, Zabusun and Qwen3 dense at equal width, depth, heads, feed-forward and vocabulary: prefill and decode throughput
+    """Vopepel, Fikerax, Zemavik, Rirusun, Zabusun, Pinedra and Qwen3 dense at equal width, depth, heads, feed-forward and vocabulary: prefill and decode throughput
     and the time of every kernel entry point, random weights."""
     import gc
 
     import numpy as np
 
     from pylon_b200.config import EngineConfig, Qwen3Config
-    from pylon_b200.config.model_config import FikeraxConfig, RirusunConfig, VopepelConfig, ZabusunConfig, ZemavikConfig
+    from pylon_b200.config.model_config import FikeraxConfig, PinedraConfig, RirusunConfig, VopepelConfig, ZabusunConfig, ZemavikConfig
     from pylon_b200.engine import Engine
     from pylon_b200.kernels import ops
 
     peak = peaks()
     made = {"vopepel": lambda size: VopepelConfig.from_dict(vopepel_fields(size)), "qwen3": lambda size: Qwen3Config(**qwen3_fields(size)),
             "fikerax": lambda size: FikeraxConfig.from_dict(fikerax_fields(size)), "zemavik": lambda size: ZemavikConfig.from_dict(zemavik_fields(size)),
-            "rirusun": lambda size: RirusunConfig.from_dict(rirusun_fields(size)), "zabusun": lambda size: ZabusunConfig.from_dict(zabusun_fields(size))}
+            "rirusun": lambda size: RirusunConfig.from_dict(rirusun_fields(size)), "zabusun": lambda size: ZabusunConfig.from_dict(zabusun_fields(size)),
+            "pinedra": lambda size: PinedraConfig.from_dict(pinedra_fields(size))}
     record = {"metric": "prefill and decode, " + ", ".join(designs) + " at equal size", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16",
               "data": "synthetic: random weights, uniform random token ids, caches filled by real prefill",
               "config": {"prefill_tokens": PREFILL_TOKENS, "decode_batch": batch, "decode_context": DESIGN_CONTEXT, "decode_steps": steps,
@@ -794,7 +812,7 @@ def main() -> int:
     parser.add_argument("--skip-points", action="store_true", help="leave out the batch 1 and 64 points")
     parser.add_argument("--workload", choices=["decode4b", "mixed8b", "sampled14b", "designs"], default="decode4b",
                         help="decode4b: the headline measurement (default); mixed8b, sampled14b: the serving workloads of the 8B and 14B shapes; "
-                             "designs: Vopepel, Fikerax, Zemavik, Rirusun and Zabusun beside Qwen3 at equal size, prefill and decode with the time of every kernel entry point")
+                             "designs: Vopepel, Fikerax, Zemavik, Rirusun, Zabusun and Pinedra beside Qwen3 at equal size, prefill and decode with the time of every kernel entry point")
     parser.add_argument("--design-sizes", default="2k,4k", help="with --workload designs: which of the sizes 2k, 4k")
     parser.add_argument("--designs", default=",".join(DESIGNS), help="with --workload designs: which of " + ", ".join(DESIGNS))
     parser.add_argument("--profile", choices=["decode", "prefill"],

@@ -123,7 +123,7 @@ def draw_mixer(rand, matrix, kind, m, width):
 def draw_mixture(rand, matrix, mlp, width):
     router, ff = mlp["router"], mlp["expert"]["ff"]
     choices = router["experts"] + router.get("identity", 0)
-    w = {"router": matrix(choices, width, 1.2), "correction": 0.15 * rand(choices) - 0.2}
+    w = {"router": matrix(choices, width, 1.2), "correction": rand(choices) / choices - 0.2}
     for name, inner in [(f"e{e}.", ff) for e in range(router["experts"])] + ([] if mlp.get("shared") is None else [("shared.", mlp["shared"]["ff"])]):
         w[name + "gate"], w[name + "up"], w[name + "down"] = matrix(inner, width, 1.6), matrix(inner, width, 1.6), matrix(width, inner)
     return w
@@ -286,7 +286,7 @@ def test_bfloat16_generation_from_graphs_follows_the_plain_logits(models):
 # ---------------------------------------------------------------------------------------
 # mixers alone
 # ---------------------------------------------------------------------------------------
-SIZES = {"narrow": (4, 2, 20, 12, 0.35), "equal": (6, 2, 32, 32, 0.3), "wider": (3, 1, 8, 24, 0.5), "cores": (8, 2, 64, 64, 0.15), "odd": (2, 2, 5, 3, 0.6)}
+SIZES = {"narrow": (4, 2, 20, 12, 0.35), "equal": (6, 2, 32, 32, 0.3), "wider": (3, 1, 8, 24, 0.5), "cores": (8, 2, 64, 64, 0.15), "odd": (2, 2, 5, 3, 0.35)}
 MIXER_NAMES = ["attention-equal", "attention-odd", "attention-cores", "attention_2-narrow", "attention_2-wider", "attention_2-cores", "attention_2-odd",
                "attention_3-narrow", "attention_3-wider", "attention_3-cores", "attention_3-odd"]
 
