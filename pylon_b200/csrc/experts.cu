@@ -30,14 +30,18 @@
 //   experts_plan      one block: tokens per expert, the experts' first tiles, a slot for every pair
 //   experts_product   a block per (row tile, column tile): rows gathered by slot, the expert's matrix, float32 sums in a
 //                     fixed order of k; with GLU the gate and up tiles side by side and act(gate) * up written
-//   experts_product_mma   the same on tensor cores (bfloat16, mma.sync m16n8k16), the matrices through a ring of cp.async stages:
-//                     the products of a step of few tokens
+//   experts_product_mma   the same on tensor cores (bfloat16, mma.sync m16n8k16), the matrices through a ring of cp.async stages
+//   experts_stream    the products of a step of few tokens where the matrices' rows can be fetched by TMA: as experts_product_mma, the
+//                     matrices as 64 x 64 boxes in a ring that TMA fills, the rows gathered into it beside them
 //   experts_sort_rows the tokens' rows copied into the order of their slots, for a step of many tokens: its products are the
 //                     grouped form of the tcgen05 kernel (gemm_tcgen05.cu) over row tiles of 128 slots
 //   experts_gather    out[t] = sum_k share[t, k] * y[slot(t, k)], float32
 // A row's sums do not depend on where in a tile it lies or what else is in the batch.
 #include "common.cuh"
-#include <mma.h>
+#include <cuda.h>
+
+#include <mutex>
+#include <unordered_map>
 
 namespace pylon {
 
@@ -199,7 +203,7 @@ __device__ __forceinline__ void route_choose_scored(float* logits, float* choice
 // columns.  A thread takes V neighbouring columns at a time (V 4 where the rows are whole pieces of it, else 1; by the sizes alone): warp k's
 // lane l adds up the columns V (128 i + 32 k + l) .. + V - 1 in order of i, its 32 lanes' sums are added by a butterfly, and the four warps'
 // sums in order of k.  So a token's logits, and with them its choice, do not depend on how many tokens the step has.
-// Shared memory: TOKENS * (4 * 8 + what a token takes) floats.
+// Shared memory: TOKENS * (4 * ROUTE_SIDE + what a token takes) floats.
 template <typename T, int V>
 __device__ __forceinline__ void route_load(float (&x)[V], const T* from) {
   if constexpr (V == 1) x[0] = to_float<T>(from[0]);
@@ -213,56 +217,73 @@ __device__ __forceinline__ void route_load(float (&x)[V], const T* from) {
   }
 }
 
+constexpr int ROUTE_SIDE = 8;   // router rows side by side at most: the tokens' rows are read once per so many
+
+// The logits of the block's tokens for router rows e0 .. e0 + SIDE - 1 (those below `rows`).
+template <typename T, int TOKENS, int V, int SIDE>
+__device__ __forceinline__ void route_logits(const T* __restrict__ h, long long ld, const float* __restrict__ router, const float* __restrict__ bias, float* parts,
+                                             float* logits, int per_token, int t0, int num_tokens, int width, int e0, int rows, int experts) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float acc[TOKENS][SIDE];
+#pragma unroll
+  for (int i = 0; i < TOKENS; ++i)
+#pragma unroll
+    for (int j = 0; j < SIDE; ++j) acc[i][j] = 0.f;
+#pragma unroll(TOKENS == 1 ? 4 : 2)
+  for (int c = V * threadIdx.x; c < width; c += V * 128) {
+    float x[TOKENS][V], r[SIDE][V];
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i) route_load<T, V>(x[i], h + (long long)(t0 + i < num_tokens ? t0 + i : t0) * ld + c);
+#pragma unroll
+    for (int j = 0; j < SIDE; ++j) route_load<float, V>(r[j], router + (long long)(e0 + j < rows ? e0 + j : e0) * width + c);
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i)
+#pragma unroll
+      for (int j = 0; j < SIDE; ++j)
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[i][j] = fmaf(x[i][v], r[j][v], acc[i][j]);
+  }
+#pragma unroll
+  for (int i = 0; i < TOKENS; ++i)
+#pragma unroll
+    for (int j = 0; j < SIDE; ++j) {
+      const float z = warp_sum(acc[i][j]);
+      if (lane == 0) parts[(warp * TOKENS + i) * SIDE + j] = z;
+    }
+  __syncthreads();
+  if (threadIdx.x < TOKENS * SIDE) {
+    const int i = threadIdx.x / SIDE, j = threadIdx.x % SIDE;
+    if (e0 + j < rows)
+      logits[i * per_token + e0 + j] = ((parts[i * SIDE + j] + parts[(TOKENS + i) * SIDE + j]) + parts[(2 * TOKENS + i) * SIDE + j]) + parts[(3 * TOKENS + i) * SIDE + j] +
+                                       (bias != nullptr && e0 + j < experts ? bias[e0 + j] : 0.f);
+  }
+  __syncthreads();
+}
+
 template <typename T, int TOKENS, int V>
 __global__ void __launch_bounds__(128) experts_route_kernel(const T* __restrict__ h, long long ld, const float* __restrict__ router, const float* __restrict__ bias,
                                                             int* __restrict__ chosen, float* __restrict__ share, int width, int experts, int top, int num_tokens,
                                                             int always, RouteScored mode) {
   extern __shared__ float route_shared[];
-  constexpr int SIDE = 8;   // experts side by side: the tokens' rows are read once per eight experts
   const int rows = experts + mode.extra;                                        // rows of the router
   const int per_token = rows + (mode.on ? experts + mode.groups : 0);           // logits, then with mode.on choice scores and the groups' worths
-  float* parts = route_shared;                                                  // [4][TOKENS][SIDE]
-  float* logits = route_shared + 4 * TOKENS * SIDE;                             // [TOKENS][per_token]
-  grid_dependency_wait();
-  allow_dependents();
+  float* parts = route_shared;                                                  // [4][TOKENS][ROUTE_SIDE]
+  float* logits = route_shared + 4 * TOKENS * ROUTE_SIDE;                       // [TOKENS][per_token]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t0 = blockIdx.x * TOKENS;
-  for (int e0 = 0; e0 < rows; e0 += SIDE) {
-    float acc[TOKENS][SIDE];
-#pragma unroll
-    for (int i = 0; i < TOKENS; ++i)
-#pragma unroll
-      for (int j = 0; j < SIDE; ++j) acc[i][j] = 0.f;
-#pragma unroll 2
-    for (int c = V * threadIdx.x; c < width; c += V * 128) {
-      float x[TOKENS][V], r[SIDE][V];
-#pragma unroll
-      for (int i = 0; i < TOKENS; ++i) route_load<T, V>(x[i], h + (long long)(t0 + i < num_tokens ? t0 + i : t0) * ld + c);
-#pragma unroll
-      for (int j = 0; j < SIDE; ++j) route_load<float, V>(r[j], router + (long long)(e0 + j < rows ? e0 + j : e0) * width + c);
-#pragma unroll
-      for (int i = 0; i < TOKENS; ++i)
-#pragma unroll
-        for (int j = 0; j < SIDE; ++j)
-#pragma unroll
-          for (int v = 0; v < V; ++v) acc[i][j] = fmaf(x[i][v], r[j][v], acc[i][j]);
-    }
-#pragma unroll
-    for (int i = 0; i < TOKENS; ++i)
-#pragma unroll
-      for (int j = 0; j < SIDE; ++j) {
-        const float z = warp_sum(acc[i][j]);
-        if (lane == 0) parts[(warp * TOKENS + i) * SIDE + j] = z;
-      }
-    __syncthreads();
-    if (threadIdx.x < TOKENS * SIDE) {
-      const int i = threadIdx.x / SIDE, j = threadIdx.x % SIDE;
-      if (e0 + j < rows)
-        logits[i * per_token + e0 + j] = ((parts[i * SIDE + j] + parts[(TOKENS + i) * SIDE + j]) + parts[(2 * TOKENS + i) * SIDE + j]) + parts[(3 * TOKENS + i) * SIDE + j] +
-                                         (bias != nullptr && e0 + j < experts ? bias[e0 + j] : 0.f);
-    }
-    __syncthreads();
+  if (TOKENS == 1) {   // the router's rows are nobody's work: on their way to L2 before the wait for the kernel ahead
+    const long long bytes = (long long)rows * width * 4;
+    for (long long at = (long long)threadIdx.x * 128; at < bytes; at += 128 * 128) asm volatile("prefetch.global.L2 [%0];\n" ::"l"((const char*)router + at));
   }
+  grid_dependency_wait();
+  allow_dependents();
+  int e0 = 0;
+  for (; rows - e0 > ROUTE_SIDE / 2; e0 += ROUTE_SIDE)
+    route_logits<T, TOKENS, V, ROUTE_SIDE>(h, ld, router, bias, parts, logits, per_token, t0, num_tokens, width, e0, rows, experts);
+  if (e0 < rows && rows - e0 <= 2)        // the few rows that are left
+    route_logits<T, TOKENS, V, 2>(h, ld, router, bias, parts, logits, per_token, t0, num_tokens, width, e0, rows, experts);
+  else if (e0 < rows)
+    route_logits<T, TOKENS, V, ROUTE_SIDE / 2>(h, ld, router, bias, parts, logits, per_token, t0, num_tokens, width, e0, rows, experts);
   for (int i = warp; i < TOKENS && t0 + i < num_tokens; i += 4) {
     float* mine = logits + i * per_token;
     const int per = top + always;
@@ -539,6 +560,168 @@ __global__ void __launch_bounds__(128) experts_product_mma_kernel(const __nv_bfl
     }
 }
 
+// ---------------------------------------------------------------------------------------------
+// The products of a step of few tokens, the matrices by TMA.  A block takes 64 weight rows of one expert (with GLU: 32 gate rows and their up
+// rows, alternating in groups of 8) and a row tile of 32 slots.  Warp 0 fills a ring: its first lane asks TMA for the 64 x 64 box of the
+// matrix (128-byte swizzle), every lane copies its own slot's 128 bytes beside it (cp.async, in the same swizzle), and both complete on the
+// stage's one mbarrier (33 arrivals).  Four consumer warps, 16 weight rows each, multiply with mma.sync, the weights as the 16-row A operand,
+// the slots as 8-column B operands - as many of them as the tile holds.  Rows of empty slots are never filled: a column of the product depends
+// on its own slot alone, and theirs are not written.  Every wait is bounded (error word 1: the producer, 2: a consumer gave up); a block that
+// gives up waits for the copies it asked for before it leaves.  Bound by the matrices coming from memory: 64 KB in flight a block, three to
+// an SM.  (The ring of cp.async stages reaches 3.3 TB/s.)
+// ---------------------------------------------------------------------------------------------
+constexpr int ES_SLAB = 64, ES_BK = 64, ES_CONSUMERS = 4, ES_THREADS = 32 * (1 + ES_CONSUMERS), ES_STAGES = 5;
+constexpr int ES_W_BYTES = ES_SLAB * ES_BK * 2, ES_STAGE_BYTES = ES_W_BYTES + EXPERT_ROWS * ES_BK * 2;
+constexpr size_t ES_SMEM = (size_t)ES_STAGES * ES_STAGE_BYTES + 1024 /* alignment slack */ + 128 /* barriers */;
+constexpr unsigned ES_WAIT_LIMIT = 1u << 22;
+enum ExpertStreamForm { ES_SUMS = 0, ES_GATED = 1, ES_ACTIVATED = 2 };
+
+__device__ __forceinline__ unsigned es_smem(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ bool es_wait(uint64_t* bar, unsigned parity) {
+  for (unsigned tries = 0; tries < ES_WAIT_LIMIT; ++tries) {
+    unsigned done;
+    asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\nselp.u32 %0, 1, 0, p;\n}\n"
+                 : "=r"(done) : "r"(es_smem(bar)), "r"(parity) : "memory");
+    if (done) return true;
+  }
+  return false;
+}
+__device__ __forceinline__ void es_ldmatrix(unsigned (&r)[4], unsigned address) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(address));
+}
+__device__ __forceinline__ void es_mma(float (&c)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// Grid (slabs of 64 weight rows, row tiles, parts of k).  map_w: the stacked matrices [experts * w_rows, k_size] in boxes of 64 x 64.
+template <int FORM>
+__global__ void __launch_bounds__(ES_THREADS, 3) experts_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __nv_bfloat16* __restrict__ a, long long lda,
+                                                                        const int* __restrict__ source, const int* __restrict__ tile_expert, int gathered, int divide,
+                                                                        void* __restrict__ out_v, int n_out, int k_size, int w_rows, int kind,
+                                                                        const float* __restrict__ slot_share, float limit, float alpha, int k_each, long long part_stride,
+                                                                        int* __restrict__ error) {
+  constexpr int TILES = EXPERT_ROWS / 8;
+  extern __shared__ unsigned char es_shared[];
+  unsigned char* stages = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(es_shared) + 1023) & ~(uintptr_t)1023);
+  uint64_t* full = reinterpret_cast<uint64_t*>(stages + (size_t)ES_STAGES * ES_STAGE_BYTES);
+  uint64_t* empty = full + ES_STAGES;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int tile = blockIdx.y, n0 = blockIdx.x * ES_SLAB;
+  if (threadIdx.x == 0) {
+#pragma unroll
+    for (int s = 0; s < ES_STAGES; ++s) {
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;\n" ::"r"(es_smem(&full[s])), "r"(33));
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;\n" ::"r"(es_smem(&empty[s])), "r"(ES_CONSUMERS));
+    }
+    asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
+  }
+  __syncthreads();
+  grid_dependency_wait();
+  allow_dependents();
+  const int expert = tile_expert[tile];
+  if (expert < 0) return;
+  const int pair = source[tile * EXPERT_ROWS + lane];   // every warp knows the tile's slots, one a lane; the filled ones come first
+  const int filled = __popc(__ballot_sync(0xffffffffu, pair >= 0));
+  const int k_first = blockIdx.z * k_each;
+  const int k_last = k_first + k_each < k_size ? k_first + k_each : k_size;
+  const int boxes = (k_last - k_first + ES_BK - 1) / ES_BK;
+
+  if (warp == 0) {
+    const __nv_bfloat16* row = pair < 0 ? nullptr : a + (long long)(gathered ? pair / divide : tile * EXPERT_ROWS + lane) * lda + k_first;
+    unsigned stage = 0, phase = 0;
+    for (int box = 0; box < boxes; ++box) {
+      if (box >= ES_STAGES && !es_wait(&empty[stage], phase ^ 1)) {
+        if (lane == 0) atomicExch(error, 1);
+        break;
+      }
+      unsigned char* to = stages + (size_t)stage * ES_STAGE_BYTES;
+      if (lane == 0) {
+        asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");   // the consumers read the stage with ordinary loads: TMA is another proxy
+        asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(es_smem(&full[stage])), "r"(ES_W_BYTES) : "memory");
+        asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];\n"
+                     ::"r"(es_smem(to)), "l"((unsigned long long)&map_w), "r"(es_smem(&full[stage])), "r"(k_first + box * ES_BK), "r"(expert * w_rows + n0) : "memory");
+      }
+      if (row) {
+        unsigned char* mine = to + ES_W_BYTES + lane * 128;
+#pragma unroll
+        for (int unit = 0; unit < 8; ++unit) {
+          const int k = box * ES_BK + unit * 8;
+          const bool real = k_first + k < k_last;
+          copy_16_or_zeros(mine + ((unit ^ (lane & 7)) << 4), real ? row + k : row, real);
+        }
+      }
+      asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];\n" ::"r"(es_smem(&full[stage])) : "memory");
+      if (++stage == ES_STAGES) { stage = 0; phase ^= 1; }
+    }
+    asm volatile("cp.async.wait_all;\n" ::: "memory");
+    return;
+  }
+
+  // In the 128-byte swizzle the 16-byte unit u of row r sits at unit u ^ (r % 8).
+  const int slab_row = (warp - 1) * 16 + (lane & 7) + 8 * ((lane >> 3) & 1);
+  const unsigned w_row_offset = (unsigned)slab_row * 128, w_xor = (unsigned)(slab_row & 7);
+  const unsigned x_row_offset = (unsigned)ES_W_BYTES + (unsigned)(lane & 7) * 128, x_xor = (unsigned)(lane & 7);
+  float acc[TILES][2][4];   // per 8 slots: even and odd k-steps, two MMA chains
+#pragma unroll
+  for (int j = 0; j < TILES; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[j][0][i] = acc[j][1][i] = 0.f;
+  unsigned stage = 0, phase = 0;
+  for (int box = 0; box < boxes; ++box) {
+    if (!es_wait(&full[stage], phase)) {
+      if (lane == 0) atomicExch(error, 2);
+      return;
+    }
+    const unsigned here = es_smem(stages + (size_t)stage * ES_STAGE_BYTES);
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {   // 32 k each
+      unsigned w[2][4];
+#pragma unroll
+      for (int step = 0; step < 2; ++step)    // 16 k each
+        es_ldmatrix(w[step], here + w_row_offset + ((((unsigned)(4 * half + 2 * step) + (lane >> 4)) ^ w_xor) << 4));
+#pragma unroll
+      for (int j = 0; j < TILES; ++j) {
+        if (8 * j >= filled) break;            // the same for every lane
+        unsigned x[4];                         // units 4 * half .. + 3 of slots 8j .. 8j + 7
+        es_ldmatrix(x, here + (unsigned)(j * 8 * 128) + x_row_offset + ((((unsigned)(4 * half) + (lane >> 3)) ^ x_xor) << 4));
+        es_mma(acc[j][0], w[0], x[0], x[1]);
+        es_mma(acc[j][1], w[1], x[2], x[3]);
+      }
+    }
+    __syncwarp();
+    if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(es_smem(&empty[stage])) : "memory");
+    if (++stage == ES_STAGES) { stage = 0; phase ^= 1; }
+  }
+
+  // Accumulator element i of lane (group, quad): weight row group + 8 * (i / 2), slot 2 * quad + (i % 2) of its eight.
+  const int group = lane >> 2, quad = lane & 3;
+  const int row0 = n0 + (warp - 1) * 16 + group;
+#pragma unroll
+  for (int j = 0; j < TILES; ++j) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int m = j * 8 + 2 * quad + e;
+      if (m >= filled) continue;
+      const long long slot = (long long)tile * EXPERT_ROWS + m;
+      const float low = acc[j][0][e] + acc[j][1][e], high = acc[j][0][2 + e] + acc[j][1][2 + e];
+      if (FORM == ES_GATED) {   // rows row0 (gate) and row0 + 8 (its up row)
+        const int n = (n0 + (warp - 1) * 16) / 2 + group;
+        const float reads = slot_share ? slot_share[slot] : 1.f;
+        if (n < n_out) ((__nv_bfloat16*)out_v)[slot * n_out + n] = __float2bfloat16_rn(expert_unit(reads * low, reads * high, kind, limit, alpha));
+      } else if (FORM == ES_ACTIVATED) {
+        if (row0 < n_out) ((__nv_bfloat16*)out_v)[slot * n_out + row0] = __float2bfloat16_rn(expert_activation(low, kind));
+        if (row0 + 8 < n_out) ((__nv_bfloat16*)out_v)[slot * n_out + row0 + 8] = __float2bfloat16_rn(expert_activation(high, kind));
+      } else {
+        float* out = (float*)out_v + blockIdx.z * part_stride + slot * n_out;
+        if (row0 < n_out) out[row0] = low;
+        if (row0 + 8 < n_out) out[row0 + 8] = high;
+      }
+    }
+  }
+}
+
 // share null: the rows are added up as they are.
 // out[t, c] = sum_k share[t, k] * y[slot_of[t * top + k], c], the choices in their order; y in float32 or in the compute dtype.
 // With `same` (rows in C, same_ld apart) and same_share (float32 [T]): + same_share[t] * same[t, c].  A slot of -1 is none.
@@ -609,7 +792,7 @@ extern "C" int pylon_experts_route(const void* h, long long ld, const float* rou
   const bool pieces = width % 4 == 0 && ld % 4 == 0 && (uintptr_t)h % (4 * element) == 0 && (uintptr_t)router % 16 == 0;
 #define PYLON_ROUTE(T, TOKENS, V)                                                                                                            \
   launch_dependent(experts_route_kernel<T, TOKENS, V>, dim3((unsigned)((num_tokens + TOKENS - 1) / TOKENS)), dim3(128),                      \
-                   (size_t)TOKENS * (4 * 8 + per_token) * sizeof(float), stream, (const T*)h, ld, router, bias, chosen, share, width, experts, top, num_tokens, always, mode)
+                   (size_t)TOKENS * (4 * ROUTE_SIDE + per_token) * sizeof(float), stream, (const T*)h, ld, router, bias, chosen, share, width, experts, top, num_tokens, always, mode)
 #define PYLON_ROUTE_SIZES(T)                                                                                                                 \
   if (few) { if (pieces) PYLON_ROUTE(T, 1, 4); else PYLON_ROUTE(T, 1, 1); }                                                                  \
   else { if (pieces) PYLON_ROUTE(T, 4, 4); else PYLON_ROUTE(T, 4, 1); }
@@ -634,6 +817,62 @@ extern "C" int pylon_experts_plan(const int* chosen, int* slot_of, int* source, 
   PYLON_CHECK_LAUNCH("experts_plan");
 }
 
+typedef CUresult (*EncodeTiled)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+// The stacked matrices [rows, cols], contiguous, in boxes of 64 x 64 in the 128-byte swizzle.  Maps are kept by their arguments: a model
+// multiplies by the same matrices at every step.
+static bool stacked_map(CUtensorMap* map, const void* base, long long rows, long long cols) {
+  struct Key {
+    const void* base; long long rows, cols;
+    bool operator==(const Key& o) const { return base == o.base && rows == o.rows && cols == o.cols; }
+  };
+  struct Hash {
+    size_t operator()(const Key& k) const { return std::hash<const void*>()(k.base) ^ (size_t)(k.rows * 1315423911LL) ^ (size_t)(k.cols * 2654435761LL); }
+  };
+  static std::unordered_map<Key, CUtensorMap, Hash> known;
+  static std::mutex mutex;
+  std::lock_guard<std::mutex> guard(mutex);
+  const Key key{base, rows, cols};
+  auto found = known.find(key);
+  if (found != known.end()) { *map = found->second; return true; }
+  static EncodeTiled encode = [] {
+    void* symbol = nullptr;
+    cudaDriverEntryPointQueryResult result;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &symbol, cudaEnableDefault, &result) != cudaSuccess || result != cudaDriverEntryPointSuccess) symbol = nullptr;
+    return (EncodeTiled)symbol;
+  }();
+  if (!encode) return false;
+  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+  cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+  cuuint32_t box[2] = {(cuuint32_t)ES_BK, (cuuint32_t)ES_SLAB};
+  cuuint32_t element_strides[2] = {1, 1};
+  if (encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, element_strides, CU_TENSOR_MAP_INTERLEAVE_NONE,
+             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+    return false;
+  if (known.size() >= 4096) known.clear();
+  known.emplace(key, *map);
+  return true;
+}
+
+template <int FORM>
+static int launch_experts_stream(const CUtensorMap& map_w, const __nv_bfloat16* a, long long lda, const int* source, const int* tile_expert, int gathered, int divide,
+                                 void* out, int n_out, int k_size, int w_rows, int max_tiles, int kind, const float* slot_share, float limit, float alpha, int k_parts,
+                                 int* error, cudaStream_t stream) {
+  static bool configured_on[pylon::MAX_DEVICES] = {};   // function attributes belong to a device
+  bool& configured = configured_on[pylon::current_device_slot()];
+  if (!configured) {
+    cudaError_t err = cudaFuncSetAttribute(experts_stream_kernel<FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ES_SMEM);
+    if (err != cudaSuccess) PYLON_REFUSE("experts_stream: %s", cudaGetErrorString(err));
+    configured = true;
+  }
+  launch_dependent(experts_stream_kernel<FORM>, dim3((unsigned)((w_rows + ES_SLAB - 1) / ES_SLAB), (unsigned)max_tiles, (unsigned)k_parts), dim3(ES_THREADS), ES_SMEM, stream,
+                   map_w, a, lda, source, tile_expert, gathered, divide, out, n_out, k_size, w_rows, kind, slot_share, limit, alpha, k_size / k_parts,
+                   (long long)max_tiles * EXPERT_ROWS * n_out, error);
+  PYLON_CHECK_LAUNCH("experts_stream");
+}
+
 template <bool GLU>
 static void allow_mma_shared_memory() {
   static bool configured_on[pylon::MAX_DEVICES] = {};   // function attributes belong to a device
@@ -647,9 +886,11 @@ static void allow_mma_shared_memory() {
 // or, interleaved != 0, alternating in groups of 8); out: [max_tiles * EXPERT_ROWS, n_out], in dtype with glu, else float32.
 // k_parts > 1 (a plain bfloat16 product): k in so many equal parts, out float32 [k_parts, max_tiles * EXPERT_ROWS, n_out] whose sum the product is.
 // glu == 2: no gate, but the activation on the product itself, out in dtype (the first product of an ungated expert).
+// experts: how many matrices w holds; error: one int that a kernel sets when a bounded wait of it ran out (the output is then void), or null: the
+// form whose matrices come by TMA is then not taken.
 extern "C" int pylon_experts_product(const void* a, long long lda, const void* w, const int* source, const int* tile_expert, int gathered,
                                      int divide, void* out, int n_out, int k_size, int max_tiles, int glu, int kind, int interleaved, int dtype,
-                                     const float* slot_share, float limit, float alpha, int k_parts, cudaStream_t stream) {
+                                     const float* slot_share, float limit, float alpha, int k_parts, int experts, int* error, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
   const int act_out = glu == 2 ? 1 : 0;
   if (act_out) glu = 0;
@@ -668,6 +909,16 @@ extern "C" int pylon_experts_product(const void* a, long long lda, const void* w
     const __nv_bfloat16* ab = (const __nv_bfloat16*)a;
     const __nv_bfloat16* wb = (const __nv_bfloat16*)w;
     const bool vectors = k_size % 8 == 0 && lda % 8 == 0 && (uintptr_t)a % 16 == 0 && (uintptr_t)w % 16 == 0;
+    const int w_rows = glu ? 2 * n_out : n_out;
+    if (vectors && error && experts > 0 && (!glu || interleaved) && (long long)experts * w_rows < 2147483647LL - ES_SLAB) {
+      CUtensorMap map_w;
+      if (!stacked_map(&map_w, w, (long long)experts * w_rows, k_size)) PYLON_REFUSE("experts_product: the tensor map of the matrices could not be made");
+#define PYLON_STREAM(FORM) return launch_experts_stream<FORM>(map_w, ab, lda, source, tile_expert, gathered, divide, out, n_out, k_size, w_rows, max_tiles, kind, slot_share, limit, alpha, k_parts, error, stream)
+      if (glu) PYLON_STREAM(ES_GATED);
+      if (act_out) PYLON_STREAM(ES_ACTIVATED);
+      PYLON_STREAM(ES_SUMS);
+#undef PYLON_STREAM
+    }
     if (vectors) {
       if (glu) {
         allow_mma_shared_memory<true>();

@@ -68,7 +68,7 @@ __device__ __forceinline__ float4 four_of(const void* from, int parts, long long
 
 // HELD: the 4-column pieces a thread keeps.
 template <typename T, int HELD>
-__global__ void __launch_bounds__(512) join_norm_vec_kernel(const JoinParams p) {
+__global__ void __launch_bounds__(512, HELD > 2 ? 1 : 2) join_norm_vec_kernel(const JoinParams p) {
   __shared__ float scratch[34];
   const int pieces = p.width / 4;
   float4 w[HELD];   // weights and bias are nobody's work: on their way before the wait for the kernel ahead
@@ -86,6 +86,18 @@ __global__ void __launch_bounds__(512) join_norm_vec_kernel(const JoinParams p) 
   grid_dependency_wait();
   allow_dependents();
   const long long t = p.rows ? p.rows[blockIdx.x] : blockIdx.x;
+  // Where the token's first rows lie, asked for before all else: the loads of the rows wait for nothing but these.
+  constexpr int SIDE = 4 / HELD;   // rows of a token on their way at once: more of them cost more in registers than they gain
+  int slot[SIDE];
+  float share[SIDE];
+  auto find = [&](int first) {
+#pragma unroll
+    for (int j = 0; j < SIDE; ++j) {
+      slot[j] = first + j < p.top ? p.slot_of[t * p.top + first + j] : -1;
+      share[j] = first + j < p.top && p.share ? p.share[t * p.top + first + j] : 1.f;
+    }
+  };
+  if (p.slot_of) find(0);
   float4 x[HELD], ff[HELD];
   const float same_share = p.same ? p.same_share[t] : 0.f;
 #pragma unroll
@@ -100,14 +112,26 @@ __global__ void __launch_bounds__(512) join_norm_vec_kernel(const JoinParams p) 
     if (p.y && !p.slot_of) add_4(ff[i], four_of<T>(p.y, p.y_parts, p.y_stride, at));
   }
   if (p.slot_of) {
-    for (int k = 0; k < p.top; ++k) {
-      const int slot = p.slot_of[t * p.top + k];
-      if (slot < 0) continue;
-      const float share = p.share ? p.share[t * p.top + k] : 1.f;
+    for (int first = 0; first < p.top; first += SIDE) {
+      if (first > 0) find(first);
+      const int parts = p.y_parts > 0 ? p.y_parts : 1;
+      for (int part = 0; part < parts; ++part) {
+        float4 row[HELD][SIDE];   // all of them on their way at once
 #pragma unroll
-      for (int i = 0; i < HELD; ++i) {
-        const int piece = threadIdx.x + i * blockDim.x;
-        if (piece < pieces) add_4_times(ff[i], share, four_of<T>(p.y, p.y_parts, p.y_stride, (long long)slot * p.width + 4 * piece));
+        for (int i = 0; i < HELD; ++i) {
+          const int piece = threadIdx.x + i * blockDim.x;
+#pragma unroll
+          for (int j = 0; j < SIDE; ++j) {
+            row[i][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (slot[j] < 0 || piece >= pieces) continue;
+            const long long at = (long long)slot[j] * p.width + 4 * piece;
+            row[i][j] = p.y_parts > 0 ? four<float>(p.y, part * p.y_stride + at) : four<T>(p.y, at);
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < HELD; ++i)
+#pragma unroll
+          for (int j = 0; j < SIDE; ++j) add_4_times(ff[i], share[j], row[i][j]);
       }
     }
   }
@@ -192,13 +216,14 @@ extern "C" int pylon_join_norm(float* x, const void* a, int a_parts, const float
   const JoinParams p{x, a, a_parts, (long long)tokens * width, bias, y, y_parts, y_rows * width, slot_of, share, slot_of ? top : 1, same, same_ld, same_share, weight, rows, out, width, eps};
   // threads by the width alone, so that a token's sum does not depend on the step
   int threads = 64;
-  while (threads < 512 && threads * 2 < width / 4) threads *= 2;
+  while (threads < 512 && threads < width / 4) threads *= 2;
   const uintptr_t piece = dtype == PYLON_DTYPE_F32 ? 16 : 8;
   const bool pieces = width % 4 == 0 && same_ld % 4 == 0 && width / 4 <= threads * 4 && (uintptr_t)x % 16 == 0 && (uintptr_t)a % (a_parts ? 16 : piece) == 0 &&
                       (uintptr_t)y % (y_parts ? 16 : piece) == 0 && (uintptr_t)same % piece == 0 && (uintptr_t)out % piece == 0 && (uintptr_t)weight % 16 == 0 && (uintptr_t)bias % 16 == 0;
   const size_t row_bytes = (size_t)width * sizeof(float);
 #define PYLON_JOIN_NORM(T)                                                                                                                        \
-  if (pieces && width / 4 <= threads * 2) launch_dependent(join_norm_vec_kernel<T, 2>, dim3((unsigned)n_rows), dim3(threads), 0, stream, p);      \
+  if (pieces && width / 4 <= threads) launch_dependent(join_norm_vec_kernel<T, 1>, dim3((unsigned)n_rows), dim3(threads), 0, stream, p);          \
+  else if (pieces && width / 4 <= threads * 2) launch_dependent(join_norm_vec_kernel<T, 2>, dim3((unsigned)n_rows), dim3(threads), 0, stream, p); \
   else if (pieces) launch_dependent(join_norm_vec_kernel<T, 4>, dim3((unsigned)n_rows), dim3(threads), 0, stream, p);                             \
   else launch_dependent(join_norm_kernel<T>, dim3((unsigned)n_rows), dim3(256), row_bytes, stream, p)
   if (dtype == PYLON_DTYPE_F32) { PYLON_JOIN_NORM(float); } else { PYLON_JOIN_NORM(__nv_bfloat16); }

@@ -234,7 +234,7 @@ _SIGNATURES = {
                                 c_float, c_int, c_int, c_void_p, c_int, c_float, c_int, c_void_p, c_int, c_void_p],
         "pylon_experts_plan": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "pylon_experts_product": [c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_int, c_void_p, c_float, c_float, c_int, c_void_p],
+                                  c_int, c_void_p, c_float, c_float, c_int, c_int, c_void_p, c_void_p],
         "pylon_experts_sort_rows": [c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "pylon_experts_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p,
                                  c_longlong, c_void_p, c_void_p],
@@ -1849,11 +1849,12 @@ def expert_mixture(h: torch.Tensor, router: torch.Tensor, router_bias: Optional[
         return out
     act = torch.empty((max_slots, inner), dtype=h.dtype, device=device)
     _check(library, library.pylon_experts_product(_ptr(h), h.stride(0), _ptr(w_gate_up), _ptr(source), _ptr(tile_expert), 1, per, _ptr(act), inner, width,
-                                                  max_tiles, 1 if gated else 2, kind, int(interleaved), code, _ptr(slot_share), limit, float(alpha), 1, _stream()))
+                                                  max_tiles, 1 if gated else 2, kind, int(interleaved), code, _ptr(slot_share), limit, float(alpha), 1,
+                                                  experts, _ptr(stream_error_word(device)), _stream()))
     parts = _expert_parts(experts, width, inner, _multiprocessors(device)) if h.dtype == torch.bfloat16 else 1
     y = torch.empty((parts, max_slots, width), dtype=torch.float32, device=device)
     _check(library, library.pylon_experts_product(_ptr(act), inner, _ptr(w_down), _ptr(source), _ptr(tile_expert), 0, 1, _ptr(y), width, inner,
-                                                  max_tiles, 0, kind, 0, code, None, 0.0, 1.0, parts, _stream()))
+                                                  max_tiles, 0, kind, 0, code, None, 0.0, 1.0, parts, experts, _ptr(stream_error_word(device)), _stream()))
     if scattered:
         return ScatteredRows(y, slot_of, per, out_share, same, same_share)
     out = torch.empty((1, tokens, width), dtype=torch.float32, device=device)
