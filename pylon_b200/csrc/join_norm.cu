@@ -160,10 +160,9 @@ __global__ void __launch_bounds__(512, HELD > 2 ? 1 : 2) join_norm_vec_kernel(co
   }
 }
 
-// Any width and alignment.  The new sum is kept in shared memory [width].
+// Any width and alignment; the sum is formed a second time for the result where it was not written.
 template <typename T>
 __global__ void __launch_bounds__(256) join_norm_kernel(const JoinParams p) {
-  extern __shared__ float join_row[];
   __shared__ float scratch[34];
   grid_dependency_wait();
   allow_dependents();
@@ -174,8 +173,7 @@ __global__ void __launch_bounds__(256) join_norm_kernel(const JoinParams p) {
     for (int part = 0; part < parts; ++part) sum += ((const float*)from)[part * stride + at];
     return sum;
   };
-  float squares = 0.f;
-  for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
+  auto sum = [&](int c) {
     const long long at = t * p.width + c;
     float mixer = p.bias ? p.bias[c] : 0.f, ff = 0.f;
     if (p.a) mixer += value(p.a, p.a_parts, p.a_stride, at);
@@ -187,14 +185,18 @@ __global__ void __launch_bounds__(256) join_norm_kernel(const JoinParams p) {
         if (slot >= 0) ff = fmaf(p.share ? p.share[t * p.top + k] : 1.f, value(p.y, p.y_parts, p.y_stride, (long long)slot * p.width + c), ff);
       }
     }
-    const float x = p.x[at] + (mixer + ff);
-    if (!p.rows) p.x[at] = x;
-    if (p.weight) join_row[c] = x;
+    return p.x[at] + (mixer + ff);
+  };
+  float squares = 0.f;
+  for (int c = threadIdx.x; c < p.width; c += blockDim.x) {
+    const float x = sum(c);
+    if (!p.rows) p.x[t * p.width + c] = x;
     squares = fmaf(x, x, squares);
   }
   if (!p.weight) return;
   const float inv = 1.f / sqrtf(block_sum(squares, scratch) / p.width + p.eps);
-  for (int c = threadIdx.x; c < p.width; c += blockDim.x) ((T*)p.out)[(long long)blockIdx.x * p.width + c] = from_float<T>(join_row[c] * inv * p.weight[c]);
+  for (int c = threadIdx.x; c < p.width; c += blockDim.x)
+    ((T*)p.out)[(long long)blockIdx.x * p.width + c] = from_float<T>((p.rows ? sum(c) : p.x[t * p.width + c]) * inv * p.weight[c]);
 }
 
 }  // namespace pylon
@@ -209,7 +211,7 @@ extern "C" int pylon_join_norm(float* x, const void* a, int a_parts, const float
                                const float* share, int top, const void* same, long long same_ld, const float* same_share, const float* weight, const int* rows,
                                void* out, int n_rows, int tokens, int width, float eps, int dtype, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
-  if (width < 1 || width > 12000 || a_parts < 0 || y_parts < 0 || (!rows && n_rows != tokens) || (weight != nullptr) != (out != nullptr) || (rows && !weight))
+  if (width < 1 || a_parts < 0 || y_parts < 0 || (!rows && n_rows != tokens) || (weight != nullptr) != (out != nullptr) || (rows && !weight))
     PYLON_REFUSE("join_norm: width %d, %d and %d parts, %d of %d rows", width, a_parts, y_parts, n_rows, tokens);
   if ((slot_of && (!y || top < 1 || y_rows < 1)) || (share && !slot_of) || (same != nullptr) != (same_share != nullptr)) PYLON_REFUSE("join_norm: experts' rows without slots, or shares without rows");
   if (dtype != PYLON_DTYPE_F32 && dtype != PYLON_DTYPE_BF16) PYLON_REFUSE("join_norm: unknown dtype %d", dtype);
@@ -220,12 +222,11 @@ extern "C" int pylon_join_norm(float* x, const void* a, int a_parts, const float
   const uintptr_t piece = dtype == PYLON_DTYPE_F32 ? 16 : 8;
   const bool pieces = width % 4 == 0 && same_ld % 4 == 0 && width / 4 <= threads * 4 && (uintptr_t)x % 16 == 0 && (uintptr_t)a % (a_parts ? 16 : piece) == 0 &&
                       (uintptr_t)y % (y_parts ? 16 : piece) == 0 && (uintptr_t)same % piece == 0 && (uintptr_t)out % piece == 0 && (uintptr_t)weight % 16 == 0 && (uintptr_t)bias % 16 == 0;
-  const size_t row_bytes = (size_t)width * sizeof(float);
 #define PYLON_JOIN_NORM(T)                                                                                                                        \
   if (pieces && width / 4 <= threads) launch_dependent(join_norm_vec_kernel<T, 1>, dim3((unsigned)n_rows), dim3(threads), 0, stream, p);          \
   else if (pieces && width / 4 <= threads * 2) launch_dependent(join_norm_vec_kernel<T, 2>, dim3((unsigned)n_rows), dim3(threads), 0, stream, p); \
   else if (pieces) launch_dependent(join_norm_vec_kernel<T, 4>, dim3((unsigned)n_rows), dim3(threads), 0, stream, p);                             \
-  else launch_dependent(join_norm_kernel<T>, dim3((unsigned)n_rows), dim3(256), row_bytes, stream, p)
+  else launch_dependent(join_norm_kernel<T>, dim3((unsigned)n_rows), dim3(256), 0, stream, p)
   if (dtype == PYLON_DTYPE_F32) { PYLON_JOIN_NORM(float); } else { PYLON_JOIN_NORM(__nv_bfloat16); }
 #undef PYLON_JOIN_NORM
   PYLON_CHECK_LAUNCH("join_norm");

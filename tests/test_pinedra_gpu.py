@@ -654,7 +654,7 @@ def test_the_mixture_against_token_by_token(width, tokens, mlp, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("width", [1, 30, 72, 200, 2048, 4096, 8192, 9000])
+@pytest.mark.parametrize("width", [1, 30, 72, 200, 2048, 4096, 8192, 9000, 16384])
 def test_outputs_side_by_side_join_the_stream_in_one_pass(width, dtype):
     """Every form of the two outputs - a block, partial sums of one part to five, rows in slots with and without shares, some of them nowhere, rows
     handed back, nothing - with and without a bias, with the norm, without it, and with a selection of rows that leaves the stream as it is."""
