@@ -104,3 +104,44 @@ def test_norm_and_sampling():
     top_p = torch.tensor([0.95, 0.9, 1.0, 0.5] * 2, device=DEVICE)
     uniform = torch.rand(8, device=DEVICE)
     assert same_bits(lambda: ops.sample(logits, temperature, top_p, uniform), 500) == 0
+
+
+@pytest.mark.parametrize("tokens", [1, 8, 70])
+def test_experts_of_few_tokens(tokens):
+    """The experts' products whose matrices come by TMA and whose rows are gathered beside them: gated ones and ungated ones with their activation,
+    rings that go round, parts of k; and the join of what they leave with the stream."""
+    from pylon_b200.kernels import ops
+
+    torch.manual_seed(tokens)
+    make = lambda *shape: (torch.randn(*shape, device=DEVICE) * 0.02).to(torch.bfloat16)
+    width, inner, experts = 1_024, 2_048, 6
+    h, residual = torch.randn(tokens, width, device=DEVICE).to(torch.bfloat16), torch.randn(tokens, width, device=DEVICE)
+    router, correction, weight = torch.randn(experts + 1, width, device=DEVICE) * 0.05, torch.zeros(experts + 1, device=DEVICE), torch.ones(width, device=DEVICE)
+    gate_up, down, up = make(experts, 2 * inner, width), make(experts, width, inner), make(experts, inner, width)
+    options = dict(routing="softmax_all", share_normalized=False, group_score="best", share_scale=1.5, correction=correction, identity=2, always=1)
+    mixture = lambda: ops.expert_mixture(h, router, None, gate_up, down, 2, "silu", True, **options)
+    assert same_bits(mixture, 1_000) == 0
+
+    def joined():
+        stream = residual.clone()
+        rows = ops.expert_mixture(h, router, None, gate_up, down, 2, "silu", True, scattered=True, **options)
+        return torch.cat((stream, ops.join_norm(stream, ops.SideBySide(h, None, rows), weight, 1e-5, torch.bfloat16).float()))
+
+    assert same_bits(joined, 500) == 0
+    ungated = lambda: ops.expert_mixture(h, router[:experts].contiguous(), None, up, down, 2, "gelu", gated=False, routing="sigmoid")
+    assert same_bits(ungated, 500) == 0
+    ops.raise_on_kernel_errors(torch.device(DEVICE))
+
+
+def test_attention_with_a_softmaxs_options():
+    from pylon_b200.kernels import ops
+
+    nq, nkv, d = 32, 8, 128
+    slopes, sinks = torch.tensor([2.0 ** (-8.0 * (h + 1) / nq) for h in range(nq)], device=DEVICE), torch.zeros(nq, device=DEVICE)
+    for lengths, new, alike, calls in (([2_048], 2_048, True, 200), ([2_000] * 4, 1, True, 1_000), ([700, 3_000, 1_500, 90], 1, False, 1_000)):
+        cache = Paged(lengths, [new] * len(lengths), nkv, d, 256, torch.bfloat16, seed=6)
+        q, gate = (torch.randn(new * len(lengths), nq * d, device=DEVICE).to(torch.bfloat16) for _ in range(2))
+        call = lambda: ops.paged_attention(q, cache.k_pages, cache.v_pages, cache.positions, cache.token_row, cache.q_start, cache.kv_len, cache.table, nq, new, max(lengths),
+                                           rows_alike=alike, head_gate=gate, distance_slopes=slopes, sinks=sinks, row_tokens=[new] * len(lengths))
+        assert same_bits(call, calls) == 0, (lengths, new)
+    ops.raise_on_kernel_errors(torch.device(DEVICE))
